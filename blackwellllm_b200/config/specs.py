@@ -80,6 +80,14 @@ class RMSNormSpec:
 
 
 @dataclass(frozen=True)
+class LayerNormSpec:
+    """(x - mean) / sqrt(mean of the squared deviations + eps) * weight, without a bias."""
+    eps: float
+    kind: str = "layernorm"
+    param: str = "weight"   # the weight's name below the norm's prefix
+
+
+@dataclass(frozen=True)
 class AttentionSpec:
     """Grouped-query softmax attention over a paged key/value cache.
 
@@ -140,6 +148,13 @@ class AttentionSpec:
     distance_table_rows: Optional[int] = None
     fixed_sink: Optional[float] = None
     value_mix: Optional[str] = None
+    # ``qk_norm`` = "unit": every query and key head is divided by its root mean square (``qk_norm_eps`` under the root) AFTER
+    # the rotation, without gains.  ``values_from_keys``: there is no value projection; the key projection as it is, before
+    # norm and rotation, is the value (the value size is ``head_dim``).  ``head_temperature``: a learned number per query head
+    # (tensor "temp" [heads]) multiplies the head's scores.  ``output_scale``: a constant the mixer's output is multiplied by.
+    values_from_keys: bool = False
+    head_temperature: bool = False
+    output_scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -206,6 +221,60 @@ class GatedLinearAttentionSpec:
 
 
 @dataclass(frozen=True)
+class GatedDeltaSpec:
+    """A recurrent mixer with a [key_dim, value_dim] state per head that follows the gated delta rule:
+    ``S <- g S``, ``u = beta (v - S^T k)``, ``S <- S + k u^T``, ``o = S^T q``.  q, k (``num_kv_heads`` heads, head h of v uses
+    number floor(h / (num_heads / num_kv_heads))) and v pass a causal convolution over time of ``conv_taps`` columns per
+    channel and silu; q and k become unit vectors per head (eps 1e-6 under the root of the sum of squares), q times
+    key_dim ** -0.5; ``beta = sigmoid(W_b x)``, ``g = exp(-exp(A_log) softplus(W_a x + dt_bias))``, one of each per head.  Each
+    head's o is RMS-normed over value_dim with a gain shared by the heads, multiplied by ``silu(W_g x)`` and projected.
+    ``output_scale``: a constant the mixer's output is multiplied by.  ``names``: (role, name) pairs for q, k, v, b, a, g, o,
+    norm, q_conv, k_conv, v_conv, A_log, dt_bias."""
+    num_heads: int
+    num_kv_heads: int
+    key_dim: int
+    value_dim: int
+    conv_taps: int
+    norm_eps: float
+    output_scale: float = 1.0
+    kind: str = "gated_delta"
+    names: Tuple[Tuple[str, str], ...] = ()
+
+
+@dataclass(frozen=True)
+class StateSpaceSpec:
+    """A state-space mixer with one decay per head (Mamba-2): ``W_in x`` is [z: inner | x: inner | B: groups * state_dim |
+    C: groups * state_dim | dt: heads], inner = num_heads * value_dim; x, B and C together pass a causal convolution over
+    time of ``conv_taps`` columns per channel with a bias, then silu; ``dt <- softplus(dt + dt_bias)``; head h uses group
+    floor(h / (num_heads / groups)): ``S <- exp(-exp(A_log) dt) S + dt B x^T``, ``y = S^T C + D x``; the heads side by side
+    times ``silu(z)``, RMS-normed in ``norm_groups`` equal parts, times a gain per channel, then projected.
+    ``names``: (role, name) pairs for in, conv, conv_bias, dt_bias, A_log, D, norm, o."""
+    num_heads: int
+    value_dim: int
+    state_dim: int
+    groups: int
+    conv_taps: int
+    norm_groups: int
+    norm_eps: float
+    kind: str = "state_space"
+    names: Tuple[Tuple[str, str], ...] = ()
+
+
+@dataclass(frozen=True)
+class SideBySideSpec:
+    """Two mixers that read the same input, their tensors below ``prefixes``.  ``combine``: "sum" (their outputs added; a
+    factor on either is the child's ``output_scale``) or "norm_mean" (half the sum of the two outputs, each RMS-normed over
+    the width with a gain of its own, tensors ``out_norms``, eps ``norm_eps``)."""
+    left: Any
+    right: Any
+    combine: str = "sum"
+    norm_eps: float = 0.0
+    kind: str = "side_by_side"
+    prefixes: Tuple[str, str] = ("left.", "right.")
+    out_norms: Tuple[str, str] = ("left.out", "right.out")
+
+
+@dataclass(frozen=True)
 class RoutedFFNSpec:
     """Mixture of experts: ``num_experts`` gated feed-forwards ``down(silu(gate u) * (up u))`` without biases,
     of which each token uses the ``top_k`` with the largest router scores.  ``score``: "sigmoid" or
@@ -255,7 +324,7 @@ class SwiGLUSpec:
 
 @dataclass(frozen=True)
 class DenseMLPSpec:
-    """Dense feed-forward without a gate: down(act(up(x))); ``activation`` "relu2": max(z, 0)^2."""
+    """Dense feed-forward without a gate: down(act(up(x))); ``activation`` "relu2": max(z, 0)^2; "gelu": 0.5 z (1 + erf(z / sqrt(2)))."""
     intermediate_size: int
     activation: str = "relu2"
     kind: str = "dense_mlp"
@@ -305,8 +374,11 @@ class LayerSpec:
     # token; the feed-forward reads h_t as it is), and the block keeps h of a request's last token between steps.
     token_shift: Optional[str] = None
     # the "parallel" arrangement: the names of two vectors [hidden] ("layer scale"); the mixer's output is multiplied
-    # channel by channel by the first and the feed-forward's by the second before they are added to the stream
+    # channel by channel by the first and the feed-forward's by the second before they are added to the stream.  In the
+    # "sandwich" arrangement the outputs are multiplied after their second norms.  ``residual_mult`` ("sandwich"): a constant
+    # that multiplies both on top of that.
     layer_scale: Optional[Tuple[str, str]] = None
+    residual_mult: float = 1.0
 
 
 @dataclass(frozen=True)

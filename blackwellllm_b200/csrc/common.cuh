@@ -24,10 +24,12 @@
 //   BW_ACT_CLAMPED_SWISH  gated:  g' = min(g, limit), u' = clamp(u, -limit, limit):  g' sigmoid(alpha g') (u' + 1)
 //   BW_ACT_RELU2          no gate: max(x, 0)^2
 //   BW_ACT_GELU_TANH      gated:  0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))) * u
+//   BW_ACT_GELU           no gate: 0.5 x (1 + erf(x / sqrt(2)))
 #define BW_ACT_SILU 0
 #define BW_ACT_CLAMPED_SWISH 1
 #define BW_ACT_RELU2 2
 #define BW_ACT_GELU_TANH 3
+#define BW_ACT_GELU 4
 
 // Programmatic dependent launch: a kernel launched through bw::launch may start while the kernel
 // before it in the stream is still draining.  Such a kernel calls BW_PDL_TRIGGER() early (the next
@@ -180,7 +182,20 @@ __device__ __forceinline__ float glu(int act, float g, float u, float limit, flo
 }
 __device__ __forceinline__ float unary_act(int act, float x) {
     if (act == BW_ACT_RELU2) { const float r = fmaxf(x, 0.f); return r * r; }
+    if (act == BW_ACT_GELU) return 0.5f * x * (1.f + erff(x * 0.70710678118654752f));
     return x;
+}
+// The same gelu for results that are rounded to 16 bits: erf by formula 7.1.26 of Abramowitz and Stegun, Handbook of
+// Mathematical Functions (absolute error below 1.5e-7): erf(z) = 1 - (a1 t + .. + a5 t^5) exp(-z^2), t = 1 / (1 + 0.3275911 z).
+__device__ __forceinline__ float gelu_fast(float x) {
+    const float z = fabsf(x) * 0.70710678118654752f;
+    const float t = __fdividef(1.f, fmaf(0.3275911f, z, 1.f));
+    float q = fmaf(1.061405429f, t, -1.453152027f);
+    q = fmaf(q, t, 1.421413741f);
+    q = fmaf(q, t, -0.284496736f);
+    q = fmaf(q, t, 0.254829592f);
+    const float tail = q * t * __expf(-z * z);        // 1 - erf(z)
+    return 0.5f * x * (x >= 0.f ? 2.f - tail : tail);
 }
 
 // The output gate of an attention mixer: sigmoid(gate[token, head * dv + c]) for c < dv, 0 for the pad channels beyond

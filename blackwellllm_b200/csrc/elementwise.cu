@@ -305,7 +305,7 @@ __global__ void swiglu_kernel(const IT* __restrict__ gu, OT* __restrict__ out, i
     }
 }
 
-// An activation without a gate, element by element: BW_ACT_RELU2: max(x, 0)^2.
+// An activation without a gate, element by element: BW_ACT_RELU2: max(x, 0)^2; BW_ACT_GELU: 0.5 x (1 + erf(x / sqrt(2))).
 template <typename IT, typename OT>
 __global__ void unary_act_kernel(const IT* __restrict__ x, OT* __restrict__ out, size_t total, int act) {
     BW_PDL_TRIGGER();
@@ -723,10 +723,10 @@ BW_EXPORT int bw_glu(const void* gu, int in_type, void* out, int out_type, int T
     return launch_glu(gu, in_type, out, out_type, T, I, act, limit, alpha, stream);
 }
 
-// out[i] = act(x[i]) over n elements; act: BW_ACT_RELU2
+// out[i] = act(x[i]) over n elements; act: BW_ACT_RELU2 or BW_ACT_GELU
 BW_EXPORT int bw_unary_act(const void* x, int in_type, void* out, int out_type, long long n, int act, void* stream) {
     if (n <= 0) return 0;
-    if (act != BW_ACT_RELU2) return BW_ERR_BAD_ARG;
+    if (act != BW_ACT_RELU2 && act != BW_ACT_GELU) return BW_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = 256;
     const int blocks = (int)((n + threads - 1) / threads < 148 * 16 ? (n + threads - 1) / threads : 148 * 16);

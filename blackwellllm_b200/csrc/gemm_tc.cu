@@ -77,7 +77,7 @@ struct Epilogue {
     int stream;           // the k-blocks of all tiles, laid end to end, are cut into one equal range per CTA
     int planes;           // split-K: the partial planes ARE the result (the bias in plane 0); whoever reads them adds them up
     // an activation of common.cuh on the finished sums.  With swiglu: the gated one that replaces silu(g) * u
-    // (BW_ACT_SILU, BW_ACT_CLAMPED_SWISH with its limit and alpha); without: 0 = none, BW_ACT_RELU2 on every value.
+    // (BW_ACT_SILU, BW_ACT_CLAMPED_SWISH with its limit and alpha); without: 0 = none, BW_ACT_RELU2 or BW_ACT_GELU on every value.
     int act; float act_limit, act_alpha;
     RopeOut rope;
 };
@@ -94,6 +94,7 @@ __device__ __forceinline__ float ep_glu(const Epilogue& ep, float g, float u) {
 }
 __device__ __forceinline__ float ep_unary(const Epilogue& ep, float v) {
     if (ep.act == BW_ACT_RELU2) { v = fmaxf(v, 0.f); return v * v; }
+    if (ep.act == BW_ACT_GELU) return bw::gelu_fast(v);
     return v;
 }
 
@@ -1199,8 +1200,8 @@ static int run_gemm_tc(const void* x, const void* w, const void* bias, int bias_
                        int force_splits, const RopeOut* rope, void* stream, int* planes_out = nullptr,
                        int act = 0, float act_limit = 0.f, float act_alpha = 1.f) {
     if (M <= 0 || N <= 0) return 0;
-    // act: with swiglu the gated activation (BW_ACT_SILU, BW_ACT_CLAMPED_SWISH or BW_ACT_GELU_TANH); without, 0 or BW_ACT_RELU2 on the sums
-    if (swiglu ? (act != BW_ACT_SILU && act != BW_ACT_CLAMPED_SWISH && act != BW_ACT_GELU_TANH) : (act != 0 && act != BW_ACT_RELU2)) return BW_ERR_BAD_ARG;
+    // act: with swiglu the gated activation (BW_ACT_SILU, BW_ACT_CLAMPED_SWISH or BW_ACT_GELU_TANH); without, 0, BW_ACT_RELU2 or BW_ACT_GELU on the sums
+    if (swiglu ? (act != BW_ACT_SILU && act != BW_ACT_CLAMPED_SWISH && act != BW_ACT_GELU_TANH) : (act != 0 && act != BW_ACT_RELU2 && act != BW_ACT_GELU)) return BW_ERR_BAD_ARG;
     if (!swiglu && act != 0 && (accumulate || rope || planes_out)) return BW_ERR_BAD_ARG;
     // planes_out: the product is left as *planes_out float32 planes [M, N] in `out` (row stride N, the bias
     // in the first), to be added up by its reader; K is split as if the sums were made here.
@@ -1325,7 +1326,7 @@ BW_EXPORT int bw_gemm_tc(const void* x, const void* w, const void* bias, int bia
 
 // bw_gemm_tc with an activation on the finished sums: with swiglu the gated activation `act` in place of
 // silu(gate) * up (BW_ACT_CLAMPED_SWISH: g sigmoid(alpha g) (u + 1) on the clamped gate and up); without swiglu
-// BW_ACT_RELU2 on every value of a result that is written (not added).
+// BW_ACT_RELU2 or BW_ACT_GELU on every value of a result that is written (not added).
 BW_EXPORT int bw_gemm_tc_act(const void* x, const void* w, const void* bias, int bias_type, void* out, int out_type,
                              int M, int N, int K, long long ldx, long long ldo, int swiglu, int act, float act_limit,
                              float act_alpha, float* workspace, long long workspace_elems, int* counters,

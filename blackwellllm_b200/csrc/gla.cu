@@ -48,6 +48,7 @@ struct ScanParams {
     const float* k_scale;
     int scalar_decay, ones_col;
     int sld;               // floats between the state's rows (>= dv; columns from dv on stay zero)
+    int rep;               // head h reads query/key head h / rep (heads / rep of them; the plain form has rep == 1)
 };
 
 __device__ __forceinline__ float log_sigmoid(float z) {
@@ -81,7 +82,8 @@ gla_decay_kernel(const float* __restrict__ x, long long ldx, int x_off, const WT
 // and used for CPT columns.  In shared memory a token's rows are padded with zeros to DKP = 32 * RPL channels
 // (a padded channel stays at zero and adds nothing), so the inner loop has no bounds.  The CPT sums over the
 // 32 lanes take six shuffles: two that halve the number of columns a lane carries, then three over what is left.
-// MEM: the form for a matrix memory (ScanParams: one decay per head, keys times k_scale, the column of ones); the plain
+// MEM: the form for a matrix memory (ScanParams: one decay per head, keys times k_scale, the column of ones, query/key
+// heads shared by several heads); the plain
 // form's code does not know of it.  What a fetch loads is not touched before it is staged: a thread never waits for a
 // load inside the fetch, so the key's scale travels in registers of its own and multiplies at staging.
 template <int RPL, bool MEM>
@@ -100,6 +102,7 @@ gla_scan_kernel(ScanParams p) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int cbase = c0 + warp * CPT;
     const int t0 = p.cu_q[r], t1 = p.cu_q[r + 1];
+    const int hk = MEM ? h / p.rep : h;
     float* S = p.state + (((size_t)p.state_slot[r] * p.heads + h) * p.dk) * p.sld;
     BW_PDL_WAIT();
     float s[RPL][CPT];
@@ -129,8 +132,8 @@ gla_scan_kernel(ScanParams p) {
             if constexpr (MEM) rs[u] = 1.f;
             if (tt < n && i < p.dk) {
                 const float* row = p.qkv + (size_t)(tb + tt) * p.ld;
-                rq[u] = row[p.q_off + h * p.dk + i];
-                rk[u] = row[p.k_off + h * p.dk + i];
+                rq[u] = row[p.q_off + hk * p.dk + i];
+                rk[u] = row[p.k_off + hk * p.dk + i];
                 if constexpr (MEM) {
                     if (p.k_scale) rs[u] = p.k_scale[(size_t)(tb + tt) * p.heads + h];
                     ra[u] = p.scalar_decay ? p.decay[(size_t)(tb + tt) * p.heads + h]
@@ -240,23 +243,27 @@ gla_gate_kernel(const float* __restrict__ o, const float* __restrict__ g, long l
 // decay: float32 [T, heads * dk] from bw_gla_decay; with scalar_decay [T, heads].  k_scale: float32 [T, heads] or null.
 // ones_col != 0: dv counts a last column of ones that v does not hold (state [slots, heads, dk, state_ld], o [T, heads * dv]).
 // state_ld: floats between the state's rows (0: dv); with a multiple of 4 a lane moves its columns of a row in one access.
+// qk_rep: head h uses query/key head h / qk_rep (1: every head has its own).
 BW_EXPORT int bw_gla_scan(const float* qkv, long long ld, int q_off, int k_off, int v_off, const float* decay,
                           const int* cu_q, const int* state_slot, float* state, float* o, int R, int heads, int dk,
                           int dv, float q_scale, const float* k_scale, int scalar_decay, int ones_col, int state_ld,
-                          void* stream) {
+                          int qk_rep, void* stream) {
     if (R <= 0) return 0;
-    if (heads <= 0 || dk <= 0 || dv <= 0 || (ones_col && dv < 2) || (state_ld != 0 && state_ld < dv)) return BW_ERR_BAD_ARG;
+    if (heads <= 0 || dk <= 0 || dv <= 0 || (ones_col && dv < 2) || (state_ld != 0 && state_ld < dv) ||
+        qk_rep <= 0 || heads % qk_rep)
+        return BW_ERR_BAD_ARG;
     if (dk > MAX_DK) return BW_ERR_UNSUPPORTED;
     ScanParams p;
     p.qkv = qkv; p.decay = decay; p.cu_q = cu_q; p.state_slot = state_slot; p.state = state; p.o = o; p.ld = ld;
     p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.heads = heads; p.dk = dk; p.dv = dv;
     p.q_scale = q_scale;
     p.k_scale = k_scale; p.scalar_decay = scalar_decay; p.ones_col = ones_col; p.sld = state_ld ? state_ld : dv;
+    p.rep = qk_rep;
     const dim3 grid(R, heads, (dv + COLS - 1) / COLS);
     const int rpl = dk <= 128 ? 4 : 8;
     const size_t smem = (size_t)(3 * TOK_CHUNK * 32 * rpl + TOK_CHUNK * COLS) * sizeof(float);
     cudaStream_t s = (cudaStream_t)stream;
-    const bool mem = k_scale || scalar_decay || ones_col;
+    const bool mem = k_scale || scalar_decay || ones_col || qk_rep > 1;
     if (rpl == 4) {
         if (mem) bw::launch((gla_scan_kernel<4, true>), grid, dim3(THREADS), smem, s, p);
         else bw::launch((gla_scan_kernel<4, false>), grid, dim3(THREADS), smem, s, p);

@@ -103,7 +103,9 @@ __device__ __forceinline__ void put4(bf16* p, float4 v) {
 // has_kv == 0: a run that reads another run's keys and values projects none.  One block per token, one warp
 // per head at a time; all arithmetic float32.  v_first != null: the values become (1 - lam) v + lam v_first on their way
 // into the cache, v_first being float32 rows `v_first_ld` apart with nkv * dv values of the same token (another layer's
-// values of this step) and lam = *v_lam a number on the device.
+// values of this step) and lam = *v_lam a number on the device.  q_head_mult != null: every query head is multiplied by its
+// own number (float32 [nh]).  v_col: the column where the values' heads begin (behind the keys, or the keys' own columns:
+// values that are the key projection before norm and rotation).  v_scale multiplies the values last of all.
 template <typename OT>
 __global__ void __launch_bounds__(256)
 head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __restrict__ positions,
@@ -113,11 +115,12 @@ head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __
                       float q_coef, float q_every,
                       OT* __restrict__ q_out, OT* __restrict__ k_pages, OT* __restrict__ v_pages,
                       int nh, int nkv, int dq, int dv, int dpad, int page_size, int num_pages, int has_kv, int vec,
-                      float v_eps, const float* __restrict__ v_first, long long v_first_ld, const float* __restrict__ v_lam) {
+                      float v_eps, const float* __restrict__ v_first, long long v_first_ld, const float* __restrict__ v_lam,
+                      const float* __restrict__ q_head_mult, int v_col, float v_scale) {
     BW_PDL_TRIGGER();
     const int t = blockIdx.x;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
-    const int nq = nh * dq, nk = nkv * dq;
+    const int nq = nh * dq;
     const int pos = positions[t];
     int page = -1;
     const int slot = pos % page_size;
@@ -143,7 +146,7 @@ head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __
             for (int c = lane; c < dq; c += 32) { const float v = src[c]; ss = fmaf(v, v, ss); }
             r = rsqrtf(bw::warp_sum(ss) / (float)dq + eps);
         }
-        const float mult = is_q ? q_mult : 1.f;
+        const float mult = is_q ? (q_head_mult ? q_mult * q_head_mult[h] : q_mult) : 1.f;
         OT* dst = is_q ? q_out + ((size_t)t * nh + h) * dpad
                        : k_pages + (((size_t)page * nkv + (h - nh)) * page_size + slot) * dpad;
         if (vec) {
@@ -180,7 +183,7 @@ head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __
         }
     }
     // a value as it is cached: mixed with the same token's value of another layer where the launch says so
-    const float* vsrc = row + nq + nk;
+    const float* vsrc = row + v_col;
     const float* vf = v_first ? v_first + (size_t)t * v_first_ld : nullptr;
     const float lam = v_first ? *v_lam : 0.f;
     auto value = [&](size_t i) { const float v = vsrc[i]; return vf ? (1.f - lam) * v + lam * vf[i] : v; };
@@ -191,7 +194,7 @@ head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __
             for (int c = lane; c < dv; c += 32) { const float v = value((size_t)h * dv + c); ss = fmaf(v, v, ss); }
             const float r = rsqrtf(bw::warp_sum(ss) / (float)dv + v_eps);
             OT* dst = v_pages + (((size_t)page * nkv + h) * page_size + slot) * dpad;
-            for (int c = lane; c < dpad; c += 32) dst[c] = bw::from_f32<OT>(c < dv ? value((size_t)h * dv + c) * r : 0.f);
+            for (int c = lane; c < dpad; c += 32) dst[c] = bw::from_f32<OT>(c < dv ? value((size_t)h * dv + c) * r * v_scale : 0.f);
         }
         return;
     }
@@ -199,14 +202,15 @@ head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __
         if (vec && !vf) {
             for (int idx = threadIdx.x * 4; idx < nkv * dpad; idx += blockDim.x * 4) {
                 const int h = idx / dpad, c = idx - h * dpad;
-                const float4 o = c < dv ? *reinterpret_cast<const float4*>(vsrc + (size_t)h * dv + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+                float4 o = c < dv ? *reinterpret_cast<const float4*>(vsrc + (size_t)h * dv + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+                o.x *= v_scale; o.y *= v_scale; o.z *= v_scale; o.w *= v_scale;
                 put4(v_pages + (((size_t)page * nkv + h) * page_size + slot) * dpad + c, o);
             }
             return;
         }
         for (int idx = threadIdx.x; idx < nkv * dpad; idx += blockDim.x) {
             const int h = idx / dpad, c = idx - h * dpad;
-            const float o = c < dv ? value((size_t)h * dv + c) : 0.f;
+            const float o = c < dv ? value((size_t)h * dv + c) * v_scale : 0.f;
             v_pages[(((size_t)page * nkv + h) * page_size + slot) * dpad + c] = bw::from_f32<OT>(o);
         }
     }
@@ -217,18 +221,21 @@ head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __
 // The per-head form (head_norm_rope_kernel).  ld: floats between rows of qkv; q_gain / k_gain: float32 [dq] or
 // null; q_coef, q_every: the queries' temperature (q_coef == 0: none; q_every > 0); has_kv == 0: the rows hold
 // no keys and values and nothing is appended.  v_eps > 0: every value head is divided by sqrt(mean(v^2) + v_eps) on its way
-// into the cache.  v_first, v_first_ld, v_lam: the value mixing (see the kernel), or nulls.
+// into the cache.  v_first, v_first_ld, v_lam: the value mixing (see the kernel), or nulls.  q_head_mult: float32 [nh] or
+// null; kv_shared != 0: the rows hold no values, the keys' columns (before norm and rotation) are the values (dv == dq);
+// v_scale: a factor on the values as they are cached.
 BW_EXPORT int bw_head_norm_rope_append(const float* qkv, long long ld, const int* positions, const int* req_of_token,
                                        const int* block_table, int max_blocks, const float* table, int rotary_dim,
                                        int interleaved, const float* q_gain, const float* k_gain, float eps,
                                        float q_coef, float q_every, void* q_out, void* k_pages, void* v_pages,
                                        int out_type, int T, int nh, int nkv, int dq, int dv, int dpad, int page_size,
                                        int num_pages, int has_kv, float v_eps, const float* v_first, long long v_first_ld,
-                                       const float* v_lam, void* stream) {
+                                       const float* v_lam, const float* q_head_mult, int kv_shared, float v_scale, void* stream) {
     if (T <= 0) return 0;
+    if (kv_shared && (dv != dq || !has_kv || v_first)) return BW_ERR_BAD_ARG;
     if (rotary_dim < 0 || rotary_dim > dq || (rotary_dim & 1) || dq <= 0 || dv <= 0 || dpad < dq || dpad < dv ||
         nh <= 0 || nkv <= 0 || page_size <= 0 || (rotary_dim > 0 && !table) || (q_coef != 0.f && !(q_every > 0.f)) ||
-        ld < (long long)nh * dq + (has_kv ? (long long)nkv * (dq + dv) : 0) ||
+        ld < (long long)nh * dq + (has_kv ? (long long)nkv * (kv_shared ? dq : dq + dv) : 0) ||
         (v_first && (!v_lam || !has_kv || v_first_ld < (long long)nkv * dv)))
         return BW_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
@@ -236,7 +243,8 @@ BW_EXPORT int bw_head_norm_rope_append(const float* qkv, long long ld, const int
                     (((uintptr_t)qkv | (uintptr_t)q_gain | (uintptr_t)k_gain | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages) & 15) == 0;
 #define BW_HN(OT) bw::launch((head_norm_rope_kernel<OT>), dim3(T), dim3(256), 0, s, qkv, ld, positions, req_of_token, block_table, \
         max_blocks, table, rotary_dim, interleaved, q_gain, k_gain, eps, q_coef, q_every, (OT*)q_out, (OT*)k_pages, (OT*)v_pages, \
-        nh, nkv, dq, dv, dpad, page_size, num_pages, has_kv, vec, v_eps, v_first, v_first_ld, v_lam)
+        nh, nkv, dq, dv, dpad, page_size, num_pages, has_kv, vec, v_eps, v_first, v_first_ld, v_lam, \
+        q_head_mult, kv_shared ? nh * dq : nh * dq + nkv * dq, v_scale)
     if (out_type == BW_F32) BW_HN(float);
     else if (out_type == BW_BF16) BW_HN(bf16);
     else return BW_ERR_BAD_ARG;

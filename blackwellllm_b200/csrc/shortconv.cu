@@ -1,0 +1,182 @@
+// What stands between a recurrent mixer's projections and its recurrence:
+//
+//   short_conv   a causal convolution over time per channel with `taps` columns (the last one is the current token's),
+//                an optional bias, silu, and for the channels that ask for it the unit norm of each head:
+//                u / sqrt(sum(u^2) + unit_eps) * scale
+//   step_gates   per head: d = softplus(z + dt_bias), decay = exp(A d) with A = -exp(A_log), and either the step size d
+//                itself or a second gate sigmoid(z2)
+//
+// in one kernel.  The convolution's earlier inputs of a request are part of its state: `state` [slots, taps, channels]
+// float32 holds the input of position p at entry p mod taps.  A token at position p reads the entries of p - 1 ..
+// p - (taps - 1) where they lie before the step's own tokens, so a step of one token per request may write the entry of p
+// at once; a step with longer portions writes the last taps - 1 inputs with a kernel of its own afterwards (another block
+// may still read the entries it replaces).  Positions before the sequence's start count as zeros and are never read.
+// All arithmetic is float32.
+#include "common.cuh"
+
+using bf16 = __nv_bfloat16;
+
+namespace {
+
+constexpr int MAX_SEGS = 3;
+constexpr int CHUNK = 128;      // channels of a warp's piece where a segment has no norm
+
+struct Seg {
+    int c0;            // first channel
+    int pieces;        // warps: heads of a normed segment, stretches of CHUNK channels otherwise
+    int size;          // channels of a piece
+    int channels;      // channels of the segment
+    int unit;          // 1: every piece is a head that becomes a unit vector times scale
+    float scale;
+};
+
+struct ConvParams {
+    const float* x; long long ld;          // the projections' rows; channel c of the convolution is column c
+    const float* w;                        // [taps, C]
+    const float* bias;                     // [C] or null
+    float* state;                          // [slots, taps, C]
+    const int *positions, *req_of_token, *cu_q, *state_slot;
+    float* out;                            // [T, C]
+    int T, C, taps, single;                // single: one token per request, the state is written here
+    int nseg; Seg seg[MAX_SEGS];
+    float unit_eps;
+    // gates: z at column z_off of zx (rows zld apart), z2 at z2_off (< 0: none, the step size is written instead)
+    const float* zx; long long zld; int z_off, z2_off, heads;
+    const float *A, *dt_bias;              // [heads]: -exp(A_log), dt_bias
+    float *decay, *second;                 // [T, heads]
+};
+
+constexpr int TILE = 8;        // tokens of a warp, one after another (their rows overlap in the cache)
+constexpr int WARPS = 8;
+
+__device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
+
+__device__ __forceinline__ float conv_at(const ConvParams& p, int t, int local, int pos, const float* st, int c) {
+    float acc = p.bias ? p.bias[c] : 0.f;
+    for (int j = p.taps - 1; j >= 0; --j) {          // j tokens back, the oldest first
+        if (j > pos) continue;                        // before the sequence's start
+        const float v = j <= local ? p.x[(size_t)(t - j) * p.ld + c] : st[(size_t)((pos - j) % p.taps) * p.C + c];
+        acc = fmaf(p.w[(size_t)(p.taps - 1 - j) * p.C + c], v, acc);
+    }
+    return acc;
+}
+
+template <int NR>   // registers a lane holds of a normed head: heads of up to 32 * NR channels
+__global__ void __launch_bounds__(32 * WARPS)
+short_conv_kernel(ConvParams p) {
+    BW_PDL_TRIGGER();
+    BW_PDL_WAIT();
+    const int lane = threadIdx.x & 31;
+    int item = blockIdx.y * WARPS + (threadIdx.x >> 5);
+    const int tile = p.single ? 1 : TILE;
+    const int t0 = blockIdx.x * tile, t1 = min(p.T, t0 + tile);
+    int s = 0;
+    while (s < p.nseg && item >= p.seg[s].pieces) { item -= p.seg[s].pieces; ++s; }
+    if (s == p.nseg) {
+        // the gates: the pieces behind the last segment, 32 heads each
+        const int h = item * 32 + lane;
+        if (h >= p.heads) return;
+        const float A = p.A[h], b = p.dt_bias[h];
+        for (int t = t0; t < t1; ++t) {
+            const float* z = p.zx + (size_t)t * p.zld;
+            const float d = softplus(z[p.z_off + h] + b);
+            p.decay[(size_t)t * p.heads + h] = expf(A * d);
+            p.second[(size_t)t * p.heads + h] = p.z2_off >= 0 ? 1.f / (1.f + expf(-z[p.z2_off + h])) : d;
+        }
+        return;
+    }
+    const Seg sg = p.seg[s];
+    const int first = sg.c0 + item * sg.size;
+    const int n = min(sg.size, sg.channels - item * sg.size);
+    for (int t = t0; t < t1; ++t) {
+        const int r = p.req_of_token[t], local = t - p.cu_q[r], pos = p.positions[t];
+        float* st = p.state + (size_t)p.state_slot[r] * p.taps * p.C;
+        float* dst = p.out + (size_t)t * p.C;
+        if (sg.unit) {
+            float u[NR];
+            float ss = 0.f;
+#pragma unroll
+            for (int k = 0; k < NR; ++k) {
+                const int c = k * 32 + lane;
+                u[k] = c < n ? silu(conv_at(p, t, local, pos, st, first + c)) : 0.f;
+                ss = fmaf(u[k], u[k], ss);
+            }
+            const float f = sg.scale * rsqrtf(bw::warp_sum(ss) + p.unit_eps);
+#pragma unroll
+            for (int k = 0; k < NR; ++k) {
+                const int c = k * 32 + lane;
+                if (c < n) dst[first + c] = u[k] * f;
+            }
+        } else {
+            for (int c = lane; c < n; c += 32) dst[first + c] = silu(conv_at(p, t, local, pos, st, first + c));
+        }
+        if (p.single) {
+            for (int c = lane; c < n; c += 32)
+                st[(size_t)(pos % p.taps) * p.C + first + c] = p.x[(size_t)t * p.ld + first + c];
+        }
+    }
+}
+
+// the last taps - 1 inputs of every request's portion to its state
+__global__ void __launch_bounds__(256)
+conv_state_kernel(const float* __restrict__ x, long long ld, float* __restrict__ state, const int* __restrict__ cu_q,
+                  const int* __restrict__ positions, const int* __restrict__ state_slot, int C, int taps) {
+    BW_PDL_TRIGGER();
+    BW_PDL_WAIT();
+    const int r = blockIdx.x;
+    const int a = cu_q[r], e = cu_q[r + 1];
+    const int from = max(a, e - (taps - 1));
+    float* st = state + (size_t)state_slot[r] * taps * C;
+    for (int t = from; t < e; ++t)
+        for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x)
+            st[(size_t)(positions[t] % taps) * C + c] = x[(size_t)t * ld + c];
+}
+
+}  // namespace
+
+// x: float32 rows `ld` apart, the convolution's C channels side by side (segments in order: n heads of `size` channels,
+// unit != 0: unit vectors times scale).  w: float32 [taps, C] (oldest tap first).  single: one token per request.  Gates
+// (heads > 0): see ConvParams.  max piece of a unit segment: 256 channels.
+BW_EXPORT int bw_short_conv(const float* x, long long ld, const float* w, const float* bias, float* state,
+                            const int* positions, const int* req_of_token, const int* cu_q, const int* state_slot,
+                            float* out, int T, int R, int C, int taps, int single, int nseg, const int* seg_heads,
+                            const int* seg_size, const int* seg_unit, const float* seg_scale, float unit_eps,
+                            const float* zx, long long zld, int z_off, int z2_off, int heads, const float* A,
+                            const float* dt_bias, float* decay, float* second, void* stream) {
+    if (T <= 0) return 0;
+    if (C <= 0 || taps <= 0 || nseg <= 0 || nseg > MAX_SEGS || R <= 0 || (single && T != R) || ld < C ||
+        (heads > 0 && (!A || !dt_bias || !decay || !second || !zx)))
+        return BW_ERR_BAD_ARG;
+    ConvParams p;
+    p.x = x; p.ld = ld; p.w = w; p.bias = bias; p.state = state; p.positions = positions; p.req_of_token = req_of_token;
+    p.cu_q = cu_q; p.state_slot = state_slot; p.out = out; p.T = T; p.C = C; p.taps = taps; p.single = single;
+    p.nseg = nseg; p.unit_eps = unit_eps;
+    p.zx = zx; p.zld = zld; p.z_off = z_off; p.z2_off = z2_off; p.heads = heads; p.A = A; p.dt_bias = dt_bias;
+    p.decay = decay; p.second = second;
+    int c0 = 0, pieces = 0, widest = 0;
+    for (int s = 0; s < nseg; ++s) {
+        Seg& g = p.seg[s];
+        if (seg_heads[s] <= 0 || seg_size[s] <= 0) return BW_ERR_BAD_ARG;
+        g.c0 = c0; g.channels = seg_heads[s] * seg_size[s]; g.unit = seg_unit[s]; g.scale = seg_scale[s];
+        g.size = g.unit ? seg_size[s] : CHUNK;
+        g.pieces = (g.channels + g.size - 1) / g.size;
+        if (g.unit && g.size > widest) widest = g.size;
+        c0 += g.channels; pieces += g.pieces;
+    }
+    if (c0 != C) return BW_ERR_BAD_ARG;
+    if (widest > 256) return BW_ERR_UNSUPPORTED;
+    pieces += (heads + 31) / 32;
+    const int tile = single ? 1 : TILE;
+    const dim3 grid((T + tile - 1) / tile, (pieces + WARPS - 1) / WARPS);
+    cudaStream_t s = (cudaStream_t)stream;
+    if (widest <= 128) bw::launch((short_conv_kernel<4>), grid, dim3(32 * WARPS), 0, s, p);
+    else bw::launch((short_conv_kernel<8>), grid, dim3(32 * WARPS), 0, s, p);
+    BW_LAUNCH_CHECK();
+    if (!single && taps > 1) {
+        const int blocks = (C + 255) / 256;
+        bw::launch((conv_state_kernel), dim3(R, blocks < 32 ? blocks : 32), dim3(256), 0, s, x, ld, state, cu_q, positions, state_slot, C, taps);
+        BW_LAUNCH_CHECK();
+    }
+    return 0;
+}

@@ -247,6 +247,12 @@ def gemm_tc_planes(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor
     return buf[:n.value * M * N].view(n.value, M, N)
 
 
+def planes_fit_behind(first: torch.Tensor) -> bool:
+    """Whether another product's planes may go behind ``first`` in this module's buffer (``gemm_tc_planes(..., after=)``)."""
+    return (first.numel() % 64 == 0 and first.numel() * 4 <= PLANE_BUFFER_ELEMS
+            and first.data_ptr() == _plane_buffer(first.device).data_ptr())
+
+
 def planes_generation() -> int:
     """A number that changes with every product that leaves planes in this module's buffer."""
     return _plane_generation
@@ -260,8 +266,7 @@ def gemm_tc_deferred(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tens
     if out.dtype != torch.float32 or not out.is_contiguous() or out.shape != (x.shape[0], w.shape[0]):
         raise KernelError("gemm_tc_deferred: out must be contiguous float32 [M, N]")
     if (_pending is not None and not overwrite and _pending[0].data_ptr() == out.data_ptr() and _pending[0].shape == out.shape
-            and _pending[1].numel() % 64 == 0 and _pending[1].numel() * 4 <= PLANE_BUFFER_ELEMS
-            and _pending[1].data_ptr() == _plane_buffer(x.device).data_ptr()):
+            and planes_fit_behind(_pending[1])):
         # a second sum into the same tensor (a block whose two sublayers both add to the stream): its planes go
         # behind the first's, and the reader adds them all in one pass, in plane order
         target, first, ow = _pending
@@ -328,9 +333,9 @@ def swiglu(gu: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.T
     return out
 
 
-ACT_SILU, ACT_CLAMPED_SWISH, ACT_RELU2, ACT_GELU_TANH = 0, 1, 2, 3   # the activation codes of csrc/common.cuh
+ACT_SILU, ACT_CLAMPED_SWISH, ACT_RELU2, ACT_GELU_TANH, ACT_GELU = 0, 1, 2, 3, 4   # the activation codes of csrc/common.cuh
 GATED_ACTIVATIONS = {"silu": ACT_SILU, "clamped_swish": ACT_CLAMPED_SWISH, "gelu_tanh": ACT_GELU_TANH}
-UNARY_ACTIVATIONS = {"relu2": ACT_RELU2}
+UNARY_ACTIVATIONS = {"relu2": ACT_RELU2, "gelu": ACT_GELU}
 GEMM_TC_GATED_ACTIVATIONS = (ACT_SILU, ACT_CLAMPED_SWISH, ACT_GELU_TANH)   # what gemm_tc's fused gate/up epilogue computes
 GEMM_TC_GATED_BIAS = True                                   # ... and whether it takes biases on gate and up (interleaved like the rows)
 
@@ -350,7 +355,7 @@ def glu(gu: torch.Tensor, act: int, limit: float = 0.0, alpha: float = 1.0, out_
 
 
 def unary_act(x: torch.Tensor, act: int, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-    """Element by element: ACT_RELU2 ``max(x, 0) ** 2`` (float32 arithmetic)."""
+    """Element by element (float32 arithmetic): ACT_RELU2 ``max(x, 0) ** 2``; ACT_GELU ``0.5 x (1 + erf(x / sqrt(2)))``."""
     _dev(x, "x")
     out = torch.empty(x.shape, dtype=out_dtype or x.dtype, device=x.device)
     fn = _fn("elementwise", "bw_unary_act", [c_void_p, c_int, c_void_p, c_int, c_ll, c_int, c_void_p])
@@ -701,7 +706,8 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = Non
     bfloat16 [M, N / 2] = silu(gate) * up, computed in the epilogue; ``act`` = ACT_CLAMPED_SWISH (with its
     ``limit`` and ``alpha``) or ACT_GELU_TANH puts that gated activation in its place (:func:`glu`); a ``bias`` (interleaved
     like the rows) is added to gate and up before it.  Without ``swiglu``,
-    ``act`` = ACT_RELU2 squares the positive part of every sum of a result that is written (not added)."""
+    ``act`` = ACT_RELU2 (the squared positive part) or ACT_GELU (gelu with the error function, to about 1e-7) is applied to
+    every sum of a result that is written (not added)."""
     _dev(x, "x", torch.bfloat16, contiguous=False); _dev(w, "w", torch.bfloat16)
     if not gemm_tc_supports(x, w):
         raise KernelError("gemm_tc: operands must be bfloat16 with K and the row stride multiples of 8 "
@@ -1236,7 +1242,8 @@ def head_norm_rope_append(qkv: torch.Tensor, batch, block_table: torch.Tensor, t
                           k_gain: Optional[torch.Tensor], eps: float, k_pages: torch.Tensor, v_pages: torch.Tensor,
                           nh: int, nkv: int, dq: int, dv: int, has_kv: bool = True, append: bool = True,
                           q_temp: Optional[tuple] = None, v_eps: float = 0.0,
-                          v_mix: Optional[tuple] = None) -> torch.Tensor:
+                          v_mix: Optional[tuple] = None, q_head_mult: Optional[torch.Tensor] = None,
+                          kv_shared: bool = False, v_scale: float = 1.0) -> torch.Tensor:
     """:func:`qk_norm_rope_append` with the norm taken per head: every query head is divided by its own root mean
     square and multiplied by ``q_gain`` (float32 [dq], shared by the heads; ``k_gain`` for the key heads).
     ``qkv`` float32 [T, >= nh*dq (+ nkv*dq + nkv*dv with ``has_kv``)]: further columns (a gate's projection) are
@@ -1244,8 +1251,19 @@ def head_norm_rope_append(qkv: torch.Tensor, batch, block_table: torch.Tensor, t
     multiplied by ``1 + coef * log(1 + n)``, n the whole periods of ``every`` positions in p + 1.  Without ``has_kv`` (a run that reads another
     run's keys and values) nothing is appended.  ``v_eps`` > 0: every value head is divided by
     sqrt(mean(v^2) + v_eps) on its way into the cache.  ``v_mix`` = (v_first float32 [T, nkv * dv], possibly a column
-    range of a wider tensor; lam, a float32 number on the device): the values are cached as (1 - lam) v + lam v_first."""
-    _dev(qkv, "qkv", torch.float32); _dev(block_table, "block_table", torch.int32)
+    range of a wider tensor; lam, a float32 number on the device): the values are cached as (1 - lam) v + lam v_first.
+    ``q_head_mult`` (float32 [nh]): every query head is multiplied by its own number.  ``kv_shared``: the rows hold no values,
+    the key projection before norm and rotation is cached as the values (dv == dq).  ``v_scale``: a factor on the values as
+    they are cached.  qkv may be a range of columns of a wider tensor."""
+    _dev(qkv, "qkv", torch.float32, contiguous=False); _dev(block_table, "block_table", torch.int32)
+    if qkv.dim() != 2 or qkv.stride(1) != 1:
+        raise KernelError("head_norm_rope_append: qkv must be [T, columns] with contiguous rows")
+    if q_head_mult is not None:
+        _dev(q_head_mult, "q_head_mult", torch.float32)
+        if q_head_mult.numel() != nh:
+            raise KernelError("head_norm_rope_append: q_head_mult must have one entry per query head")
+    if kv_shared and (dv != dq or not has_kv or v_mix is not None):
+        raise KernelError("head_norm_rope_append: values that are the keys have the keys' head size and are not mixed")
     vf = lam = None
     if v_mix is not None:
         vf, lam = v_mix
@@ -1255,7 +1273,7 @@ def head_norm_rope_append(qkv: torch.Tensor, batch, block_table: torch.Tensor, t
     _dev(k_pages, "k_pages"); _dev(v_pages, "v_pages", k_pages.dtype)
     T = qkv.shape[0]
     num_pages, pk, page_size, dpad = k_pages.shape
-    need = nh * dq + (nkv * (dq + dv) if has_kv else 0)
+    need = nh * dq + (nkv * (dq if kv_shared else dq + dv) if has_kv else 0)
     if qkv.shape[1] < need or pk != nkv or v_pages.shape != k_pages.shape:
         raise KernelError("head_norm_rope_append: qkv must be [T, >= nh*dq (+ nkv*dq + nkv*dv)], pages [num_pages, nkv, page, dpad]")
     for name, g in (("q_gain", q_gain), ("k_gain", k_gain)):
@@ -1271,12 +1289,12 @@ def head_norm_rope_append(qkv: torch.Tensor, batch, block_table: torch.Tensor, t
     q_out = torch.empty((T, nh * dpad), dtype=k_pages.dtype, device=qkv.device)
     fn = _fn("qk_norm_rope", "bw_head_norm_rope_append",
              [c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_float,
-              c_float, c_void_p, c_void_p, c_void_p] + [c_int] * 10 + [c_float, c_void_p, c_ll, c_void_p, c_void_p])
+              c_float, c_void_p, c_void_p, c_void_p] + [c_int] * 10 + [c_float, c_void_p, c_ll, c_void_p, c_void_p, c_int, c_float, c_void_p])
     _check(fn(_ptr(qkv), qkv.stride(0), _ptr(batch.positions), _ptr(batch.req_of_token), _ptr(block_table),
               block_table.shape[1], _ptr(table), int(rotary_dim), int(interleaved), _ptr(q_gain), _ptr(k_gain), float(eps),
               coef, every, _ptr(q_out), _ptr(k_pages), _ptr(v_pages), _code(k_pages, "pages"), T, nh, nkv, dq, dv, dpad,
               page_size, num_pages if (append and has_kv) else 0, int(has_kv), float(v_eps or 0.0), _ptr(vf),
-              vf.stride(0) if vf is not None else 0, _ptr(lam), _stream()),
+              vf.stride(0) if vf is not None else 0, _ptr(lam), _ptr(q_head_mult), int(kv_shared), float(v_scale), _stream()),
            "head_norm_rope_append")
     return q_out
 
@@ -1469,7 +1487,7 @@ def gla_decay(proj: torch.Tensor, x_off: int, w: torch.Tensor, b: torch.Tensor, 
 
 def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torch.Tensor, batch, state: torch.Tensor,
              heads: int, dk: int, dv: int, q_scale: float, k_scale: Optional[torch.Tensor] = None,
-             scalar_decay: bool = False, ones_col: bool = False) -> torch.Tensor:
+             scalar_decay: bool = False, ones_col: bool = False, qk_rep: int = 1) -> torch.Tensor:
     """The recurrence ``S <- diag(a) S + k v^T, o = S^T (q_scale q)`` over the step's tokens, request by request
     in order, from and into ``state`` [slots, heads, dk, dv] (float32) at the requests' slots.  ``proj`` float32
     [T, ld] holds q, k, v at the given column offsets (head-major); ``decay`` float32 [T, heads * dk] holds a
@@ -1477,7 +1495,8 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torc
     ``scalar_decay``: ``decay`` is [T, heads]; ``k_scale`` float32 [T, heads]: the keys are multiplied by it as they are
     read; ``ones_col``: ``dv`` counts one more value column than ``proj`` holds, the constant 1, so that the state's
     last column is n <- a n + k and the output's last column n . q.  The state's rows may be longer than ``dv`` (padding that
-    stays zero): with a length that is a multiple of 4 the kernel moves a lane's columns of a row in one access."""
+    stays zero): with a length that is a multiple of 4 the kernel moves a lane's columns of a row in one access.
+    ``qk_rep``: ``proj`` holds ``heads / qk_rep`` query and key heads, head h uses number h / qk_rep (``scalar_decay`` only)."""
     _dev(proj, "proj", torch.float32); _dev(decay, "decay", torch.float32); _dev(state, "state", torch.float32)
     T = proj.shape[0]
     if dk > GLA_MAX_KEY_DIM:
@@ -1489,23 +1508,26 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torc
         _dev(k_scale, "k_scale", torch.float32)
         if k_scale.shape != (T, heads):
             raise KernelError("gla_scan: k_scale must be [T, heads]")
-    if max(q_off + heads * dk, k_off + heads * dk, v_off + heads * (dv - int(ones_col))) > proj.shape[1]:
+    if qk_rep < 1 or heads % qk_rep or (qk_rep > 1 and not scalar_decay):
+        raise KernelError("gla_scan: shared query/key heads go with one decay per head, heads a multiple of qk_rep")
+    hk = heads // qk_rep
+    if max(q_off + hk * dk, k_off + hk * dk, v_off + heads * (dv - int(ones_col))) > proj.shape[1]:
         raise KernelError("gla_scan: q, k or v lie outside the projection's columns")
     o = torch.empty((T, heads * dv), dtype=torch.float32, device=proj.device)
     fn = _fn("gla", "bw_gla_scan", [c_void_p, c_ll, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                    c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p])
+                                    c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
     _check(fn(_ptr(proj), proj.stride(0), q_off, k_off, v_off, _ptr(decay), _ptr(batch.cu_q), _ptr(batch.state_slot),
               _ptr(state), _ptr(o), batch.R, heads, dk, dv, float(q_scale), _ptr(k_scale), int(scalar_decay),
-              int(ones_col), int(state.shape[3]), _stream()), "gla_scan")
+              int(ones_col), int(state.shape[3]), int(qk_rep), _stream()), "gla_scan")
     return o
 
 
 def gla_gate(o: torch.Tensor, proj: torch.Tensor, g_off: int, gain: torch.Tensor, heads: int, dv: int, eps: float,
              out_dtype: torch.dtype) -> torch.Tensor:
     """Per token and head ``o / rms(o) * gain * silu(g)`` with g at column ``g_off`` of ``proj``."""
-    _dev(o, "o", torch.float32); _dev(proj, "proj", torch.float32); _dev(gain, "gain", torch.float32)
+    _dev(o, "o", torch.float32); _dev(proj, "proj", torch.float32, contiguous=False); _dev(gain, "gain", torch.float32)
     T = o.shape[0]
-    if o.shape[1] != heads * dv or gain.numel() != dv or g_off + heads * dv > proj.shape[1]:
+    if o.shape[1] != heads * dv or gain.numel() != dv or proj.stride(1) != 1 or g_off + heads * dv > proj.shape[1]:
         raise KernelError("gla_gate: o must be [T, heads * dv], the gain [dv], the gate inside the projection")
     out = torch.empty((T, heads * dv), dtype=out_dtype, device=o.device)
     fn = _fn("gla", "bw_gla_gate", [c_void_p, c_void_p, c_ll, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
@@ -1551,6 +1573,177 @@ def mlstm_out(o: torch.Tensor, e: torch.Tensor, proj: torch.Tensor, g_off: int, 
                                        c_float, c_float, c_void_p])
     _check(fn(_ptr(o), _ptr(e), _ptr(proj), proj.stride(0), int(g_off), _ptr(gain), _ptr(out), _code(out, "out"), T, heads, dv,
               float(eps), float(den_eps), _stream()), "mlstm_out")
+    return out
+
+
+# ------------------------------------------------------------------ short convolution, gated delta rule, state space
+
+def short_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor, batch, segments,
+               unit_eps: float = 0.0, gates: Optional[tuple] = None):
+    """A causal convolution over time per channel, then silu, of the step's tokens: ``x`` float32 [T, >= C] (a range of
+    columns of the projections), ``w`` float32 [taps, C] (the last row is the current token's), ``bias`` [C] or None;
+    ``state`` float32 [slots, taps, C]: the earlier inputs of the requests, position p at entry p mod taps; it takes the
+    step's last inputs.  ``segments``: (heads, size, scale) per stretch of channels; a stretch with a scale that is not None
+    has every head divided by sqrt(sum + ``unit_eps``) and multiplied by the scale.  ``gates`` = (z, column, column of the
+    second gate or None, A [heads], dt_bias [heads]): in the same kernel decay = exp(A d), d = softplus(z + dt_bias).
+    Returns (float32 [T, C], decay, second) where second is sigmoid of the second gate, or d without one."""
+    _dev(x, "x", torch.float32, contiguous=False); _dev(w, "w", torch.float32); _dev(state, "state", torch.float32)
+    T = x.shape[0]
+    taps, C = w.shape
+    if x.dim() != 2 or x.stride(1) != 1 or x.shape[1] < C or T != batch.T or state.dim() != 3 or tuple(state.shape[1:]) != (taps, C):
+        raise KernelError("short_conv: x [T, >= C] with contiguous rows, w [taps, C], state [slots, taps, C]")
+    if bias is not None:
+        _dev(bias, "bias", torch.float32)
+        if bias.numel() != C:
+            raise KernelError("short_conv: the bias must have one entry per channel")
+    if not 1 <= len(segments) <= 3 or sum(n * size for n, size, _ in segments) != C:
+        raise KernelError("short_conv: one to three segments that cover the channels")
+    out = torch.empty((T, C), dtype=torch.float32, device=x.device)
+    z = A = dtb = decay = second = None
+    z_off, z2_off, heads = 0, -1, 0
+    if gates is not None:
+        z, z_off, z2, A, dtb = gates
+        _dev(z, "z", torch.float32, contiguous=False); _dev(A, "A", torch.float32); _dev(dtb, "dt_bias", torch.float32)
+        heads = A.numel()
+        z2_off = -1 if z2 is None else int(z2)
+        if dtb.numel() != heads or z.shape[0] != T or z.stride(1) != 1 or max(z_off, z2_off) + heads > z.shape[1]:
+            raise KernelError("short_conv: the gates' columns lie outside the projections")
+        decay = torch.empty((T, heads), dtype=torch.float32, device=x.device)
+        second = torch.empty((T, heads), dtype=torch.float32, device=x.device)
+    n = len(segments)
+    heads_c, size_c = (c_int * n)(*[s[0] for s in segments]), (c_int * n)(*[s[1] for s in segments])
+    unit_c = (c_int * n)(*[int(s[2] is not None) for s in segments])
+    scale_c = (c_float * n)(*[float(s[2] or 0.0) for s in segments])
+    fn = _fn("shortconv", "bw_short_conv", [c_void_p, c_ll] + [c_void_p] * 8 + [c_int] * 6 + [c_void_p] * 4 + [c_float, c_void_p, c_ll] +
+             [c_int] * 3 + [c_void_p] * 5)
+    _check(fn(_ptr(x), x.stride(0), _ptr(w), _ptr(bias), _ptr(state), _ptr(batch.positions), _ptr(batch.req_of_token),
+              _ptr(batch.cu_q), _ptr(batch.state_slot), _ptr(out), T, batch.R, C, taps, int(T == batch.R), n, heads_c, size_c,
+              unit_c, scale_c, float(unit_eps), _ptr(z), 0 if z is None else z.stride(0), int(z_off), z2_off, heads, _ptr(A),
+              _ptr(dtb), _ptr(decay), _ptr(second), _stream()), "short_conv")
+    return out, decay, second
+
+
+DELTA_MAX_KEY_DIM = 256
+
+
+def delta_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torch.Tensor, beta: torch.Tensor, batch,
+               state: torch.Tensor, heads: int, qk_rep: int, dk: int, dv: int) -> torch.Tensor:
+    """The gated delta rule ``S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q`` over the step's tokens, request by
+    request in order, from and into ``state`` [slots, heads, dk, dv] (float32).  ``qkv`` float32 [T, ld] holds q and k
+    (``heads / qk_rep`` heads) and v (``heads`` heads) at the given columns; ``decay`` (g), ``beta`` float32 [T, heads].
+    Returns o float32 [T, heads * dv]."""
+    _dev(qkv, "qkv", torch.float32); _dev(decay, "decay", torch.float32); _dev(beta, "beta", torch.float32)
+    _dev(state, "state", torch.float32)
+    T = qkv.shape[0]
+    if dk > DELTA_MAX_KEY_DIM:
+        raise KernelError(f"delta_scan: key size {dk} exceeds {DELTA_MAX_KEY_DIM}")
+    if (qk_rep < 1 or heads % qk_rep or decay.shape != (T, heads) or beta.shape != (T, heads) or state.dim() != 4
+            or tuple(state.shape[1:]) != (heads, dk, dv)):
+        raise KernelError("delta_scan: decay and beta [T, heads], state [slots, heads, dk, dv], heads a multiple of qk_rep")
+    hk = heads // qk_rep
+    if max(q_off + hk * dk, k_off + hk * dk, v_off + heads * dv) > qkv.shape[1]:
+        raise KernelError("delta_scan: q, k or v lie outside the rows")
+    o = torch.empty((T, heads * dv), dtype=torch.float32, device=qkv.device)
+    fn = _fn("delta", "bw_delta_scan", [c_void_p, c_ll, c_int, c_int, c_int] + [c_void_p] * 6 + [c_int] * 5 + [c_void_p])
+    _check(fn(_ptr(qkv), qkv.stride(0), int(q_off), int(k_off), int(v_off), _ptr(decay), _ptr(beta), _ptr(batch.cu_q),
+              _ptr(batch.state_slot), _ptr(state), _ptr(o), batch.R, heads, int(qk_rep), dk, dv, _stream()), "delta_scan")
+    return o
+
+
+def ssd_out(y: torch.Tensor, x: torch.Tensor, z: torch.Tensor, D: torch.Tensor, gain: torch.Tensor, vdim: int, parts: int,
+            eps: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """``u = (y + D x) * silu(z)`` per channel (D one number per head of ``vdim`` channels), then ``u / rms(u) * gain`` with
+    the root mean square taken over each of ``parts`` equal parts.  y float32 [T, inner]; x, z float32 [T, >= inner]
+    (possibly ranges of columns); D [inner / vdim], gain [inner]."""
+    _dev(y, "y", torch.float32); _dev(x, "x", torch.float32, contiguous=False); _dev(z, "z", torch.float32, contiguous=False)
+    _dev(D, "D", torch.float32); _dev(gain, "gain", torch.float32)
+    T, inner = y.shape
+    if (x.shape[0] != T or z.shape[0] != T or min(x.shape[1], z.shape[1]) < inner or x.stride(1) != 1 or z.stride(1) != 1
+            or D.numel() * vdim != inner or gain.numel() != inner or parts < 1 or inner % parts):
+        raise KernelError("ssd_out: y [T, inner], x and z [T, >= inner], D [inner / vdim], gain [inner], inner a multiple of parts")
+    out = torch.empty((T, inner), dtype=out_dtype, device=y.device)
+    fn = _fn("ssd", "bw_ssd_out", [c_void_p, c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_void_p, c_void_p] + [c_int] * 5 +
+             [c_float, c_void_p])
+    _check(fn(_ptr(y), _ptr(x), x.stride(0), _ptr(z), z.stride(0), _ptr(D), _ptr(gain), _ptr(out), _code(out, "out"), T, inner,
+              int(vdim), int(parts), float(eps), _stream()), "ssd_out")
+    return out
+
+
+# ------------------------------------------------------------------ the seam between two sublayers
+
+NORM_NONE, NORM_RMS, NORM_LAYER = 0, 1, 2    # what a norm does to a row (csrc/rownorm.cu)
+
+
+class NormedPair:
+    """A sublayer's output that is the mean of two rows, each RMS-normed with a gain: ``0.5 (rms(y) gy + rms(z) gz)``.
+    ``y`` / ``z``: float32 [T, H], or planes [S, T, H] from :func:`gemm_tc_planes` (good until this module's plane buffer
+    is written again, which ``generation`` watches)."""
+
+    def __init__(self, y: torch.Tensor, gy: torch.Tensor, z: torch.Tensor, gz: torch.Tensor, eps: float):
+        self.y, self.gy, self.z, self.gz, self.eps = y, gy, z, gz, float(eps)
+        self.generation = _plane_generation
+
+
+def _row_source(t: torch.Tensor, T: int, H: int, name: str):
+    """(base, planes, stride, number of planes) of a row source; takes over a sum that is outstanding for it."""
+    global _pending
+    if t.dim() == 3:
+        if tuple(t.shape[1:]) != (T, H) or t.dtype != torch.float32:
+            raise KernelError(f"row_step: {name} planes must be float32 [S, T, H]")
+        return None, t, t.stride(0), t.shape[0]
+    if _pending is not None and _pending[0].data_ptr() == t.data_ptr() and _pending[0].shape == t.shape:
+        (_, planes, overwrite), _pending = _pending, None
+        return (None if overwrite else t), planes, planes.stride(0), planes.shape[0]
+    _dev(t, name, torch.float32)
+    if tuple(t.shape) != (T, H):
+        raise KernelError(f"row_step: {name} must be float32 [T, H]")
+    return t, None, 0, 0
+
+
+def row_step(stream: torch.Tensor, branch=None, post: Optional[tuple] = None, then: Optional[tuple] = None,
+             rows: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
+    """One pass over the stream (float32 [T, H]): ``stream += post(branch)`` and then ``then(stream)``, the next sublayer's
+    input, which is returned.  ``branch``: a float32 tensor [T, H] (a sum that is outstanding for it is added while it is
+    read) or a :class:`NormedPair`; None: nothing is added.  ``post``, ``then`` = (kind, gain, eps): kind NORM_NONE, NORM_RMS
+    or NORM_LAYER, gain float32 [H] or None; without ``then`` nothing is returned.  ``rows`` (int32): only these rows are
+    made, and the stream is left as it is (the model's last norm on the rows whose logits are wanted)."""
+    T, H = stream.shape
+    y = z = (None, None, 0, 0)
+    gy = gz = None
+    pair_eps = 0.0
+    pair = isinstance(branch, NormedPair)
+    if pair:
+        if branch.y.dim() == 3 or branch.z.dim() == 3:
+            if branch.generation != _plane_generation:
+                raise KernelError("row_step: the pair's planes were overwritten by a later product")
+        z = _row_source(branch.z, T, H, "z")
+        y = _row_source(branch.y, T, H, "y")
+        gy, gz, pair_eps = branch.gy, branch.gz, branch.eps
+        for g in (gy, gz):
+            _dev(g, "gain", torch.float32)
+            if g.numel() != H:
+                raise KernelError("row_step: a gain must have the stream's width")
+    elif branch is not None:
+        y = _row_source(branch, T, H, "branch")
+    _dev(stream, "stream", torch.float32)
+    p_kind, p_gain, p_eps = post if post is not None else (NORM_NONE, None, 0.0)
+    n_kind, n_gain, n_eps = then if then is not None else (NORM_NONE, None, 0.0)
+    for g in (p_gain, n_gain):
+        if g is not None:
+            _dev(g, "gain", torch.float32)
+            if g.numel() != H:
+                raise KernelError("row_step: a gain must have the stream's width")
+    n = T
+    if rows is not None:
+        _dev(rows, "rows", torch.int32)
+        n = rows.numel()
+    out = torch.empty((n, H), dtype=out_dtype or torch.float32, device=stream.device) if then is not None else None
+    fn = _fn("rownorm", "bw_row_step", [c_void_p, c_int, c_void_p, c_void_p, c_ll, c_int, c_int, c_void_p, c_void_p, c_ll, c_int,
+                                        c_void_p, c_void_p, c_float, c_int, c_void_p, c_float, c_int, c_void_p, c_float,
+                                        c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+    _check(fn(_ptr(stream), int(branch is not None), _ptr(y[0]), _ptr(y[1]), y[2], y[3], int(pair), _ptr(z[0]), _ptr(z[1]), z[2],
+              z[3], _ptr(gy), _ptr(gz), pair_eps, int(p_kind), _ptr(p_gain), float(p_eps), int(n_kind), _ptr(n_gain), float(n_eps),
+              _ptr(rows), _ptr(out), _code(out, "out") if out is not None else F32, n, H, _stream()), "row_step")
     return out
 
 

@@ -23,7 +23,7 @@ import torch
 from ..config.specs import ModelConfig
 from ..kernels import ops
 from ..parts import BuildContext, FixedStateRequest, ParamSpec, build_block, build_norm
-from ..parts.block import flush_hyper_write, flush_scaled_sum
+from ..parts.block import flush_hyper_write, flush_open_sums
 from ..parts.linear import Linear
 
 
@@ -152,8 +152,8 @@ class DecoderModel:
             blk = self.blocks[e.layer]
             if not blk.takes_pending or e.add_embedding or e.pass_input is not None:
                 ops.resolve_pending()   # the block before may have left its last sum to the next reader
-            if not getattr(blk, "takes_scaled_sum", False) or e.add_embedding or e.pass_input is not None:
-                flush_scaled_sum(h, batch)   # sublayer outputs that a block left to the stream's next reader
+            # sublayer outputs that the block before left to the stream's next reader
+            flush_open_sums(h, batch, () if e.add_embedding or e.pass_input is not None else getattr(blk, "takes_open", ()))
             if e.add_embedding:
                 ops.add_into(h, h0)
             if e.pass_input is not None:
@@ -161,8 +161,8 @@ class DecoderModel:
                 self.pass_in[e.pass_input](ops.concat2_cast(h, h0, self.ctx.dtype), out=h)
             blk.forward(h, batch, cache, owns_cache=e.cache_of is None)
             if self.stream_hook is not None:
+                flush_open_sums(h, batch)
                 ops.resolve_pending()
-                flush_scaled_sum(h, batch)
                 if S is not None:   # the hook sees the sum of the copies
                     flush_hyper_write(h, batch, S)
                     self.stream_hook(pos, ops.hc_step(h, S, in_w=self._ones))
@@ -173,6 +173,7 @@ class DecoderModel:
             ops.discard_pending(h)
             batch.extras.pop("hc_write", None)
             batch.extras.pop("scaled_sum", None)
+            batch.extras.pop("post_sum", None)
             return torch.empty((0, self.config.vocab_size), dtype=torch.float32, device=h.device)
         if S is not None:
             # the last block's write, the sum of the copies and the model's norm, on the wanted rows only
@@ -184,10 +185,12 @@ class DecoderModel:
             ops.resolve_pending()
             x, _ = ops.scale_add_norm2(h, batch.extras.pop("scaled_sum"), self.final_norm.weight, self.final_norm.eps, None, 0.0,
                                        self.ctx.dtype, rows=batch.logit_rows)
+        elif "post_sum" in batch.extras and hasattr(self.final_norm, "row_norm"):
+            # the last block's open seam and the model's norm, on the wanted rows only
+            branch, post = batch.extras.pop("post_sum")
+            x = ops.row_step(h, branch, post, then=self.final_norm.row_norm(), rows=batch.logit_rows, out_dtype=self.ctx.dtype)
         else:
-            if "scaled_sum" in batch.extras:
-                ops.resolve_pending()
-                flush_scaled_sum(h, batch)
+            flush_open_sums(h, batch)
             if not self.final_norm.adds_pending:
                 ops.resolve_pending()
             x = self.final_norm.forward(h, rows=batch.logit_rows)

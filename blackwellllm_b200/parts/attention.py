@@ -40,6 +40,12 @@ what the kernels read), ``fixed_sink`` (a sink whose score is a constant of the 
 denominator as a learned sink) and ``value_mix`` (the values of every layer that has it, but the first such layer of
 the model, are cached as (1 - lam) v + lam v_first, v_first the first such layer's values of the same token: that
 layer leaves its values of the step in ``batch.extras``, the others read them in the kernel that appends).
+
+And: ``qk_norm = "unit"`` (queries and keys divided by their root mean square after the rotation, without gains: a rotation
+keeps a head's sum of squares, so the kernel divides before it rotates, which is the same number), ``values_from_keys`` (no
+value projection: the key projection is cached twice, normed and rotated as the key, as it is as the value),
+``head_temperature`` (a learned number per query head on its scores: the queries are multiplied by it) and
+``output_scale`` (a constant on the mixer's output: the values are multiplied by it in float32 before they are cached).
 """
 from __future__ import annotations
 
@@ -55,7 +61,7 @@ from .linear import Linear
 _DEFAULT_NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
                   "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias",
                   "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sink": "sinks", "g": "g_proj.weight",
-                  "r1": "r1", "r2": "r2", "rel": "rel", "vmix": "vmix"}
+                  "r1": "r1", "r2": "r2", "rel": "rel", "vmix": "vmix", "temp": "temp"}
 
 
 class GQAAttention(Mixer):
@@ -69,9 +75,15 @@ class GQAAttention(Mixer):
         self.chunk = getattr(spec, "chunk", None)
         self.dv = int(getattr(spec, "v_head_dim", None) or self.hd)
         self.qk_norm_eps = getattr(spec, "qk_norm_eps", None)
-        self.norm_per_head = getattr(spec, "qk_norm", "whole") == "head"
-        if getattr(spec, "qk_norm", "whole") not in ("whole", "head"):
-            raise ValueError(f"qk_norm must be 'whole' or 'head', got {spec.qk_norm!r}")
+        self.unit_norm = getattr(spec, "qk_norm", "whole") == "unit"
+        self.norm_per_head = self.unit_norm or getattr(spec, "qk_norm", "whole") == "head"
+        if getattr(spec, "qk_norm", "whole") not in ("whole", "head", "unit"):
+            raise ValueError(f"qk_norm must be 'whole', 'head' or 'unit', got {spec.qk_norm!r}")
+        if self.unit_norm and self.qk_norm_eps is None:
+            raise ValueError("qk_norm 'unit' needs qk_norm_eps")
+        self.values_from_keys = bool(getattr(spec, "values_from_keys", False))
+        self.head_temperature = bool(getattr(spec, "head_temperature", False))
+        self.output_scale = float(getattr(spec, "output_scale", 1.0))
         qt = getattr(spec, "q_temperature", None)
         self.q_temp = (float(qt[0]), float(qt[1])) if qt is not None and float(qt[0]) != 0.0 else None
         if self.q_temp is not None and not self.q_temp[1] > 0:
@@ -108,6 +120,11 @@ class GQAAttention(Mixer):
             raise ValueError("a soft cap or a table of biases by distance does not go with the logarithmic distance bias")
         if self.value_mix is not None and self.shares_kv:
             raise ValueError("a mixer that shares another run's keys and values mixes no values")
+        if self.values_from_keys and (self.shares_kv or self.value_mix is not None or self.qkv_bias or self.dv != self.hd):
+            raise ValueError("values that are the keys: own keys, no biases, no value mixing, and the value size is head_dim")
+        if self.output_scale != 1.0 and self.shares_kv:
+            raise ValueError("output_scale scales the values as they are cached: not for a mixer that reads another run's")
+        self.temp = None
         self.names = dict(_DEFAULT_NAMES)
         self._given_names = dict(getattr(spec, "names", ()) or ())
         self.names.update(self._given_names)
@@ -116,11 +133,13 @@ class GQAAttention(Mixer):
         self.dpad = -(-max(self.hd, self.dv) // step) * step
         self.general = (self.qk_norm_eps is not None or self.dv != self.hd or self.dpad != self.hd or self.norm_per_head
                         or self.q_temp is not None or self.gated or self.shares_kv or self.v_eps is not None
-                        or self.value_mix is not None)
+                        or self.value_mix is not None or self.values_from_keys or self.head_temperature
+                        or self.output_scale != 1.0)
         # the kernel that norms per head also takes rows with a gate's columns behind q, k, v, or without k and v,
         # and norms the values
         self.per_head_route = (self.norm_per_head or self.q_temp is not None or self.shares_kv
-                               or self.v_eps is not None or self.gate_per_head or self.value_mix is not None)
+                               or self.v_eps is not None or self.gate_per_head or self.value_mix is not None
+                               or self.values_from_keys or self.head_temperature or self.output_scale != 1.0)
         if self.shares_kv and self.qkv_bias:
             raise ValueError("a mixer that shares another run's keys and values has no key and value biases")
         if self.per_head_route and self.qk_norm_eps is not None and not self.norm_per_head:
@@ -131,6 +150,8 @@ class GQAAttention(Mixer):
         self.scale = float(spec.softmax_scale) if spec.softmax_scale is not None else self.hd ** -0.5
         self.ctx = ctx
         self.position = build_position(spec.position, self.hd, ctx)
+        if self.unit_norm and getattr(self.position, "magnitude", 1.0) != 1.0:
+            raise ValueError("qk_norm 'unit' stands after a rotation that keeps lengths (no magnitude factor)")
         # (the general route hands ops.paged_attention finished queries: beyond the query heads per kv head that the
         # tensor-core kernels stack, it takes the CUDA-core kernel; the fused route goes to the tensor-core kernels only)
         ops.check_attention_supported(ctx.dtype, self.dpad, 1 if self.general else self.nh // self.nkv)
@@ -147,13 +168,15 @@ class GQAAttention(Mixer):
         n = self.names
         specs = [ParamSpec(n["q"], (q, H))]
         if not self.shares_kv:
-            specs += [ParamSpec(n["k"], (k, H)), ParamSpec(n["v"], (v, H))]
+            specs += [ParamSpec(n["k"], (k, H))] + ([] if self.values_from_keys else [ParamSpec(n["v"], (v, H))])
         specs.append(ParamSpec(n["o"], (H, self.nh * self.dv)))
         if self.qkv_bias:
             specs += [ParamSpec(n["q_bias"], (q,), role="bias", init="bias_normal"),
                       ParamSpec(n["k_bias"], (k,), role="bias", init="bias_normal"),
                       ParamSpec(n["v_bias"], (v,), role="bias", init="bias_normal")]
-        if self.qk_norm_eps is not None:
+        if self.head_temperature:
+            specs.append(ParamSpec(n["temp"], (self.nh,), role="bias", init="ones"))
+        if self.qk_norm_eps is not None and not self.unit_norm:
             specs.append(ParamSpec(n["q_norm"], (self.hd if self.norm_per_head else q,), role="gain", init="ones"))
             if not self.shares_kv:
                 specs.append(ParamSpec(n["k_norm"], (self.hd if self.norm_per_head else k,), role="gain", init="ones"))
@@ -176,7 +199,11 @@ class GQAAttention(Mixer):
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         n = self.names
-        parts = [tensors[n["q"]]] + ([] if self.shares_kv else [tensors[n["k"]], tensors[n["v"]]])
+        parts = [tensors[n["q"]]] + ([] if self.shares_kv else [tensors[n["k"]]])
+        if not self.shares_kv and not self.values_from_keys:
+            parts.append(tensors[n["v"]])
+        if self.head_temperature:
+            self.temp = tensors[n["temp"]].float().contiguous()
         if self.has_sink:
             self.sink = tensors[n["sink"]].float().contiguous()
         elif self.fixed_sink is not None:
@@ -206,7 +233,10 @@ class GQAAttention(Mixer):
             if w.shape[0] > b.numel():    # the gate's rows ride behind q, k, v and have no bias
                 b = torch.cat([b, torch.zeros(w.shape[0] - b.numel(), dtype=dt, device=b.device)])
         wo = tensors[n["o"]]
-        if self.qk_norm_eps is not None:
+        if self.unit_norm:
+            self.q_gain = torch.ones(self.hd, dtype=torch.float32, device=tensors[n["q"]].device)
+            self.k_gain = None if self.shares_kv else self.q_gain
+        elif self.qk_norm_eps is not None:
             self.q_gain = tensors[n["q_norm"]].float().contiguous()
             self.k_gain = None if self.shares_kv else tensors[n["k_norm"]].float().contiguous()
         if self.general:
@@ -220,33 +250,55 @@ class GQAAttention(Mixer):
         self.qkv = Linear(w, b) if self.project is None else None
         self.o = Linear(wo)
 
+    def input_projection(self):
+        """The product of everything this mixer reads of its input (None where it needs more than one)."""
+        return self.qkv if self.per_head_route and self.gate is None and self.qkv is not None and self.qkv.bias is None else None
+
+    def take_projection(self) -> torch.Tensor:
+        """Hands the projection's weight over to a wider product whose rows :meth:`from_projection` then gets."""
+        w, self.qkv = self.qkv.weight, None
+        return w
+
     def forward(self, x, residual, batch, cache, owns_cache: bool = True, accumulate: bool = True) -> None:
         if self.project is not None:
-            q = self.project(x, batch, cache, owns_cache)
+            o = self._attend(self.project(x, batch, cache, owns_cache), None, x, batch, cache)
         else:
-            qkv = self.qkv(x, out_dtype=torch.float32)
-            if self.per_head_route or (self.gated and self.gate is None):
-                v_mix = None
-                if self.value_mix is not None:
-                    # this step's values of the model's first layer that mixes values: it leaves them, the others read them
-                    v_off = (self.nh + self.nkv) * self.hd
-                    mine = qkv[:, v_off:v_off + self.nkv * self.dv]
-                    first = batch.extras.get("value_mix_first")
-                    if first is None:
-                        batch.extras["value_mix_first"] = mine
-                    elif first.shape != mine.shape:
-                        raise ops.KernelError("value mixing: the layers' values differ in size")
-                    else:
-                        v_mix = (first, self.lam)
-                q = self.position.norm_rotate_append(qkv, batch, cache, self.nh, self.nkv, self.hd, self.dv, self.q_gain,
-                                                     self.k_gain, float(self.qk_norm_eps or 0.0), append=owns_cache,
-                                                     per_head=True, q_temp=self.q_temp, has_kv=not self.shares_kv,
-                                                     v_eps=float(self.v_eps or 0.0), v_mix=v_mix)
-            elif self.general:
-                q = self.position.norm_rotate_append(qkv, batch, cache, self.nh, self.nkv, self.hd, self.dv, self.q_gain,
-                                                     self.k_gain, float(self.qk_norm_eps or 0.0), append=owns_cache)
-            else:
-                q = self.position.rotate_append(qkv, batch, cache, self.nh, self.nkv, self.hd, append=owns_cache)
+            o = self.from_projection(self.qkv(x, out_dtype=torch.float32), batch, cache, owns_cache, x)
+        if accumulate:
+            self.o.add_to(o, residual)
+        elif accumulate is None:
+            self.o.write_to(o, residual)
+        else:
+            self.o(o, out=residual)
+
+    def from_projection(self, qkv, batch, cache, owns_cache: bool = True, x=None):
+        """From the projections' float32 rows to the concatenated heads that the output projection reads."""
+        if self.per_head_route or (self.gated and self.gate is None):
+            v_mix = None
+            if self.value_mix is not None:
+                # this step's values of the model's first layer that mixes values: it leaves them, the others read them
+                v_off = (self.nh + self.nkv) * self.hd
+                mine = qkv[:, v_off:v_off + self.nkv * self.dv]
+                first = batch.extras.get("value_mix_first")
+                if first is None:
+                    batch.extras["value_mix_first"] = mine
+                elif first.shape != mine.shape:
+                    raise ops.KernelError("value mixing: the layers' values differ in size")
+                else:
+                    v_mix = (first, self.lam)
+            q = self.position.norm_rotate_append(qkv, batch, cache, self.nh, self.nkv, self.hd, self.dv, self.q_gain,
+                                                 self.k_gain, float(self.qk_norm_eps or 0.0), append=owns_cache,
+                                                 per_head=True, q_temp=self.q_temp, has_kv=not self.shares_kv,
+                                                 v_eps=float(self.v_eps or 0.0), v_mix=v_mix, q_head_mult=self.temp,
+                                                 kv_shared=self.values_from_keys, v_scale=self.output_scale)
+        elif self.general:
+            q = self.position.norm_rotate_append(qkv, batch, cache, self.nh, self.nkv, self.hd, self.dv, self.q_gain,
+                                                 self.k_gain, float(self.qk_norm_eps or 0.0), append=owns_cache)
+        else:
+            q = self.position.rotate_append(qkv, batch, cache, self.nh, self.nkv, self.hd, append=owns_cache)
+        return self._attend(q, qkv, x, batch, cache)
+
+    def _attend(self, q, qkv, x, batch, cache):
         gate = None
         if self.gated:   # the attention kernels multiply by the gate's sigmoid as they write a row
             if self.gate_per_head:
@@ -255,15 +307,9 @@ class GQAAttention(Mixer):
                 g = self.gate(x, out_dtype=torch.float32) if self.gate is not None \
                     else qkv[:, self.g_off:self.g_off + self.nh * self.dv]
                 gate = (g, self.dv)
-        o = ops.paged_attention(q, cache.k_pages, cache.v_pages, batch, batch.block_tables[cache.group],
-                                self.nh, self.window, self.scale, self.chunk, self.sink, gate, self.dist,
-                                self.keep_first if self.window else 0, self.softcap, self.rel)
-        if accumulate:
-            self.o.add_to(o, residual)
-        elif accumulate is None:
-            self.o.write_to(o, residual)
-        else:
-            self.o(o, out=residual)
+        return ops.paged_attention(q, cache.k_pages, cache.v_pages, batch, batch.block_tables[cache.group],
+                                   self.nh, self.window, self.scale, self.chunk, self.sink, gate, self.dist,
+                                   self.keep_first if self.window else 0, self.softcap, self.rel)
 
 
 register_mixer("gqa_attention", GQAAttention)

@@ -116,7 +116,8 @@ class PositionEncoding(Part):
 
     def norm_rotate_append(self, qkv, batch, cache, nh: int, nkv: int, dq: int, dv: int, q_gain, k_gain, eps: float,
                            append: bool = True, per_head: bool = False, q_temp=None, has_kv: bool = True,
-                           v_eps: float = 0.0, v_mix=None) -> torch.Tensor:
+                           v_eps: float = 0.0, v_mix=None, q_head_mult=None, kv_shared: bool = False,
+                           v_scale: float = 1.0) -> torch.Tensor:
         """The general form of :meth:`rotate_append`: qkv [T, nh*dq + nkv*dq + nkv*dv] float32; with gains,
         all query channels of a token (and all its key channels) are RMS-normed together first; the cache's
         head size may exceed dq and dv (the rest is written as zeros).  ``per_head``: every head is normed by
@@ -124,7 +125,9 @@ class PositionEncoding(Part):
         alone; ``q_temp`` (coef, every): the queries are multiplied by 1 + coef log(1 + n), n the whole periods of ``every`` positions in p + 1;
         ``has_kv=False``: qkv holds queries only and nothing is appended; ``v_eps`` > 0: every value head is divided
         by sqrt(mean(v^2) + v_eps) before it is written; ``v_mix`` = (v_first float32 [T, nkv * dv], lam: one float32 number
-        on the device): the values are written as (1 - lam) v + lam v_first (``per_head`` only)."""
+        on the device): the values are written as (1 - lam) v + lam v_first (``per_head`` only).  Also ``per_head`` only: ``q_head_mult`` (float32
+        [nh]) multiplies every query head by its own number; ``kv_shared``: qkv holds no values, the key projection before
+        norm and rotation is written as the values; ``v_scale`` multiplies the values as they are written."""
         raise NotImplementedError
 
     def fuse_projection(self, weight: torch.Tensor, bias: Optional[torch.Tensor], nh: int, nkv: int, hd: int):
@@ -143,6 +146,11 @@ class Mixer(Part):
 
     def forward(self, x, residual, batch, cache, owns_cache: bool = True) -> None:
         raise NotImplementedError
+
+    # A mixer that can stand beside another one on the same input (``parts/side_by_side.py``) also offers
+    #   input_projection()   the Linear that makes everything it reads of its input in one product (None: it has none),
+    #   take_projection()    hands that Linear's weight over: a wider product makes its rows from now on,
+    #   from_projection(proj, batch, cache, owns_cache)   from those rows (float32) to what its output projection ``o`` reads.
 
 
 class FeedForward(Part):

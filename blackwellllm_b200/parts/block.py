@@ -67,7 +67,15 @@ class SandwichBlock(PreNormBlock):
     """A norm before AND after each sublayer: ``x += post(mixer(pre(x)))``, ``x += post(ffn(pre(x)))``.  The
     sublayer writes its output to a float32 buffer of its own (``accumulate=False``); the second norm reads
     it and adds the result to the stream in one kernel.  A feed-forward with ``forward_post`` does the
-    second norm inside its own last kernel."""
+    second norm inside its own last kernel.
+
+    With the layer's ``layer_scale`` (two vectors), a ``residual_mult`` other than 1 or layer norms, the arrangement is
+    ``x += mult * s1 * post(mixer(pre(x)))`` and so on, and the seams between the sublayers are one kernel each
+    (``ops.row_step``): the norm of a sublayer's output with scale and constant in its gain, the sum into the stream, and the
+    norm before the next sublayer.  The seam behind the block's last sublayer is left to whoever reads the stream next
+    (``batch.extras["post_sum"]`` holds the output and its norm until then): the next such block, the model's last norm on
+    the wanted rows, or :func:`flush_open_sums`.  A sublayer's output may come with its last product open, or as a pair of
+    outputs (``forward_open``): the seam's kernel takes either."""
     takes_pending = False
 
     def __init__(self, layer_spec, hidden_size: int, ctx: BuildContext):
@@ -79,6 +87,19 @@ class SandwichBlock(PreNormBlock):
         for norm in (self.mixer_post, self.ffn_post):
             if norm is not None and not hasattr(norm, "add_to"):
                 raise ValueError(f"{type(norm).__name__} cannot follow a sublayer (it has no add_to)")
+        self.hidden_size = hidden_size
+        self.ctx = ctx
+        self.scale_names = getattr(layer_spec, "layer_scale", None)
+        self.mult = float(getattr(layer_spec, "residual_mult", 1.0))
+        from .norm import LayerNorm
+        norms = [n for n in (self.mixer_norm, self.mixer_post, self.ffn_norm, self.ffn_post) if n is not None]
+        self.seams = self.scale_names is not None or self.mult != 1.0 or any(isinstance(n, LayerNorm) for n in norms)
+        self.posts = []        # with seams: (kind, gain with layer scale and constant, eps) after the mixer, after the feed-forward
+        if self.seams:
+            if not all(hasattr(n, "row_norm") for n in norms):
+                raise ValueError("a layer scale or a constant on the sublayers' outputs needs norms that describe themselves (row_norm)")
+            self.takes_pending = True
+            self.takes_open = ("post_sum",)
 
     def _children(self):
         s = self.spec
@@ -87,7 +108,35 @@ class SandwichBlock(PreNormBlock):
             kids.append((s.ffn_post_norm_prefix, self.ffn_post))
         return kids
 
+    def param_specs(self) -> List[ParamSpec]:
+        out = super().param_specs()
+        if self.scale_names is not None:
+            for k, name in enumerate(self.scale_names[:2]):
+                # (a layer without a feed-forward may still store the second vector, and the norms: taken and not used)
+                out.append(ParamSpec(name, (self.hidden_size,), role="gain", init="ones", optional=k == 1 and self.ffn is None))
+        if self.ffn is None:
+            s = self.spec
+            for norm, prefix in ((s.ffn_norm, s.ffn_norm_prefix), (s.ffn_post_norm, s.ffn_post_norm_prefix)):
+                if norm is not None:
+                    out.append(ParamSpec(prefix + getattr(norm, "param", "weight"), (self.hidden_size,), role="gain", init="ones",
+                                         optional=True))
+        return out
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        super().bind(tensors)
+        if self.seams:
+            self.posts = []
+            for k, norm in enumerate((self.mixer_post, self.ffn_post)):
+                if norm is None:
+                    continue
+                kind, gain, eps = norm.row_norm()
+                if self.scale_names is not None:
+                    gain = gain * tensors[self.scale_names[k]].float()
+                self.posts.append((kind, (gain * self.mult).contiguous(), eps))
+
     def forward(self, residual, batch, cache, owns_cache: bool = True) -> None:
+        if self.seams:
+            return self._forward_seams(residual, batch, cache, owns_cache)
         x = self._normed(self.mixer_norm, residual)
         branch = torch.empty_like(residual)
         self.mixer.forward(x, branch, batch, cache, owns_cache, accumulate=False)
@@ -105,6 +154,23 @@ class SandwichBlock(PreNormBlock):
             else:
                 self.ffn.forward(x, branch, batch, accumulate=False)
                 self.ffn_post.add_to(branch, residual)
+
+    def _forward_seams(self, residual, batch, cache, owns_cache) -> None:
+        dtype = self.ctx.dtype
+        branch, post = batch.extras.pop("post_sum", (None, None))      # what the block before left
+        x = ops.row_step(residual, branch, post, then=self.mixer_norm.row_norm(), out_dtype=dtype)
+        if hasattr(self.mixer, "forward_open"):
+            y = self.mixer.forward_open(x, batch, cache, owns_cache)
+        else:
+            y = torch.empty_like(residual)
+            self.mixer.forward(x, y, batch, cache, owns_cache, accumulate=None)
+        post = self.posts[0]
+        if self.ffn is not None:
+            x = ops.row_step(residual, y, post, then=self.ffn_norm.row_norm(), out_dtype=dtype)
+            y = torch.empty_like(residual)
+            self.ffn.forward(x, y, batch, accumulate=None)
+            post = self.posts[1]
+        batch.extras["post_sum"] = (y, post)
 
 
 register_block("prenorm", PreNormBlock)
@@ -203,7 +269,7 @@ class ParallelBlock(PreNormBlock):
     else calls :func:`flush_scaled_sum` first (the decoder does, before a block of another kind, before the model's last
     norm and before it hands the stream out)."""
     takes_pending = True
-    takes_scaled_sum = True
+    takes_open = ("scaled_sum",)
 
     def __init__(self, layer_spec, hidden_size: int, ctx: BuildContext):
         self.spec = layer_spec
@@ -311,6 +377,16 @@ def flush_scaled_sum(residual, batch) -> None:
     pend = batch.extras.pop("scaled_sum", None)
     if pend is not None:
         ops.scale_add(residual, *pend)
+
+
+def flush_open_sums(residual, batch, keep=()) -> None:
+    """Makes what the block before left to the stream's next reader, except the kinds that this reader takes (``keep``)."""
+    if "scaled_sum" not in keep:
+        flush_scaled_sum(residual, batch)
+    if "post_sum" not in keep:
+        pend = batch.extras.pop("post_sum", None)
+        if pend is not None:
+            ops.row_step(residual, pend[0], pend[1])
 
 
 register_block("parallel", ParallelBlock)

@@ -49,6 +49,21 @@ class Linear:
         else:
             self(x, out=out)
 
+    def planes(self, x: torch.Tensor, behind: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+        """``x @ W.T (+ bias)`` of a few tokens on the tensor-core path as float32 planes [S, T, out] that their reader adds
+        up (``ops.gemm_tc_planes``: good until the plane buffer is written again); None where the product is not left open.
+        ``behind``: planes of the product before, which stay good: the new ones lie behind them (None if there is no room)."""
+        T = x.shape[0]
+        w = self.weight
+        if not (ops.DEFER_SUMS and w.dtype == torch.bfloat16 and x.dtype == w.dtype and T <= ops.DEFER_MAX_TOKENS
+                and T * w.shape[0] <= ops.PLANE_BUFFER_ELEMS and ops.gemm_tc_supports(x, w)):
+            return None
+        if behind is None:
+            return ops.gemm_tc_planes(x, w, self.bias)
+        if not ops.planes_fit_behind(behind):
+            return None
+        return ops.gemm_tc_planes(x, w, self.bias, after=behind.numel())
+
     def add_to(self, x: torch.Tensor, residual: torch.Tensor) -> None:
         """``residual += x @ W.T (+ bias)`` (float32).  For a few tokens on the tensor-core path the sum
         of the K splits is left to the next reader of ``residual`` (``ops.gemm_tc_deferred``)."""

@@ -5,6 +5,11 @@ double and rounds twice through bfloat16; here: one float32 computation and one
 rounding on store).  ``rows`` normalises only the named rows (final norm on the
 positions whose logits are wanted, src/core/engine.cpp:1029-1035).  With the spec's ``offset`` the gain is
 ``offset + w`` (a weight stored around zero with offset 1), made once at load in float32.
+
+:class:`LayerNorm`: (x - mean) / sqrt(mean((x - mean)^2) + eps) * w, no bias, everything float32.
+
+Both describe themselves to kernels that norm a row inside another pass over it (``row_norm``: the kind, the float32
+gain and eps, as ``ops.row_step`` takes them).
 """
 from __future__ import annotations
 
@@ -44,6 +49,9 @@ class RMSNorm(Norm):
             self._gain_f32 = self.weight.float().contiguous()
         return self._gain_f32
 
+    def row_norm(self) -> tuple:
+        return ops.NORM_RMS, self.gain_f32(), self.eps
+
     def add_to(self, x: torch.Tensor, stream: torch.Tensor) -> None:
         """``stream += norm(x)`` (float32 both): the norm of a sublayer's output on its way into the stream."""
         ops.rmsnorm_add(x, self.weight, self.eps, stream)
@@ -59,4 +67,29 @@ class RMSNorm(Norm):
         return ops.rmsnorm(x, self.weight, self.eps, self.ctx.dtype, rows=rows)
 
 
+class LayerNorm(Norm):
+    def __init__(self, spec, hidden_size: int, ctx: BuildContext):
+        self.eps = float(spec.eps)
+        self.hidden_size = hidden_size
+        self.ctx = ctx
+        self.param = getattr(spec, "param", "weight")
+        self.gain: Optional[torch.Tensor] = None
+
+    def param_specs(self) -> List[ParamSpec]:
+        return [ParamSpec(self.param, (self.hidden_size,), role="gain", init="ones")]
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.gain = tensors[self.param].float().contiguous()
+
+    def row_norm(self) -> tuple:
+        return ops.NORM_LAYER, self.gain, self.eps
+
+    def add_to(self, x: torch.Tensor, stream: torch.Tensor) -> None:
+        ops.row_step(stream, x, post=self.row_norm())
+
+    def forward(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        return ops.row_step(x, then=self.row_norm(), rows=rows, out_dtype=self.ctx.dtype)
+
+
 register_norm("rmsnorm", RMSNorm)
+register_norm("layernorm", LayerNorm)
