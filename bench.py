@@ -406,8 +406,41 @@ VUBOTAR_SHAPES = {
     "2k": (2048, 16, 4, 128, 1024, 4, 8, 128, 256, 16, 128, 64, 128, 192, 768, 16, 2, 1024, 32000),
     "4k": (4096, 32, 8, 128, 1024, 4, 16, 128, 256, 32, 128, 64, 128, 192, 1536, 8, 2, 3584, 32000),
 }
+
+
+def _zanivik_shape(width, heads, kv, hd, window, d_heads, d_kv, d_dk, d_dv, s_heads, s_dv, s_state, s_groups, ff, gla, vocab, pairs):
+    """``pairs`` times (a layer with sink attention beside the gated delta rule, a layer with shared-kv attention beside the
+    state-space mixer), each with a dense gelu feed-forward; beside it the dense decoder of equal width, depth and heads with
+    a gated feed-forward of about as many weights, and the closest designs the engine had before: Gafulix (norms on both sides
+    of a sublayer, gated linear attention with as many state entries as the delta rule) and Vubotar (per-head norms,
+    windowed attention with a sink, a recurrence with one decay per head) with the same heads and window."""
+    rot = {"base": 500000.0, "dims": hd, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}
+    att = {"heads": heads, "kv_heads": kv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": {"size": window}, "rot": rot}
+    mlp = {"kind": "dense", "ff": ff}
+    a = {"type": "parallel", "mlp": mlp,
+         "mixer": {"left": att, "left_scale": 0.7, "right_scale": 0.6,
+                   "right": {"heads": d_heads, "kv_heads": d_kv, "dim": d_dk, "vdim": d_dv, "conv": 4}}}
+    b = {"type": "parallel_2", "mlp": mlp,
+         "mixer": {"left": att, "right": {"heads": s_heads, "vdim": s_dv, "state": s_state, "groups": s_groups, "conv": 4,
+                                          "norm_groups": s_groups}}}
+    design = {"architecture": "Zanivik", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+              "layers": [a, b] * pairs}
+    gafulix, dense = _gafulix_shape(width, heads, kv, hd, *gla, 16, 2, ff * 2 // 6 // 64 * 64, window, vocab, pairs)
+    dense["intermediate_size"] = ff * 2 // 3 // 64 * 64
+    vubotar = _vubotar_shape(width, heads, kv, hd, window, 4, *gla, heads, hd, 64, hd, 192, 768, 16, 2, ff * 2 // 6 // 64 * 64, vocab)[0]
+    return design, dense, {"gafulix": gafulix, "vubotar": vubotar}
+
+
+ZANIVIK_SHAPES = {
+    # width, heads, kv heads, head size, window, delta rule: heads, query/key heads, key size, value size, state space: heads,
+    # value size, state size, groups, feed-forward size, gated linear attention of the closest: heads, key size, value size,
+    # vocab, layer pairs
+    "2k": (2048, 16, 4, 128, 1024, 16, 8, 128, 128, 64, 64, 128, 4, 8192, (16, 128, 128), 32000, 2),
+    "4k": (4096, 32, 8, 128, 1024, 32, 16, 128, 128, 128, 64, 128, 8, 16384, (32, 128, 128), 32000, 2),
+}
 DESIGNS = {"gafulix": (_gafulix_shape, DESIGN_SHAPES), "fuvevik": (_fuvevik_shape, FUVEVIK_SHAPES),
-           "zigipel": (_zigipel_shape, ZIGIPEL_SHAPES), "vubotar": (_vubotar_shape, VUBOTAR_SHAPES)}
+           "zigipel": (_zigipel_shape, ZIGIPEL_SHAPES), "vubotar": (_vubotar_shape, VUBOTAR_SHAPES),
+           "zanivik": (_zanivik_shape, ZANIVIK_SHAPES)}
 
 
 def design_comparison(args):

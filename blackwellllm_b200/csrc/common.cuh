@@ -208,6 +208,115 @@ __device__ __forceinline__ float out_gate(const float* __restrict__ gate, long l
     return 1.f / (1.f + expf(-gate[token * (size_t)ld + (size_t)head * dv + c]));
 }
 
+// Two float32 operations in one instruction (sm_100: the packed form of fma and mul); a pair is a 64-bit register, the first
+// value in the low half.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float lo, float hi) {
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ void unpack2(f32x2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ float sum2(f32x2 v) { float a, b; unpack2(v, a, b); return a + b; }
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+
+// The register tiles of the recurrent scans (gla.cu, delta.cu): lane = 8 * rg + cg; a lane holds TILE_ROWS state rows of its
+// row group rg (4 groups a warp) and a few neighbouring value columns of its column group cg (8 groups).  What a lane reads
+// of a token from shared memory (its rows' key and query channels, its columns' values) then serves rows x columns elements.
+constexpr int TILE_ROWS = 8, TILE_RG = 4, TILE_CG = 8, TILE_WARP_ROWS = TILE_ROWS * TILE_RG;
+
+// Sums over the row groups (lane bits 3 and 4).  Four values per lane: the lane gets the sum of value 2 b4 + b3 (b4, b3: its
+// bits 4 and 3); two values: of value b4 (in both lanes of bit 3).
+__device__ __forceinline__ float tile_sum4(float a0, float a1, float a2, float a3) {
+    const bool hi16 = threadIdx.x & 16, hi8 = threadIdx.x & 8;
+    const float g0 = __shfl_xor_sync(0xffffffffu, hi16 ? a0 : a2, 16);
+    const float g1 = __shfl_xor_sync(0xffffffffu, hi16 ? a1 : a3, 16);
+    const float b0 = (hi16 ? a2 : a0) + g0, b1 = (hi16 ? a3 : a1) + g1;
+    return (hi8 ? b1 : b0) + __shfl_xor_sync(0xffffffffu, hi8 ? b0 : b1, 8);
+}
+__device__ __forceinline__ float tile_sum2(float a0, float a1) {
+    const bool hi16 = threadIdx.x & 16;
+    const float b = (hi16 ? a1 : a0) + __shfl_xor_sync(0xffffffffu, hi16 ? a0 : a1, 16);
+    return b + __shfl_xor_sync(0xffffffffu, b, 8);
+}
+
+// A lane's tile of a state [rows, ld] in memory, row0 its first row, col0 its first column; rows from `rows` on and columns
+// from `cols` on count as zeros and are not written.  s[j][c]: rows row0 + 2 j and + 1 of column col0 + c.
+template <int CPT>
+__device__ __forceinline__ void tile_load(f32x2 (&s)[TILE_ROWS / 2][CPT], const float* __restrict__ S, int row0, int rows, int ld,
+                                          int col0, int cols) {
+    const bool vec = (ld % CPT) == 0 && col0 + CPT <= ld && ((uintptr_t)S & (4 * CPT - 1)) == 0;
+#pragma unroll
+    for (int j = 0; j < TILE_ROWS / 2; ++j) {
+        float v[2][CPT];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int i = row0 + 2 * j + e;
+            const float* src = S + (size_t)i * ld + col0;
+            if (vec && i < rows) {
+                if constexpr (CPT == 4) {
+                    const float4 t = *reinterpret_cast<const float4*>(src);
+                    v[e][0] = t.x; v[e][1] = t.y; v[e][2] = t.z; v[e][3] = t.w;
+                } else {
+                    const float2 t = *reinterpret_cast<const float2*>(src);
+                    v[e][0] = t.x; v[e][1] = t.y;
+                }
+            } else {
+#pragma unroll
+                for (int c = 0; c < CPT; ++c) v[e][c] = (i < rows && col0 + c < cols) ? src[c] : 0.f;
+            }
+        }
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) s[j][c] = pack2(v[0][c], v[1][c]);
+    }
+}
+template <int CPT>
+__device__ __forceinline__ void tile_store(const f32x2 (&s)[TILE_ROWS / 2][CPT], float* __restrict__ S, int row0, int rows, int ld,
+                                           int col0, int cols) {
+    const bool vec = (ld % CPT) == 0 && col0 + CPT <= ld && ((uintptr_t)S & (4 * CPT - 1)) == 0;
+#pragma unroll
+    for (int j = 0; j < TILE_ROWS / 2; ++j) {
+        float v[2][CPT];
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) unpack2(s[j][c], v[0][c], v[1][c]);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int i = row0 + 2 * j + e;
+            if (i >= rows) continue;
+            float* dst = S + (size_t)i * ld + col0;
+            if (vec) {
+                if constexpr (CPT == 4) *reinterpret_cast<float4*>(dst) = make_float4(v[e][0], v[e][1], v[e][2], v[e][3]);
+                else *reinterpret_cast<float2*>(dst) = make_float2(v[e][0], v[e][1]);
+            } else {
+#pragma unroll
+                for (int c = 0; c < CPT; ++c)
+                    if (col0 + c < cols) dst[c] = v[e][c];
+            }
+        }
+    }
+}
+// CPT neighbouring floats from shared memory, each as a pair of itself twice
+template <int CPT>
+__device__ __forceinline__ void tile_values(f32x2 (&v)[CPT], const float* src, float scale) {
+    if constexpr (CPT == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(src);
+        v[0] = pack2(t.x * scale, t.x * scale); v[1] = pack2(t.y * scale, t.y * scale);
+        v[2] = pack2(t.z * scale, t.z * scale); v[3] = pack2(t.w * scale, t.w * scale);
+    } else {
+        const float2 t = *reinterpret_cast<const float2*>(src);
+        v[0] = pack2(t.x * scale, t.x * scale); v[1] = pack2(t.y * scale, t.y * scale);
+    }
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

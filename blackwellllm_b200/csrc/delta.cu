@@ -6,7 +6,7 @@
 // delta_scan_kernel walks the tokens of one request's portion in order (a single decoded token and a portion of a prompt
 // are the same case), from the state the steps before left in the request's slot, and leaves the new state there.  A block
 // owns (request, head, COLS value columns); LPC neighbouring lanes own one column, its dk state rows spread over them, in
-// registers.  The chain through the tokens is one product with k, a sum over LPC lanes and the update; the sum for q of
+// registers, two rows per packed instruction.  The chain through the tokens is one product with k, a sum over LPC lanes and the update; the sum for q of
 // the token before rides in the same shuffles.  The order of all sums depends on dk alone, never on how the tokens were
 // cut into steps or on the batch.  Everything is float32.
 #include "common.cuh"
@@ -15,7 +15,7 @@ using bf16 = __nv_bfloat16;
 
 namespace {
 
-constexpr int THREADS = 256;
+constexpr int THREADS = 128;
 constexpr int TOK = 16;        // tokens staged in shared memory at a time
 constexpr int MAX_DK = 256;
 
@@ -45,11 +45,12 @@ delta_scan_kernel(DeltaParams p) {
     const int hk = h / p.rep;
     float* S = p.state + ((size_t)p.state_slot[r] * p.heads + h) * (size_t)p.dk * p.dv;
     BW_PDL_WAIT();
-    float s[RPL];
+    bw::f32x2 s[RPL / 2];
 #pragma unroll
-    for (int j = 0; j < RPL; ++j) {
-        const int i = ((j >> 2) * LPC + l) * 4 + (j & 3);
-        s[j] = (i < p.dk && col < p.dv) ? S[(size_t)i * p.dv + col] : 0.f;
+    for (int j = 0; j < RPL / 2; ++j) {
+        const int i = ((j >> 1) * LPC + l) * 4 + (j & 1) * 2;
+        s[j] = bw::pack2((i < p.dk && col < p.dv) ? S[(size_t)i * p.dv + col] : 0.f,
+                         (i + 1 < p.dk && col < p.dv) ? S[(size_t)(i + 1) * p.dv + col] : 0.f);
     }
     // the next chunk's values travel into registers while this chunk is worked on from shared memory
     float rq[NST], rk[NST], rv[NSV], rg = 0.f, rb = 0.f;
@@ -77,8 +78,8 @@ delta_scan_kernel(DeltaParams p) {
         }
     };
     if (t0 < t1) fetch(t0, min(TOK, t1 - t0));
-    const float4* q4 = reinterpret_cast<const float4*>(qs);
-    const float4* k4 = reinterpret_cast<const float4*>(ks);
+    const ulonglong2* q4 = reinterpret_cast<const ulonglong2*>(qs);
+    const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(ks);
     const bool writes = l == 0 && col < p.dv;
     float* orow = p.o + (size_t)h * p.dv + col;          // + token * heads * dv
     const size_t o_ld = (size_t)p.heads * p.dv;
@@ -100,19 +101,18 @@ delta_scan_kernel(DeltaParams p) {
         for (int tt = 0; tt < n; ++tt) {
             const int base = tt * (DKP / 4) + l;
             const float g = gs[tt], beta = bs[tt], v = vs[tt * COLS + cc];
-            float a[4] = {0.f, 0.f, 0.f, 0.f};
-            float kk[RPL];
+            const bw::f32x2 g2 = bw::pack2(g, g);
+            bw::f32x2 a0 = 0, a1 = 0;          // (pairs of zeros)
+            ulonglong2 kk[RPL / 4];
 #pragma unroll
             for (int j = 0; j < RPL / 4; ++j) {
-                const float4 k = k4[base + j * LPC];
-                kk[4 * j] = k.x; kk[4 * j + 1] = k.y; kk[4 * j + 2] = k.z; kk[4 * j + 3] = k.w;
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    s[4 * j + e] *= g;
-                    a[e] = fmaf(s[4 * j + e], kk[4 * j + e], a[e]);
-                }
+                kk[j] = k4[base + j * LPC];
+                s[2 * j] = bw::mul2(s[2 * j], g2);
+                s[2 * j + 1] = bw::mul2(s[2 * j + 1], g2);
+                a0 = bw::fma2(s[2 * j], kk[j].x, a0);
+                a1 = bw::fma2(s[2 * j + 1], kk[j].y, a1);
             }
-            float pk = (a[0] + a[1]) + (a[2] + a[3]);
+            float pk = bw::sum2(a0) + bw::sum2(a1);
 #pragma unroll
             for (int d = LPC / 2; d > 0; d >>= 1) {
                 pk += __shfl_xor_sync(0xffffffffu, pk, d);
@@ -120,27 +120,29 @@ delta_scan_kernel(DeltaParams p) {
             }
             if (writes && tb + tt > t0) orow[(size_t)(tb + tt - 1) * o_ld] = pq;
             const float u = beta * (v - pk);
-            float b[4] = {0.f, 0.f, 0.f, 0.f};
+            const bw::f32x2 u2 = bw::pack2(u, u);
+            bw::f32x2 b0 = 0, b1 = 0;
 #pragma unroll
             for (int j = 0; j < RPL / 4; ++j) {
-                const float4 q = q4[base + j * LPC];
-                const float qe[4] = {q.x, q.y, q.z, q.w};
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    s[4 * j + e] = fmaf(kk[4 * j + e], u, s[4 * j + e]);
-                    b[e] = fmaf(s[4 * j + e], qe[e], b[e]);
-                }
+                const ulonglong2 q = q4[base + j * LPC];
+                s[2 * j] = bw::fma2(kk[j].x, u2, s[2 * j]);
+                s[2 * j + 1] = bw::fma2(kk[j].y, u2, s[2 * j + 1]);
+                b0 = bw::fma2(s[2 * j], q.x, b0);
+                b1 = bw::fma2(s[2 * j + 1], q.y, b1);
             }
-            pq = (b[0] + b[1]) + (b[2] + b[3]);
+            pq = bw::sum2(b0) + bw::sum2(b1);
         }
     }
 #pragma unroll
     for (int d = LPC / 2; d > 0; d >>= 1) pq += __shfl_xor_sync(0xffffffffu, pq, d);
     if (writes && t1 > t0) orow[(size_t)(t1 - 1) * o_ld] = pq;
 #pragma unroll
-    for (int j = 0; j < RPL; ++j) {
-        const int i = ((j >> 2) * LPC + l) * 4 + (j & 3);
-        if (i < p.dk && col < p.dv) S[(size_t)i * p.dv + col] = s[j];
+    for (int j = 0; j < RPL / 2; ++j) {
+        const int i = ((j >> 1) * LPC + l) * 4 + (j & 1) * 2;
+        float lo, hi;
+        bw::unpack2(s[j], lo, hi);
+        if (i < p.dk && col < p.dv) S[(size_t)i * p.dv + col] = lo;
+        if (i + 1 < p.dk && col < p.dv) S[(size_t)(i + 1) * p.dv + col] = hi;
     }
 }
 

@@ -9,11 +9,12 @@
 //
 // gla_scan_kernel walks the tokens of one request's segment in order (a single decoded token and a
 // portion of a prompt are the same case), from the state the steps before left in the request's slot,
-// and leaves the new state there.  A block owns (request, head, COLS value columns); a warp owns CPT of
-// them, their dk state rows spread over its lanes, in registers.  The order of all sums
-// depends on dk alone, never on how the tokens were cut into steps or on the batch.  The scan is a chain
-// through the tokens (state in float32, as the design asks): it is bound by the latency of one token's
-// update, not by memory or arithmetic throughput, and its parallelism is requests x heads x columns / COLS.
+// and leaves the new state there.  A block owns (request, head, COLS value columns); its state lies in registers, a tile of
+// rows x columns per lane (common.cuh), two rows per packed instruction.  A token's S^T q is summed over a warp's row groups
+// by shuffles that nothing waits for, the warps' parts go to shared memory and are added, in warp order, after 16 tokens.
+// The order of all sums depends on dk alone, never on how the tokens were cut into steps or on the batch.  The scan keeps
+// float32 throughout (as the design asks): it is bound by the issue of its packed multiply-adds and the shared-memory reads
+// that feed them, and its parallelism is requests x heads x columns / COLS.
 //
 // gla_decay_kernel makes a_t from the first projection's result (W2 has a small inner size: float32 FMAs).
 // gla_gate_kernel: per token and head, o / rms(o) * gain * silu(g) -> the output projection's operand.
@@ -23,9 +24,9 @@ using bf16 = __nv_bfloat16;
 
 namespace {
 
-constexpr int COLS = 32;        // value columns of a block
-constexpr int CPT = 4;          // value columns of a warp (and of each of its lanes)
-constexpr int THREADS = 32 * COLS / CPT;
+#ifndef SCAN_NARROW_BELOW
+#define SCAN_NARROW_BELOW 3     // quarters of the SM count: with fewer 32-column blocks than that they become 16 columns wide
+#endif
 constexpr int MAX_DK = 256;
 constexpr int TOK_CHUNK = 16;   // tokens staged in shared memory at a time
 
@@ -42,7 +43,7 @@ struct ScanParams {
     float q_scale;
     // The same recurrence serves a matrix memory with ONE decay per head and token and a normaliser:
     // scalar_decay != 0: decay is [T, heads] (a_t of the head, used for every key channel);
-    // k_scale != null: [T, heads], the token's keys are multiplied by it as they are read (an input gate);
+    // k_scale != null: [T, heads], the token's keys count times it (an input gate);
     // ones_col != 0: the head's last value column (dv - 1) is the constant 1 and v holds dv - 1 columns a head, so that
     // column of the state is n_t = a_t n_(t-1) + k_t and the last output column is n_t . q_t.
     const float* k_scale;
@@ -76,71 +77,59 @@ gla_decay_kernel(const float* __restrict__ x, long long ldx, int x_off, const WT
     a[idx] = expf(log_sigmoid(z) * inv_tau);
 }
 
-// RPL: state rows per lane (a multiple of 4): dk <= 32 * RPL.  A warp owns CPT value columns and all key
-// channels: lane l holds channels (j * 32 + l) * 4 + e (j < RPL / 4, e < 4) of each of its columns, so a token's
-// q, k and a values are read from shared memory once per warp (16-byte loads, 512 consecutive bytes a warp)
-// and used for CPT columns.  In shared memory a token's rows are padded with zeros to DKP = 32 * RPL channels
-// (a padded channel stays at zero and adds nothing), so the inner loop has no bounds.  The CPT sums over the
-// 32 lanes take six shuffles: two that halve the number of columns a lane carries, then three over what is left.
+// NW warps of 32 state rows: dk <= DKP = 32 NW.  CPT value columns a lane: COLS = 8 CPT.  In shared memory a token's q, k
+// (and a) are padded with zeros to DKP channels (a padded channel stays at zero and adds nothing), so the inner loop has no
+// bounds.
 // MEM: the form for a matrix memory (ScanParams: one decay per head, keys times k_scale, the column of ones, query/key
-// heads shared by several heads); the plain
-// form's code does not know of it.  What a fetch loads is not touched before it is staged: a thread never waits for a
-// load inside the fetch, so the key's scale travels in registers of its own and multiplies at staging.
-template <int RPL, bool MEM>
-__global__ void __launch_bounds__(THREADS)
+// heads shared by several heads); the plain form's code does not know of it.  What a fetch loads is not touched before it
+// is staged: a thread never waits for a load inside the fetch.  The key's scale multiplies the token's value instead, which is
+// the same product.
+template <int NW, int CPT, bool MEM>
+struct ScanSmem {
+    static constexpr int DKP = NW * bw::TILE_WARP_ROWS, COLS = bw::TILE_CG * CPT;
+    static constexpr int floats = (MEM ? 2 : 3) * TOK_CHUNK * DKP + TOK_CHUNK * COLS + 2 * TOK_CHUNK + TOK_CHUNK * NW * COLS;
+};
+
+template <int NW, int CPT, bool MEM>
+__global__ void __launch_bounds__(32 * NW)
 gla_scan_kernel(ScanParams p) {
     BW_PDL_TRIGGER();
-    constexpr int DKP = 32 * RPL;
+    constexpr int THREADS = 32 * NW, DKP = NW * bw::TILE_WARP_ROWS, COLS = bw::TILE_CG * CPT, RP = bw::TILE_ROWS / 2;
     extern __shared__ __align__(16) float sm[];
-    float* qs = sm;                          // [TOK_CHUNK][DKP]
+    float* qs = sm;                                      // [TOK_CHUNK][DKP]
     float* ks = qs + TOK_CHUNK * DKP;
-    float* as = ks + TOK_CHUNK * DKP;
-    float* vs = as + TOK_CHUNK * DKP;        // [TOK_CHUNK][COLS]
-    constexpr int NST = TOK_CHUNK * DKP / THREADS;   // staged values of q, k, a per thread
-    constexpr int NSV = TOK_CHUNK * COLS / THREADS;
+    float* as = ks + TOK_CHUNK * DKP;                    // plain form: [TOK_CHUNK][DKP]
+    float* vs = as + (MEM ? 0 : TOK_CHUNK * DKP);        // [TOK_CHUNK][COLS]
+    float* gs = vs + TOK_CHUNK * COLS;                   // MEM: [TOK_CHUNK] decays, [TOK_CHUNK] scales of the keys
+    float* part = gs + 2 * TOK_CHUNK;                    // [TOK_CHUNK][NW][COLS]
+    constexpr int NST = TOK_CHUNK * DKP / THREADS;       // staged values of q, k, a per thread
+    constexpr int NSV = (TOK_CHUNK * COLS + THREADS - 1) / THREADS;
     const int r = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * COLS;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int cbase = c0 + warp * CPT;
+    const int rg = lane >> 3, cg = lane & 7;
+    const int row0 = warp * bw::TILE_WARP_ROWS + rg * bw::TILE_ROWS;
     const int t0 = p.cu_q[r], t1 = p.cu_q[r + 1];
     const int hk = MEM ? h / p.rep : h;
     float* S = p.state + (((size_t)p.state_slot[r] * p.heads + h) * p.dk) * p.sld;
     BW_PDL_WAIT();
-    float s[RPL][CPT];
-    const bool vec_state = (p.sld & 3) == 0 && cbase + CPT <= p.sld;   // a lane's CPT columns of a row as one 16-byte access
-#pragma unroll
-    for (int j = 0; j < RPL; ++j) {
-        const int i = ((j >> 2) * 32 + lane) * 4 + (j & 3);
-        if (vec_state) {
-            const float4 v = i < p.dk ? *reinterpret_cast<const float4*>(S + (size_t)i * p.sld + cbase) : make_float4(0.f, 0.f, 0.f, 0.f);
-            s[j][0] = v.x; s[j][1] = v.y; s[j][2] = v.z; s[j][3] = v.w;
-        } else {
-#pragma unroll
-            for (int cc = 0; cc < CPT; ++cc) s[j][cc] = (i < p.dk && cbase + cc < p.dv) ? S[(size_t)i * p.sld + cbase + cc] : 0.f;
-        }
-    }
+    bw::f32x2 s[RP][CPT];
+    bw::tile_load<CPT>(s, S, row0, p.dk, p.sld, c0 + cg * CPT, p.dv);
     // The next chunk's values travel from memory into registers while this chunk is worked on from shared
     // memory, so that their latency is not added to the chain through the tokens.
-    float rq[NST], rk[NST], ra[NST], rv[NSV];
-    float rs[MEM ? NST : 1];
+    float rq[NST], rk[NST], ra[MEM ? 1 : NST], rv[NSV], rg_ = 0.f, rs = 1.f;
     const int dv_in = p.dv - ((MEM && p.ones_col) ? 1 : 0);   // value columns a head has in memory
     auto fetch = [&](int tb, int n) {
 #pragma unroll
         for (int u = 0; u < NST; ++u) {
             const int idx = threadIdx.x + u * THREADS;
             const int tt = idx / DKP, i = idx % DKP;
-            rq[u] = rk[u] = ra[u] = 0.f;
-            if constexpr (MEM) rs[u] = 1.f;
+            rq[u] = rk[u] = 0.f;
+            if constexpr (!MEM) ra[u] = 0.f;
             if (tt < n && i < p.dk) {
                 const float* row = p.qkv + (size_t)(tb + tt) * p.ld;
                 rq[u] = row[p.q_off + hk * p.dk + i];
                 rk[u] = row[p.k_off + hk * p.dk + i];
-                if constexpr (MEM) {
-                    if (p.k_scale) rs[u] = p.k_scale[(size_t)(tb + tt) * p.heads + h];
-                    ra[u] = p.scalar_decay ? p.decay[(size_t)(tb + tt) * p.heads + h]
-                                           : p.decay[(size_t)(tb + tt) * p.heads * p.dk + h * p.dk + i];
-                } else {
-                    ra[u] = p.decay[(size_t)(tb + tt) * p.heads * p.dk + h * p.dk + i];
-                }
+                if constexpr (!MEM) ra[u] = p.decay[(size_t)(tb + tt) * p.heads * p.dk + h * p.dk + i];
             }
         }
 #pragma unroll
@@ -150,67 +139,93 @@ gla_scan_kernel(ScanParams p) {
             rv[u] = (tt < n && c0 + cc < dv_in) ? p.qkv[(size_t)(tb + tt) * p.ld + p.v_off + h * dv_in + c0 + cc]
                                                 : ((MEM && tt < n && p.ones_col && c0 + cc == dv_in) ? 1.f : 0.f);
         }
+        if constexpr (MEM) {
+            if (threadIdx.x < TOK_CHUNK && (int)threadIdx.x < n) {
+                rg_ = p.decay[(size_t)(tb + threadIdx.x) * p.heads + h];
+                if (p.k_scale) rs = p.k_scale[(size_t)(tb + threadIdx.x) * p.heads + h];
+            }
+        }
     };
     if (t0 < t1) fetch(t0, min(TOK_CHUNK, t1 - t0));
-    const float4* q4 = reinterpret_cast<const float4*>(qs);
-    const float4* k4 = reinterpret_cast<const float4*>(ks);
-    const float4* a4 = reinterpret_cast<const float4*>(as);
-    const float4* v4 = reinterpret_cast<const float4*>(vs);
-    const bool hi16 = lane & 16, hi8 = lane & 8;
-    const int my_col = cbase + (hi16 ? 2 : 0) + (hi8 ? 1 : 0);   // the column whose sum ends in this lane (lanes 0, 8, 16, 24)
+    const ulonglong2* q2 = reinterpret_cast<const ulonglong2*>(qs + row0);
+    const ulonglong2* k2 = reinterpret_cast<const ulonglong2*>(ks + row0);
+    const ulonglong2* a2 = reinterpret_cast<const ulonglong2*>(as + row0);
+    // the column whose sum ends in this lane, and whether this lane stores it
+    const int my_col = cg * CPT + (CPT == 4 ? ((lane & 16) ? 2 : 0) + ((lane & 8) ? 1 : 0) : ((lane & 16) ? 1 : 0));
+    const bool mine = CPT == 4 || (lane & 8) == 0;
     for (int tb = t0; tb < t1; tb += TOK_CHUNK) {
         const int n = min(TOK_CHUNK, t1 - tb);
         __syncthreads();                      // the chunk before has been read
 #pragma unroll
         for (int u = 0; u < NST; ++u) {
             const int idx = threadIdx.x + u * THREADS;
-            qs[idx] = rq[u] * p.q_scale; as[idx] = ra[u];
-            if constexpr (MEM) ks[idx] = rk[u] * rs[u]; else ks[idx] = rk[u];
+            qs[idx] = rq[u] * p.q_scale;
+            ks[idx] = rk[u];
+            if constexpr (!MEM) as[idx] = ra[u];
         }
 #pragma unroll
-        for (int u = 0; u < NSV; ++u) vs[threadIdx.x + u * THREADS] = rv[u];
+        for (int u = 0; u < NSV; ++u) {
+            const int idx = threadIdx.x + u * THREADS;
+            if (TOK_CHUNK * COLS % THREADS == 0 || idx < TOK_CHUNK * COLS) vs[idx] = rv[u];
+        }
+        if constexpr (MEM) { if (threadIdx.x < TOK_CHUNK) { gs[threadIdx.x] = rg_; gs[TOK_CHUNK + threadIdx.x] = rs; } }
         __syncthreads();
         if (tb + TOK_CHUNK < t1) fetch(tb + TOK_CHUNK, min(TOK_CHUNK, t1 - tb - TOK_CHUNK));
 #pragma unroll 2
         for (int tt = 0; tt < n; ++tt) {
-            const float4 vv = v4[tt * (COLS / 4) + warp];
-            const float v[CPT] = {vv.x, vv.y, vv.z, vv.w};
-            const int base = tt * (DKP / 4) + lane;
-            float acc[CPT] = {0.f, 0.f, 0.f, 0.f};
+            bw::f32x2 v[CPT], g = 0;
+            bw::tile_values<CPT>(v, vs + tt * COLS + cg * CPT, MEM ? gs[TOK_CHUNK + tt] : 1.f);
+            if constexpr (MEM) { const float g1 = gs[tt]; g = bw::pack2(g1, g1); }
+            bw::f32x2 acc[CPT];
 #pragma unroll
-            for (int j = 0; j < RPL / 4; ++j) {
-                const float4 a = a4[base + j * 32], k = k4[base + j * 32], q = q4[base + j * 32];
-                const float ae[4] = {a.x, a.y, a.z, a.w}, ke[4] = {k.x, k.y, k.z, k.w}, qe[4] = {q.x, q.y, q.z, q.w};
+            for (int c = 0; c < CPT; ++c) acc[c] = 0;     // (two zeros)
 #pragma unroll
-                for (int e = 0; e < 4; ++e)
+            for (int j = 0; j < RP / 2; ++j) {
+                const ulonglong2 k = k2[tt * (DKP / 4) + j], q = q2[tt * (DKP / 4) + j];
+                ulonglong2 a;
+                if constexpr (MEM) { a.x = g; a.y = g; } else a = a2[tt * (DKP / 4) + j];
 #pragma unroll
-                    for (int cc = 0; cc < CPT; ++cc) {
-                        s[4 * j + e][cc] = fmaf(ae[e], s[4 * j + e][cc], ke[e] * v[cc]);
-                        acc[cc] = fmaf(s[4 * j + e][cc], qe[e], acc[cc]);
-                    }
+                for (int c = 0; c < CPT; ++c) {
+                    s[2 * j][c] = bw::fma2(a.x, s[2 * j][c], bw::mul2(k.x, v[c]));
+                    s[2 * j + 1][c] = bw::fma2(a.y, s[2 * j + 1][c], bw::mul2(k.y, v[c]));
+                    acc[c] = bw::fma2(s[2 * j][c], q.x, acc[c]);
+                    acc[c] = bw::fma2(s[2 * j + 1][c], q.y, acc[c]);
+                }
             }
-            // lanes 0..15 go on with columns 0 and 1, lanes 16..31 with 2 and 3; then by bit 3 one column each
-            const float g0 = __shfl_xor_sync(0xffffffffu, hi16 ? acc[0] : acc[2], 16);
-            const float g1 = __shfl_xor_sync(0xffffffffu, hi16 ? acc[1] : acc[3], 16);
-            const float b0 = (hi16 ? acc[2] : acc[0]) + g0, b1 = (hi16 ? acc[3] : acc[1]) + g1;
-            float sum = (hi8 ? b1 : b0) + __shfl_xor_sync(0xffffffffu, hi8 ? b0 : b1, 8);
-            sum += __shfl_xor_sync(0xffffffffu, sum, 4);
-            sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-            sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-            if ((lane & 7) == 0 && my_col < p.dv) p.o[(size_t)(tb + tt) * p.heads * p.dv + h * p.dv + my_col] = sum;
+            float sum;
+            if constexpr (CPT == 4) sum = bw::tile_sum4(bw::sum2(acc[0]), bw::sum2(acc[1]), bw::sum2(acc[2]), bw::sum2(acc[3]));
+            else sum = bw::tile_sum2(bw::sum2(acc[0]), bw::sum2(acc[1]));
+            if (mine) part[(tt * NW + warp) * COLS + my_col] = sum;
+        }
+        __syncthreads();
+        for (int idx = threadIdx.x; idx < n * COLS; idx += THREADS) {
+            const int tt = idx / COLS, cc = idx % COLS;
+            float o = 0.f;
+#pragma unroll
+            for (int w = 0; w < NW; ++w) o += part[(tt * NW + w) * COLS + cc];
+            if (c0 + cc < p.dv) p.o[(size_t)(tb + tt) * p.heads * p.dv + h * p.dv + c0 + cc] = o;
         }
     }
-#pragma unroll
-    for (int j = 0; j < RPL; ++j) {
-        const int i = ((j >> 2) * 32 + lane) * 4 + (j & 3);
-        if (vec_state) {
-            if (i < p.dk) *reinterpret_cast<float4*>(S + (size_t)i * p.sld + cbase) = make_float4(s[j][0], s[j][1], s[j][2], s[j][3]);
-        } else {
-#pragma unroll
-            for (int cc = 0; cc < CPT; ++cc)
-                if (i < p.dk && cbase + cc < p.dv) S[(size_t)i * p.sld + cbase + cc] = s[j][cc];
-        }
-    }
+    bw::tile_store<CPT>(s, S, row0, p.dk, p.sld, c0 + cg * CPT, p.dv);
+}
+
+template <int NW, int CPT, bool MEM>
+int launch_scan(const ScanParams& p, int R, cudaStream_t s) {
+    constexpr int smem = ScanSmem<NW, CPT, MEM>::floats * (int)sizeof(float), COLS = bw::TILE_CG * CPT;
+    static bool raised[bw::MAX_DEVICES] = {};
+    if (smem > 48 * 1024)
+        if (bw::allow_dynamic_smem(gla_scan_kernel<NW, CPT, MEM>, smem, raised) != cudaSuccess) return BW_ERR_DRIVER;
+    bw::launch((gla_scan_kernel<NW, CPT, MEM>), dim3(R, p.heads, (p.dv + COLS - 1) / COLS), dim3(32 * NW), smem, s, p);
+    BW_LAUNCH_CHECK();
+    return 0;
+}
+
+// few blocks: narrower ones, so that more SMs work
+inline bool scan_narrow(int R, int heads, int dv) { return (long long)R * heads * ((dv + 31) / 32) < (long long)bw::num_sms() * SCAN_NARROW_BELOW / 4; }
+
+template <int NW, bool MEM>
+int launch_scan_any(const ScanParams& p, int R, cudaStream_t s) {
+    return scan_narrow(R, p.heads, p.dv) ? launch_scan<NW, 2, MEM>(p, R, s) : launch_scan<NW, 4, MEM>(p, R, s);
 }
 
 // one warp per (token, head): o / sqrt(mean(o^2) + eps) * gain[c] * silu(g[c])
@@ -242,7 +257,7 @@ gla_gate_kernel(const float* __restrict__ o, const float* __restrict__ g, long l
 
 // decay: float32 [T, heads * dk] from bw_gla_decay; with scalar_decay [T, heads].  k_scale: float32 [T, heads] or null.
 // ones_col != 0: dv counts a last column of ones that v does not hold (state [slots, heads, dk, state_ld], o [T, heads * dv]).
-// state_ld: floats between the state's rows (0: dv); with a multiple of 4 a lane moves its columns of a row in one access.
+// state_ld: floats between the state's rows (0: dv); columns from dv on stay zero.
 // qk_rep: head h uses query/key head h / qk_rep (1: every head has its own).
 BW_EXPORT int bw_gla_scan(const float* qkv, long long ld, int q_off, int k_off, int v_off, const float* decay,
                           const int* cu_q, const int* state_slot, float* state, float* o, int R, int heads, int dk,
@@ -259,26 +274,13 @@ BW_EXPORT int bw_gla_scan(const float* qkv, long long ld, int q_off, int k_off, 
     p.q_scale = q_scale;
     p.k_scale = k_scale; p.scalar_decay = scalar_decay; p.ones_col = ones_col; p.sld = state_ld ? state_ld : dv;
     p.rep = qk_rep;
-    const dim3 grid(R, heads, (dv + COLS - 1) / COLS);
-    const int rpl = dk <= 128 ? 4 : 8;
-    const size_t smem = (size_t)(3 * TOK_CHUNK * 32 * rpl + TOK_CHUNK * COLS) * sizeof(float);
     cudaStream_t s = (cudaStream_t)stream;
     const bool mem = k_scale || scalar_decay || ones_col || qk_rep > 1;
-    if (rpl == 4) {
-        if (mem) bw::launch((gla_scan_kernel<4, true>), grid, dim3(THREADS), smem, s, p);
-        else bw::launch((gla_scan_kernel<4, false>), grid, dim3(THREADS), smem, s, p);
-    } else {
-        static bool raised[bw::MAX_DEVICES] = {}, raised_mem[bw::MAX_DEVICES] = {};
-        if (mem) {
-            if (bw::allow_dynamic_smem(gla_scan_kernel<8, true>, (int)smem, raised_mem) != cudaSuccess) return BW_ERR_DRIVER;
-            bw::launch((gla_scan_kernel<8, true>), grid, dim3(THREADS), smem, s, p);
-        } else {
-            if (bw::allow_dynamic_smem(gla_scan_kernel<8, false>, (int)smem, raised) != cudaSuccess) return BW_ERR_DRIVER;
-            bw::launch((gla_scan_kernel<8, false>), grid, dim3(THREADS), smem, s, p);
-        }
-    }
-    BW_LAUNCH_CHECK();
-    return 0;
+    if (mem && !scalar_decay) return BW_ERR_UNSUPPORTED;     // the memory's form has one decay per head
+    if (dk <= 32) return mem ? launch_scan_any<1, true>(p, R, s) : launch_scan_any<1, false>(p, R, s);
+    if (dk <= 64) return mem ? launch_scan_any<2, true>(p, R, s) : launch_scan_any<2, false>(p, R, s);
+    if (dk <= 128) return mem ? launch_scan_any<4, true>(p, R, s) : launch_scan_any<4, false>(p, R, s);
+    return mem ? launch_scan_any<8, true>(p, R, s) : launch_scan_any<8, false>(p, R, s);
 }
 
 // x: float32 [T, ldx], the decay's first projection at column x_off; w [C, rank] and b [C] of w_type.

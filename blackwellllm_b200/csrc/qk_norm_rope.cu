@@ -94,6 +94,9 @@ __device__ __forceinline__ void put4(bf16* p, float4 v) {
     *reinterpret_cast<uint2*>(p) = make_uint2(bw::pack_bf16x2(v.x, v.y), bw::pack_bf16x2(v.z, v.w));
 }
 
+__device__ __forceinline__ void put2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void put2(bf16* p, float a, float b) { *reinterpret_cast<uint32_t*>(p) = bw::pack_bf16x2(a, b); }
+
 // The same with the norm taken per HEAD: every query head of dq channels is divided by its own root mean
 // square and multiplied by q_gain [dq], one gain vector shared by all heads (k_gain [dq] for the key heads);
 // a null gain: no norm on that side.  After norm and rotation the queries of a token at position p are
@@ -114,7 +117,7 @@ head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __
                       const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps,
                       float q_coef, float q_every,
                       OT* __restrict__ q_out, OT* __restrict__ k_pages, OT* __restrict__ v_pages,
-                      int nh, int nkv, int dq, int dv, int dpad, int page_size, int num_pages, int has_kv, int vec,
+                      int nh, int nkv, int dq, int dv, int dpad, int page_size, int num_pages, int has_kv, int vec, int vec2, int vec_v,
                       float v_eps, const float* __restrict__ v_first, long long v_first_ld, const float* __restrict__ v_lam,
                       const float* __restrict__ q_head_mult, int v_col, float v_scale) {
     BW_PDL_TRIGGER();
@@ -141,7 +144,7 @@ head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __
         const float* src = is_q ? row + (size_t)h * dq : row + nq + (size_t)(h - nh) * dq;
         const float* gain = is_q ? q_gain : k_gain;
         float r = 1.f;
-        if (gain) {
+        if (gain && !vec2) {
             float ss = 0.f;
             for (int c = lane; c < dq; c += 32) { const float v = src[c]; ss = fmaf(v, v, ss); }
             r = rsqrtf(bw::warp_sum(ss) / (float)dq + eps);
@@ -159,6 +162,47 @@ head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __
                     o.x = o.x * r * g.x * mult; o.y = o.y * r * g.y * mult; o.z = o.z * r * g.z * mult; o.w = o.w * r * g.w * mult;
                 }
                 put4(dst + c, o);
+            }
+            continue;
+        }
+        if (vec2) {
+            // rotation of halves, even sizes up to 256, aligned rows: a lane keeps pairs of neighbouring channels and their
+            // partners in registers, so a head is read once
+            float2 a[2], b[2], q[4];
+            float ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const int c = i * 64 + lane * 2;
+                a[i] = b[i] = make_float2(0.f, 0.f);
+                if (c < half) { a[i] = *reinterpret_cast<const float2*>(src + c); b[i] = *reinterpret_cast<const float2*>(src + half + c); }
+                ss = fmaf(a[i].x, a[i].x, ss); ss = fmaf(a[i].y, a[i].y, ss); ss = fmaf(b[i].x, b[i].x, ss); ss = fmaf(b[i].y, b[i].y, ss);
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {        // channels that pass, then the padding
+                const int c = rotary_dim + i * 64 + lane * 2;
+                q[i] = c < dq ? *reinterpret_cast<const float2*>(src + c) : make_float2(0.f, 0.f);
+                ss = fmaf(q[i].x, q[i].x, ss); ss = fmaf(q[i].y, q[i].y, ss);
+            }
+            const float r2 = (gain ? rsqrtf(bw::warp_sum(ss) / (float)dq + eps) : 1.f) * mult;
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const int c = i * 64 + lane * 2;
+                if (c < half) {
+                    const float2 ga = gain ? *reinterpret_cast<const float2*>(gain + c) : make_float2(1.f, 1.f);
+                    const float2 gb = gain ? *reinterpret_cast<const float2*>(gain + half + c) : make_float2(1.f, 1.f);
+                    const float2 cs = *reinterpret_cast<const float2*>(tab + c), sn = *reinterpret_cast<const float2*>(tab + half + c);
+                    const float x0 = a[i].x * r2 * ga.x, x1 = a[i].y * r2 * ga.y, y0 = b[i].x * r2 * gb.x, y1 = b[i].y * r2 * gb.y;
+                    put2(dst + c, x0 * cs.x - y0 * sn.x, x1 * cs.y - y1 * sn.y);
+                    put2(dst + half + c, y0 * cs.x + x0 * sn.x, y1 * cs.y + x1 * sn.y);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int c = rotary_dim + i * 64 + lane * 2;
+                if (c < dpad) {
+                    const float2 g = (gain && c < dq) ? *reinterpret_cast<const float2*>(gain + c) : make_float2(1.f, 1.f);
+                    put2(dst + c, q[i].x * r2 * g.x, q[i].y * r2 * g.y);
+                }
             }
             continue;
         }
@@ -199,7 +243,7 @@ head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __
         return;
     }
     if (page >= 0) {
-        if (vec && !vf) {
+        if (vec_v && !vf) {
             for (int idx = threadIdx.x * 4; idx < nkv * dpad; idx += blockDim.x * 4) {
                 const int h = idx / dpad, c = idx - h * dpad;
                 float4 o = c < dv ? *reinterpret_cast<const float4*>(vsrc + (size_t)h * dv + c) : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -241,10 +285,17 @@ BW_EXPORT int bw_head_norm_rope_append(const float* qkv, long long ld, const int
     cudaStream_t s = (cudaStream_t)stream;
     const int vec = rotary_dim == 0 && (dq & 3) == 0 && (dv & 3) == 0 && (dpad & 3) == 0 && (ld & 3) == 0 &&
                     (((uintptr_t)qkv | (uintptr_t)q_gain | (uintptr_t)k_gain | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages) & 15) == 0;
+    const int v_col = kv_shared ? nh * dq : nh * dq + nkv * dq;
+    // the rotated form two channels at a time; the values four at a time
+    const int vec2 = rotary_dim > 0 && !interleaved && (rotary_dim & 3) == 0 && (dq & 1) == 0 && (dpad & 1) == 0 && dpad <= 256 &&
+                     (ld & 1) == 0 && (((uintptr_t)qkv | (uintptr_t)q_gain | (uintptr_t)k_gain | (uintptr_t)table | (uintptr_t)q_out |
+                                        (uintptr_t)k_pages) & 7) == 0;
+    const int vec_v = (dv & 3) == 0 && (dpad & 3) == 0 && (ld & 3) == 0 && (v_col & 3) == 0 &&
+                      (((uintptr_t)qkv | (uintptr_t)v_pages) & 15) == 0;
 #define BW_HN(OT) bw::launch((head_norm_rope_kernel<OT>), dim3(T), dim3(256), 0, s, qkv, ld, positions, req_of_token, block_table, \
         max_blocks, table, rotary_dim, interleaved, q_gain, k_gain, eps, q_coef, q_every, (OT*)q_out, (OT*)k_pages, (OT*)v_pages, \
-        nh, nkv, dq, dv, dpad, page_size, num_pages, has_kv, vec, v_eps, v_first, v_first_ld, v_lam, \
-        q_head_mult, kv_shared ? nh * dq : nh * dq + nkv * dq, v_scale)
+        nh, nkv, dq, dv, dpad, page_size, num_pages, has_kv, vec, vec2, vec_v, v_eps, v_first, v_first_ld, v_lam, \
+        q_head_mult, v_col, v_scale)
     if (out_type == BW_F32) BW_HN(float);
     else if (out_type == BW_BF16) BW_HN(bf16);
     else return BW_ERR_BAD_ARG;

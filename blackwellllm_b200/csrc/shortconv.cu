@@ -52,17 +52,22 @@ constexpr int WARPS = 8;
 __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
 
+// TAPS > 0: the number of columns at compile time (all loads of a token in flight at once); 0: p.taps
+template <int TAPS>
 __device__ __forceinline__ float conv_at(const ConvParams& p, int t, int local, int pos, const float* st, int c) {
+    const int taps = TAPS > 0 ? TAPS : p.taps;
     float acc = p.bias ? p.bias[c] : 0.f;
-    for (int j = p.taps - 1; j >= 0; --j) {          // j tokens back, the oldest first
+#pragma unroll
+    for (int j = taps - 1; j >= 0; --j) {            // j tokens back, the oldest first
         if (j > pos) continue;                        // before the sequence's start
-        const float v = j <= local ? p.x[(size_t)(t - j) * p.ld + c] : st[(size_t)((pos - j) % p.taps) * p.C + c];
-        acc = fmaf(p.w[(size_t)(p.taps - 1 - j) * p.C + c], v, acc);
+        const float v = j <= local ? p.x[(size_t)(t - j) * p.ld + c] : st[(size_t)((pos - j) % taps) * p.C + c];
+        acc = fmaf(p.w[(size_t)(taps - 1 - j) * p.C + c], v, acc);
     }
     return acc;
 }
 
-template <int NR>   // registers a lane holds of a normed head: heads of up to 32 * NR channels
+// NR: channels a lane holds of a piece (pieces of up to 32 * NR channels)
+template <int NR, int TAPS>
 __global__ void __launch_bounds__(32 * WARPS)
 short_conv_kernel(ConvParams p) {
     BW_PDL_TRIGGER();
@@ -89,31 +94,67 @@ short_conv_kernel(ConvParams p) {
     const Seg sg = p.seg[s];
     const int first = sg.c0 + item * sg.size;
     const int n = min(sg.size, sg.channels - item * sg.size);
+    const int r0 = p.req_of_token[t0], local0 = t0 - p.cu_q[r0];
+    if (TAPS > 0 && t1 - t0 == TILE && local0 >= TAPS - 1 && t0 + TILE <= p.cu_q[r0 + 1]) {
+        // the whole tile and the tokens before it belong to one portion: every row is read once, all loads side by side
+        float u[TILE][NR];
+#pragma unroll
+        for (int k = 0; k < NR; ++k) {
+            const int c = first + k * 32 + lane;
+            const bool in = k * 32 + lane < n;
+            float v[TILE + TAPS - 1], w[TAPS > 0 ? TAPS : 1];
+            const float* src = p.x + (size_t)(t0 - (TAPS - 1)) * p.ld + c;
+#pragma unroll
+            for (int j = 0; j < TILE + TAPS - 1; ++j) v[j] = in ? src[(size_t)j * p.ld] : 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) w[j] = in ? p.w[(size_t)j * p.C + c] : 0.f;
+            const float b = (in && p.bias) ? p.bias[c] : 0.f;
+#pragma unroll
+            for (int i = 0; i < TILE; ++i) {
+                float acc = b;
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j], v[i + j], acc);
+                u[i][k] = silu(acc);
+            }
+        }
+        float f[TILE];
+#pragma unroll
+        for (int i = 0; i < TILE; ++i) {
+            f[i] = 1.f;
+            if (sg.unit) {
+                float ss = 0.f;
+#pragma unroll
+                for (int k = 0; k < NR; ++k) ss = fmaf(u[i][k], u[i][k], ss);
+                f[i] = sg.scale * rsqrtf(bw::warp_sum(ss) + p.unit_eps);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < TILE; ++i)
+#pragma unroll
+            for (int k = 0; k < NR; ++k)
+                if (k * 32 + lane < n) p.out[(size_t)(t0 + i) * p.C + first + k * 32 + lane] = u[i][k] * f[i];
+        return;
+    }
     for (int t = t0; t < t1; ++t) {
         const int r = p.req_of_token[t], local = t - p.cu_q[r], pos = p.positions[t];
         float* st = p.state + (size_t)p.state_slot[r] * p.taps * p.C;
         float* dst = p.out + (size_t)t * p.C;
-        if (sg.unit) {
-            float u[NR];
-            float ss = 0.f;
+        float u[NR];
+        float ss = 0.f;
 #pragma unroll
-            for (int k = 0; k < NR; ++k) {
-                const int c = k * 32 + lane;
-                u[k] = c < n ? silu(conv_at(p, t, local, pos, st, first + c)) : 0.f;
-                ss = fmaf(u[k], u[k], ss);
-            }
-            const float f = sg.scale * rsqrtf(bw::warp_sum(ss) + p.unit_eps);
-#pragma unroll
-            for (int k = 0; k < NR; ++k) {
-                const int c = k * 32 + lane;
-                if (c < n) dst[first + c] = u[k] * f;
-            }
-        } else {
-            for (int c = lane; c < n; c += 32) dst[first + c] = silu(conv_at(p, t, local, pos, st, first + c));
+        for (int k = 0; k < NR; ++k) {
+            const int c = k * 32 + lane;
+            u[k] = c < n ? silu(conv_at<TAPS>(p, t, local, pos, st, first + c)) : 0.f;
+            ss = fmaf(u[k], u[k], ss);
         }
-        if (p.single) {
-            for (int c = lane; c < n; c += 32)
-                st[(size_t)(pos % p.taps) * p.C + first + c] = p.x[(size_t)t * p.ld + first + c];
+        const float f = sg.unit ? sg.scale * rsqrtf(bw::warp_sum(ss) + p.unit_eps) : 1.f;
+#pragma unroll
+        for (int k = 0; k < NR; ++k) {
+            const int c = k * 32 + lane;
+            if (c < n) {
+                dst[first + c] = u[k] * f;
+                if (p.single) st[(size_t)(pos % p.taps) * p.C + first + c] = p.x[(size_t)t * p.ld + first + c];
+            }
         }
     }
 }
@@ -170,8 +211,13 @@ BW_EXPORT int bw_short_conv(const float* x, long long ld, const float* w, const 
     const int tile = single ? 1 : TILE;
     const dim3 grid((T + tile - 1) / tile, (pieces + WARPS - 1) / WARPS);
     cudaStream_t s = (cudaStream_t)stream;
-    if (widest <= 128) bw::launch((short_conv_kernel<4>), grid, dim3(32 * WARPS), 0, s, p);
-    else bw::launch((short_conv_kernel<8>), grid, dim3(32 * WARPS), 0, s, p);
+#define BW_CONV(NR) switch (taps) { \
+        case 2: bw::launch((short_conv_kernel<NR, 2>), grid, dim3(32 * WARPS), 0, s, p); break; \
+        case 3: bw::launch((short_conv_kernel<NR, 3>), grid, dim3(32 * WARPS), 0, s, p); break; \
+        case 4: bw::launch((short_conv_kernel<NR, 4>), grid, dim3(32 * WARPS), 0, s, p); break; \
+        default: bw::launch((short_conv_kernel<NR, 0>), grid, dim3(32 * WARPS), 0, s, p); }
+    if (widest <= 128) { BW_CONV(4) } else { BW_CONV(8) }
+#undef BW_CONV
     BW_LAUNCH_CHECK();
     if (!single && taps > 1) {
         const int blocks = (C + 255) / 256;

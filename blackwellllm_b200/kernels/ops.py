@@ -1495,7 +1495,7 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torc
     ``scalar_decay``: ``decay`` is [T, heads]; ``k_scale`` float32 [T, heads]: the keys are multiplied by it as they are
     read; ``ones_col``: ``dv`` counts one more value column than ``proj`` holds, the constant 1, so that the state's
     last column is n <- a n + k and the output's last column n . q.  The state's rows may be longer than ``dv`` (padding that
-    stays zero): with a length that is a multiple of 4 the kernel moves a lane's columns of a row in one access.
+    stays zero).
     ``qk_rep``: ``proj`` holds ``heads / qk_rep`` query and key heads, head h uses number h / qk_rep (``scalar_decay`` only)."""
     _dev(proj, "proj", torch.float32); _dev(decay, "decay", torch.float32); _dev(state, "state", torch.float32)
     T = proj.shape[0]

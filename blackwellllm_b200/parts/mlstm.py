@@ -51,8 +51,7 @@ class MatrixLSTM(Mixer):
         self.gain = self.bias_i = self.bias_f = None
 
     def cache_request(self):
-        # [S | n] per head (rows padded to a multiple of four floats: the scan moves them in 16-byte pieces), and the
-        # running maximum m per head
+        # [S | n] per head (rows padded to a multiple of four floats), and the running maximum m per head
         return (FixedStateRequest((self.heads, self.dk, -(-(self.dv + 1) // 4) * 4), torch.float32),
                 FixedStateRequest((self.heads,), torch.float32))
 

@@ -50,7 +50,7 @@ class StateSpaceMixer(Mixer):
         self.conv = self.conv_bias = self.A = self.dt_bias = self.D = self.gain = None
 
     def cache_request(self):
-        # the state of every head (rows padded to a multiple of four floats: the scan moves them in 16-byte pieces), and
+        # the state of every head (rows padded to a multiple of four floats), and
         # the convolution's earlier inputs (position p at entry p mod taps)
         return (FixedStateRequest((self.heads, self.N, -(-self.dv // 4) * 4), torch.float32),
                 FixedStateRequest((self.taps, self.C), torch.float32))
