@@ -97,7 +97,7 @@ def sink_attention(h, w, m, eps):
     k = (h @ w["k"].T).view(T, G, d)
     v = (h @ w["v"].T).view(T, G, dv)
     q, k = rms_unit(rotate_halves(q, m["rot"]), eps), rms_unit(rotate_halves(k, m["rot"]), eps)
-    o = attend(q, k, v, m["scale"], window_mask(T, m["mask"]["size"]), sink=w["sink"])
+    o = attend(q, k, v, m["scale"], window_mask(T, (m.get("mask") or {}).get("size")), sink=w["sink"])
     return (o * torch.sigmoid(h @ w["g"].T)) @ w["o"].T
 
 
@@ -111,7 +111,7 @@ def shared_kv_attention(h, w, m, eps):
     v = k
     q, k = rms_unit(q, eps) * w["q.norm"], rms_unit(k, eps) * w["k.norm"]
     q, k = rotate_halves(q, m["rot"]), rotate_halves(k, m["rot"])
-    o = attend(q, k, v, m["scale"], window_mask(T, m["mask"]["size"]), head_factor=w["temp"])
+    o = attend(q, k, v, m["scale"], window_mask(T, (m.get("mask") or {}).get("size")), head_factor=w["temp"])
     return o @ w["o"].T
 
 
