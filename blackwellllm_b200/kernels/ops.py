@@ -1650,6 +1650,40 @@ def delta_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: tor
     return o
 
 
+CHUNK_MAX_KEY_DIM = 256
+_chunk_row = {}        # form -> floats per (token, head) of the chunked scan's scratch
+
+
+def chunk_scan(delta: bool, qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torch.Tensor, second: torch.Tensor,
+               batch, state: torch.Tensor, heads: int, qk_rep: int, dk: int, dv: int) -> torch.Tensor:
+    """The recurrences with one decay per head for portions of prompts, 32 tokens at a time with compensated tensor-core
+    products (float32 state, sums and decays; a product's error about 2^-22 of it): ``delta``: as :func:`delta_scan` with
+    beta = ``second``; else ``S <- g S + c k v^T, o = S^T q`` with c = ``second`` (as :func:`gla_scan` with ``scalar_decay``
+    and ``k_scale``).  ``decay``, ``second`` float32 [T, heads]; state [slots, heads, dk, >= dv]."""
+    _dev(qkv, "qkv", torch.float32); _dev(decay, "decay", torch.float32); _dev(second, "second", torch.float32)
+    _dev(state, "state", torch.float32)
+    T = qkv.shape[0]
+    if dk > CHUNK_MAX_KEY_DIM:
+        raise KernelError(f"chunk_scan: key size {dk} exceeds {CHUNK_MAX_KEY_DIM}")
+    if (qk_rep < 1 or heads % qk_rep or decay.shape != (T, heads) or second.shape != (T, heads) or state.dim() != 4
+            or tuple(state.shape[1:3]) != (heads, dk) or state.shape[3] < dv or T != batch.T):
+        raise KernelError("chunk_scan: decay and second [T, heads], state [slots, heads, dk, >= dv], heads a multiple of qk_rep")
+    hk = heads // qk_rep
+    if max(q_off + hk * dk, k_off + hk * dk, v_off + heads * dv) > qkv.shape[1]:
+        raise KernelError("chunk_scan: q, k or v lie outside the rows")
+    n = _chunk_row.get(bool(delta))
+    if n is None:
+        n = _chunk_row[bool(delta)] = int(_fn("chunkscan", "bw_chunk_row_floats", [c_int])(int(delta)))
+    rows = torch.empty((T, heads, n), dtype=torch.float32, device=qkv.device)
+    o = torch.empty((T, heads * dv), dtype=torch.float32, device=qkv.device)
+    fn = _fn("chunkscan", "bw_chunk_scan", [c_int, c_void_p, c_ll, c_int, c_int, c_int] + [c_void_p] * 7 + [c_int] * 7 + [c_void_p],
+             tag=("delta" if delta else "linear") if _timings is not None else None)
+    _check(fn(int(delta), _ptr(qkv), qkv.stride(0), int(q_off), int(k_off), int(v_off), _ptr(decay), _ptr(second), _ptr(batch.cu_q),
+              _ptr(batch.state_slot), _ptr(rows), _ptr(state), _ptr(o), T, batch.R, heads, int(qk_rep),
+              dk, dv, int(state.shape[3]), _stream()), "chunk_scan")
+    return o
+
+
 def ssd_out(y: torch.Tensor, x: torch.Tensor, z: torch.Tensor, D: torch.Tensor, gain: torch.Tensor, vdim: int, parts: int,
             eps: float, out_dtype: torch.dtype) -> torch.Tensor:
     """``u = (y + D x) * silu(z)`` per channel (D one number per head of ``vdim`` channels), then ``u / rms(u) * gain`` with

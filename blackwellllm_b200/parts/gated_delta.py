@@ -9,8 +9,9 @@
 Queries and keys may have fewer heads than values (head h uses number floor(h / (heads / kv_heads))).  The state S and the
 convolution's last inputs are float32, live in the request's slots of the cache manager's fixed-size state and are carried
 from step to step.  q, k, v, b, a and the output gate's projection are one matrix made at load; its results are float32.
-Three kernels follow: ``ops.short_conv`` (convolution, silu, unit norms, and the two gates), ``ops.delta_scan`` (the
-recurrence) and ``ops.gla_gate`` (head norm, gain, gate).  A constant on the output rides in the gain.  Everything but the
+Three kernels follow: ``ops.short_conv`` (convolution, silu, unit norms, and the two gates), the recurrence
+(``ops.delta_scan`` token by token in the 32-bit path and in steps of single tokens, ``ops.chunk_scan`` for portions of
+prompts) and ``ops.gla_gate`` (head norm, gain, gate).  A constant on the output rides in the gain.  Everything but the
 projections is float32.
 """
 from __future__ import annotations
@@ -90,8 +91,11 @@ class GatedDeltaRule(Mixer):
         b_off = self.C + self.V
         qkv, g, beta = ops.short_conv(proj, self.conv, None, inputs.state, batch, self.segments, UNIT_EPS,
                                       gates=(proj, b_off + self.heads, b_off, self.A, self.dt_bias))
-        o = ops.delta_scan(qkv, 0, self.K, 2 * self.K, g, beta, batch, memory.state, self.heads, self.heads // self.kv_heads,
-                           self.dk, self.dv)
+        rep = self.heads // self.kv_heads
+        if self.ctx.dtype == torch.bfloat16 and batch.T > batch.R:      # portions: a chunk of tokens at a time
+            o = ops.chunk_scan(True, qkv, 0, self.K, 2 * self.K, g, beta, batch, memory.state, self.heads, rep, self.dk, self.dv)
+        else:
+            o = ops.delta_scan(qkv, 0, self.K, 2 * self.K, g, beta, batch, memory.state, self.heads, rep, self.dk, self.dv)
         return ops.gla_gate(o, proj, self.C, self.gain, self.heads, self.dv, self.eps, self.ctx.dtype)
 
     def forward(self, x, residual, batch, cache, owns_cache: bool = True, accumulate: bool = True) -> None:

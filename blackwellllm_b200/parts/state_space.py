@@ -8,8 +8,9 @@
 
 The state S and the convolution's last inputs are float32, live in the request's slots of the cache manager's fixed-size
 state and are carried from step to step.  The projection's results are float32.  Three kernels follow: ``ops.short_conv``
-(convolution, bias, silu, and dt with its decay), ``ops.gla_scan`` (the recurrence: one decay per head, the keys B times dt
-as they are read, queries C, heads of a group sharing both) and ``ops.ssd_out`` (D x, the gate, the norm of the parts).
+(convolution, bias, silu, and dt with its decay), the recurrence with one decay per head, the keys B times dt, queries C,
+heads of a group sharing both (``ops.gla_scan`` token by token in the 32-bit path and in steps of single tokens,
+``ops.chunk_scan`` for portions of prompts) and ``ops.ssd_out`` (D x, the gate, the norm of the parts).
 Everything but the projections is float32.
 """
 from __future__ import annotations
@@ -90,8 +91,13 @@ class StateSpaceMixer(Mixer):
         state, inputs = cache
         xbc, a, dt = ops.short_conv(proj[:, self.inner:], self.conv, self.conv_bias, inputs.state, batch, self.segments,
                                     gates=(proj, self.inner + self.C, None, self.A, self.dt_bias))
-        y = ops.gla_scan(xbc, self.inner + self.GN, self.inner, 0, a, batch, state.state, self.heads, self.N, self.dv, 1.0,
-                         k_scale=dt, scalar_decay=True, qk_rep=self.heads // self.groups)
+        rep = self.heads // self.groups
+        if self.ctx.dtype == torch.bfloat16 and batch.T > batch.R:      # portions: a chunk of tokens at a time
+            y = ops.chunk_scan(False, xbc, self.inner + self.GN, self.inner, 0, a, dt, batch, state.state, self.heads, rep,
+                               self.N, self.dv)
+        else:
+            y = ops.gla_scan(xbc, self.inner + self.GN, self.inner, 0, a, batch, state.state, self.heads, self.N, self.dv, 1.0,
+                             k_scale=dt, scalar_decay=True, qk_rep=rep)
         return ops.ssd_out(y, xbc, proj, self.D, self.gain, self.dv, self.parts, self.eps, self.ctx.dtype)
 
     def forward(self, x, residual, batch, cache, owns_cache: bool = True, accumulate: bool = True) -> None:

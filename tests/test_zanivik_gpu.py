@@ -165,9 +165,11 @@ def test_short_convolution_unit_norms_and_gates(ops, taps, dims):
                 o += n
 
 
-@pytest.mark.parametrize("heads,rep,dk,dv", [(4, 2, 16, 24), (2, 1, 160, 40), (3, 3, 12, 33), (2, 1, 128, 64), (4, 4, 40, 72), (1, 1, 256, 17), (2, 2, 64, 128)])
-def test_delta_rule_across_steps_and_slots(ops, heads, rep, dk, dv):
-    """Portions of several sizes down to single tokens, slots out of order; decays that are 0 and 1, step sizes 0 and 1."""
+@pytest.mark.parametrize("chunked", [False, True])
+@pytest.mark.parametrize("heads,rep,dk,dv", [(80, 2, 36, 20), (4, 2, 16, 24), (2, 1, 160, 40), (3, 3, 12, 33), (2, 1, 128, 64), (4, 4, 40, 72), (1, 1, 256, 17), (2, 2, 64, 128)])
+def test_delta_rule_across_steps_and_slots(ops, heads, rep, dk, dv, chunked):
+    """Portions of several sizes down to single tokens, slots out of order; decays that are 0 and 1, step sizes 0 and 1;
+    token by token and in chunks of tokens."""
     lens, slots = [70, 9, 131], [2, 0, 3]
     cuts = [[33, 2, 1, 1, 20, 13], [9], [1, 1, 64, 33, 2, 30]]
     K, V = heads // rep * dk, heads * dv
@@ -188,14 +190,18 @@ def test_delta_rule_across_steps_and_slots(ops, heads, rep, dk, dv):
     for part in walk(cuts, lens):
         rows = Rows([n for _, _, n in part], [a for _, a, _ in part], [slots[r] for r, _, _ in part])
         x, g, b = (d(torch.cat([data[r][i][a:a + n] for r, a, n in part])) for i in range(3))
-        got = ops.delta_scan(x, 2, 2 + K, 2 + 2 * K, g, b, rows, state, heads, rep, dk, dv)
+        if chunked:
+            got = ops.chunk_scan(True, x, 2, 2 + K, 2 + 2 * K, g, b, rows, state, heads, rep, dk, dv)
+        else:
+            got = ops.delta_scan(x, 2, 2 + K, 2 + 2 * K, g, b, rows, state, heads, rep, dk, dv)
         o = 0
         for r, a, n in part:
             assert rel_err(got[o:o + n], want[r][a:a + n]) < 3e-5, (r, a, n)
             o += n
 
 
-def test_delta_rule_keeps_and_replaces_a_far_token(ops):
+@pytest.mark.parametrize("chunked", [False, True])
+def test_delta_rule_keeps_and_replaces_a_far_token(ops, chunked):
     """No decay, orthogonal keys: a value written 400 tokens back is read in full, unless its key was written again
     since (the second value is read) or the state was closed once in between (nothing is read)."""
     dk, dv, L = 16, 8, 420
@@ -219,16 +225,18 @@ def test_delta_rule_keeps_and_replaces_a_far_token(ops):
             state.zero_()
             at = 0
             for n in lens:
-                o = ops.delta_scan(d(x[at:at + n]), 0, dk, 2 * dk, d(g[at:at + n]), d(b[at:at + n]), Rows([n], [at], [0]), state, 1, 1, dk, dv)
+                args = (d(x[at:at + n]), 0, dk, 2 * dk, d(g[at:at + n]), d(b[at:at + n]), Rows([n], [at], [0]), state, 1, 1, dk, dv)
+                o = ops.chunk_scan(True, *args) if chunked else ops.delta_scan(*args)
                 at += n
             want = {"kept": 5.0, "replaced": -2.0, "closed": 0.0}[case]
             assert float((o[-1].cpu() - want).abs().max()) < 1e-5, (case, lens)
 
 
 @pytest.mark.parametrize("heads,groups,P,N,parts", [(4, 2, 32, 32, 2), (6, 3, 8, 24, 2), (4, 1, 20, 33, 5), (3, 3, 7, 5, 3), (4, 2, 32, 160, 1),
-                                                    (2, 2, 9, 66, 6), (8, 2, 64, 128, 8), (2, 1, 16, 256, 4)])
+                                                    (2, 2, 9, 66, 6), (8, 2, 64, 128, 8), (2, 1, 16, 256, 4), (60, 3, 48, 40, 5)])
 @pytest.mark.parametrize("out_dtype", [torch.float32, torch.bfloat16])
-def test_state_space_across_steps_and_slots(ops, heads, groups, P, N, parts, out_dtype):
+@pytest.mark.parametrize("chunked", [False, True])
+def test_state_space_across_steps_and_slots(ops, heads, groups, P, N, parts, out_dtype, chunked):
     """Scan and output kernels: heads that share a group's B and C, norm parts that cut across heads, D, the gate before
     the norm."""
     lens, slots = [70, 9, 131], [2, 0, 3]
@@ -250,7 +258,10 @@ def test_state_space_across_steps_and_slots(ops, heads, groups, P, N, parts, out
     for part in walk(cuts, lens):
         rows = Rows([n for _, _, n in part], [a for _, a, _ in part], [slots[r] for r, _, _ in part])
         x, z, a_, dt = (d(torch.cat([data[r][i][a:a + n] for r, a, n in part])) for i in range(4))
-        y = ops.gla_scan(x, I + GN, I, 0, a_, rows, state, heads, N, P, 1.0, k_scale=dt, scalar_decay=True, qk_rep=heads // groups)
+        if chunked:
+            y = ops.chunk_scan(False, x, I + GN, I, 0, a_, dt, rows, state, heads, heads // groups, N, P)
+        else:
+            y = ops.gla_scan(x, I + GN, I, 0, a_, rows, state, heads, N, P, 1.0, k_scale=dt, scalar_decay=True, qk_rep=heads // groups)
         got = ops.ssd_out(y, x, z[:, 3:], d(D), d(gain), P, parts, 1e-5, out_dtype)
         o = 0
         for r, a, n in part:
