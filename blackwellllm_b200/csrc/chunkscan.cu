@@ -42,9 +42,9 @@ struct ChunkParams {
 // ------------------------------------------------------------------ the chunks' small matrices
 // One block per (chunk, query/key head); the grid has room for as many chunks as the requests can have, blocks behind the last
 // one leave.
-template <bool DELTA>
+template <bool DELTA, int DKP>
 __global__ void __launch_bounds__(128)
-chunk_rows_kernel(ChunkParams p, int dkp) {
+chunk_rows_kernel(ChunkParams p) {
     BW_PDL_TRIGGER();
     const int hk = blockIdx.y;
     // the request that holds chunk number blockIdx.x, and the chunk's first token
@@ -71,19 +71,32 @@ chunk_rows_kernel(ChunkParams p, int dkp) {
     }
     if (t0 < 0) return;
     extern __shared__ __align__(16) float sm[];
-    const int lds = dkp + 4;
+    constexpr int lds = DKP + 4;
     float* ks = sm;                        // [C][lds]
     float* qs = ks + C * lds;              // [C][lds]
     float* kk = qs + C * lds;              // [C][C + 1] each
     float* kq = kk + C * (C + 1);
     float* Ls = kq + C * (C + 1);          // [4][C][C + 4]
     BW_PDL_WAIT();
-    for (int idx = threadIdx.x; idx < C * dkp; idx += blockDim.x) {
-        const int t = idx / dkp, i = idx - t * dkp;
-        const bool in = t < n && i < p.dk;
-        const float* src = p.qkv + (size_t)(t0 + t) * p.ld + hk * p.dk + i;
-        ks[t * lds + i] = in ? src[p.k_off] : 0.f;
-        qs[t * lds + i] = in ? src[p.q_off] : 0.f;
+    if (p.vec & 1) {
+#pragma unroll 4
+        for (int idx = threadIdx.x; idx < C * DKP / 4; idx += 128) {
+            const int t = idx / (DKP / 4), i = (idx % (DKP / 4)) * 4;
+            const bool in = t < n && i < p.dk;
+            const float* src = p.qkv + (size_t)(t0 + t) * p.ld + hk * p.dk + i;
+            const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+            *reinterpret_cast<float4*>(ks + t * lds + i) = in ? *reinterpret_cast<const float4*>(src + p.k_off) : zero;
+            *reinterpret_cast<float4*>(qs + t * lds + i) = in ? *reinterpret_cast<const float4*>(src + p.q_off) : zero;
+        }
+    } else {
+#pragma unroll 4
+        for (int idx = threadIdx.x; idx < C * DKP; idx += 128) {
+            const int t = idx / DKP, i = idx % DKP;
+            const bool in = t < n && i < p.dk;
+            const float* src = p.qkv + (size_t)(t0 + t) * p.ld + hk * p.dk + i;
+            ks[t * lds + i] = in ? src[p.k_off] : 0.f;
+            qs[t * lds + i] = in ? src[p.q_off] : 0.f;
+        }
     }
     __syncthreads();
     {
@@ -91,7 +104,7 @@ chunk_rows_kernel(ChunkParams p, int dkp) {
         float x[8], y[8];
 #pragma unroll
         for (int j = 0; j < 8; ++j) x[j] = y[j] = 0.f;
-        for (int i = 0; i < dkp; i += 4) {
+        for (int i = 0; i < DKP; i += 4) {
             const float4 kt = *reinterpret_cast<const float4*>(ks + t * lds + i), qt = *reinterpret_cast<const float4*>(qs + t * lds + i);
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
@@ -428,13 +441,12 @@ chunk_scan_kernel(ChunkParams p) {
         }
 }
 
-template <bool DELTA>
-int launch_rows(const ChunkParams& p, int dkp, cudaStream_t s) {
-    const int smem = (2 * C * (dkp + 4) + 2 * C * (C + 1) + (DELTA ? 4 * C * (C + 4) : 0)) * (int)sizeof(float);
+template <bool DELTA, int DKP>
+int launch_rows(const ChunkParams& p, cudaStream_t s) {
+    constexpr int smem = (2 * C * (DKP + 4) + 2 * C * (C + 1) + (DELTA ? 4 * C * (C + 4) : 0)) * (int)sizeof(float);
     static bool raised[bw::MAX_DEVICES] = {};
-    // (the limit for the widest keys, once)
-    if (bw::allow_dynamic_smem(chunk_rows_kernel<DELTA>, (2 * C * 260 + 2 * C * (C + 1) + 4 * C * (C + 4)) * 4, raised) != cudaSuccess) return BW_ERR_DRIVER;
-    bw::launch((chunk_rows_kernel<DELTA>), dim3(p.T / C + p.R, p.heads / p.rep), dim3(128), smem, s, p, dkp);
+    if (bw::allow_dynamic_smem(chunk_rows_kernel<DELTA, DKP>, smem, raised) != cudaSuccess) return BW_ERR_DRIVER;
+    bw::launch((chunk_rows_kernel<DELTA, DKP>), dim3(p.T / C + p.R, p.heads / p.rep), dim3(128), smem, s, p);
     BW_LAUNCH_CHECK();
     return 0;
 }
@@ -454,7 +466,9 @@ int launch_scan(const ChunkParams& p, int R, cudaStream_t s) {
 template <bool DELTA>
 int run(const ChunkParams& p, int R, cudaStream_t s) {
     const int nw = p.dk <= 32 ? 1 : (p.dk <= 64 ? 2 : (p.dk <= 128 ? 4 : 8));
-    if (const int rc = launch_rows<DELTA>(p, 32 * nw, s)) return rc;
+    const int rc = nw == 1 ? launch_rows<DELTA, 32>(p, s) : (nw == 2 ? launch_rows<DELTA, 64>(p, s)
+                 : (nw == 4 ? launch_rows<DELTA, 128>(p, s) : launch_rows<DELTA, 256>(p, s)));
+    if (rc) return rc;
     // more blocks than fit side by side: two column groups share a block, its keys and its matrices
     const bool wide = (long long)R * p.heads * ((p.dv + COLS - 1) / COLS) > (long long)bw::num_sms() * (DELTA ? 1 : 2);
     switch (nw) {

@@ -6,8 +6,8 @@
 // delta_scan_kernel walks the tokens of one request's portion in order (a single decoded token and a portion of a prompt
 // are the same case), from the state the steps before left in the request's slot, and leaves the new state there.  A block
 // owns (request, head, COLS value columns); LPC neighbouring lanes own one column, its dk state rows spread over them, in
-// registers, two rows per packed instruction.  The chain through the tokens is one product with k, a sum over LPC lanes and the update; the sum for q of
-// the token before rides in the same shuffles.  The order of all sums depends on dk alone, never on how the tokens were
+// registers, two rows per packed instruction.  The chain through the tokens is one product with k, a sum over LPC lanes and
+// the update; the sum for q of the token before rides in the same shuffles.  The order of all sums depends on dk alone, never on how the tokens were
 // cut into steps or on the batch.  Everything is float32.
 #include "common.cuh"
 
@@ -16,7 +16,6 @@ using bf16 = __nv_bfloat16;
 namespace {
 
 constexpr int THREADS = 128;
-constexpr int TOK = 16;        // tokens staged in shared memory at a time
 constexpr int MAX_DK = 256;
 
 struct DeltaParams {
@@ -30,13 +29,14 @@ struct DeltaParams {
 };
 
 // LPC lanes per column, RPL rows per lane (a multiple of 4): dk <= LPC * RPL.  Lane l of a column holds rows
-// (j * LPC + l) * 4 + e (j < RPL / 4, e < 4); in shared memory a token's q and k are padded with zeros to LPC * RPL rows.
-template <int LPC, int RPL>
+// (j * LPC + l) * 4 + e (j < RPL / 4, e < 4); in shared memory a token's q and k are padded with zeros to LPC * RPL rows.  TOK
+// tokens are staged at a time: 16, or 1 in steps of single tokens.
+template <int LPC, int RPL, int TOK>
 __global__ void __launch_bounds__(THREADS)
 delta_scan_kernel(DeltaParams p) {
     BW_PDL_TRIGGER();
     constexpr int DKP = LPC * RPL, COLS = THREADS / LPC;
-    constexpr int NST = (TOK * DKP + THREADS - 1) / THREADS, NSV = TOK * COLS / THREADS;
+    constexpr int NST = (TOK * DKP + THREADS - 1) / THREADS, NSV = (TOK * COLS + THREADS - 1) / THREADS;
     __shared__ __align__(16) float qs[TOK * DKP], ks[TOK * DKP];
     __shared__ float vs[TOK * COLS], gs[TOK], bs[TOK];
     const int r = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * COLS;
@@ -93,7 +93,10 @@ delta_scan_kernel(DeltaParams p) {
             if (TOK * DKP % THREADS == 0 || idx < TOK * DKP) { qs[idx] = rq[u]; ks[idx] = rk[u]; }
         }
 #pragma unroll
-        for (int u = 0; u < NSV; ++u) vs[threadIdx.x + u * THREADS] = rv[u];
+        for (int u = 0; u < NSV; ++u) {
+            const int idx = threadIdx.x + u * THREADS;
+            if (TOK * COLS % THREADS == 0 || idx < TOK * COLS) vs[idx] = rv[u];
+        }
         if (threadIdx.x < TOK) { gs[threadIdx.x] = rg; bs[threadIdx.x] = rb; }
         __syncthreads();
         if (tb + TOK < t1) fetch(tb + TOK, min(TOK, t1 - tb - TOK));
@@ -149,10 +152,10 @@ delta_scan_kernel(DeltaParams p) {
 }  // namespace
 
 // qkv: float32 rows `ld` apart with q and k (heads / rep heads of dk channels) and v (heads of dv) at the given columns;
-// decay, beta float32 [T, heads]; state [slots, heads, dk, dv]; o [T, heads * dv].
+// decay, beta float32 [T, heads]; state [slots, heads, dk, dv]; o [T, heads * dv].  single != 0: one token per request.
 BW_EXPORT int bw_delta_scan(const float* qkv, long long ld, int q_off, int k_off, int v_off, const float* decay,
                             const float* beta, const int* cu_q, const int* state_slot, float* state, float* o, int R,
-                            int heads, int rep, int dk, int dv, void* stream) {
+                            int heads, int rep, int dk, int dv, int single, void* stream) {
     if (R <= 0) return 0;
     if (heads <= 0 || rep <= 0 || heads % rep || dk <= 0 || dv <= 0) return BW_ERR_BAD_ARG;
     if (dk > MAX_DK) return BW_ERR_UNSUPPORTED;
@@ -160,8 +163,9 @@ BW_EXPORT int bw_delta_scan(const float* qkv, long long ld, int q_off, int k_off
     p.qkv = qkv; p.ld = ld; p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.decay = decay; p.beta = beta;
     p.cu_q = cu_q; p.state_slot = state_slot; p.state = state; p.o = o; p.heads = heads; p.rep = rep; p.dk = dk; p.dv = dv;
     cudaStream_t s = (cudaStream_t)stream;
-#define BW_DELTA(LPC, RPL) bw::launch((delta_scan_kernel<LPC, RPL>), dim3(R, heads, (dv + THREADS / LPC - 1) / (THREADS / LPC)), \
-                                      dim3(THREADS), 0, s, p)
+#define BW_DELTA(LPC, RPL) do { const dim3 grid(R, heads, (dv + THREADS / LPC - 1) / (THREADS / LPC)); \
+        if (single) bw::launch((delta_scan_kernel<LPC, RPL, 1>), grid, dim3(THREADS), 0, s, p); \
+        else bw::launch((delta_scan_kernel<LPC, RPL, 16>), grid, dim3(THREADS), 0, s, p); } while (0)
     if (dk <= 32) BW_DELTA(8, 4);
     else if (dk <= 64) BW_DELTA(8, 8);
     else if (dk <= 128) BW_DELTA(8, 16);

@@ -64,6 +64,8 @@ struct RopeOut {
     int nh, nkv, hd, rd, page_size;
 };
 
+enum { BOX_NONE = 0, BOX_ADD = 1, BOX_F32 = 2, BOX_BF16 = 3 };
+
 struct Epilogue {
     void* out;            // [tokens, features] (SwiGLU: [tokens, features / 2]), row stride ldo (elements)
     float* partial;       // split-K: [splits, tokens, features] dense float32; else null
@@ -73,7 +75,9 @@ struct Epilogue {
     int out_type, bias_type, accumulate, transposed, swiglu;
     int tokens, features, splits;
     int rope_on;
-    int tma_add;          // normal orientation, out += : 32 x 32 boxes go out through the tensor map tmC
+    // normal orientation: 32 x 32 boxes go out through the tensor map tmC.  BOX_ADD: out += (float32); BOX_F32, BOX_BF16: out =
+    // (after bias and activation), float32 or bfloat16
+    int tma_add;
     int stream;           // the k-blocks of all tiles, laid end to end, are cut into one equal range per CTA
     int planes;           // split-K: the partial planes ARE the result (the bias in plane 0); whoever reads them adds them up
     // an activation of common.cuh on the finished sums.  With swiglu: the gated one that replaces silu(g) * u
@@ -347,6 +351,50 @@ __device__ __forceinline__ void load_bias32(const Epilogue& ep, int f0, int limi
     }
 }
 
+// A chunk of 32 features from f0 on of the lane's token on its way out through the tensor map (ep.tma_add): bias, activation,
+// the lane's row of the box in shared memory (swizzled as the map says: 128-byte rows of float32, 64-byte rows of bfloat16),
+// then one TMA operation per warp.  `width`: features from f0 to the tile's end (columns behind it go out as zeros; a result
+// that is written, not added, has tiles of whole chunks).  Rows and columns past the matrix are clipped.
+__device__ __forceinline__ void box_out(const Epilogue& ep, const CUtensorMap* map, uint32_t (&v)[32], uint8_t* box, int f0, int width,
+                                        int limit, int row0, int lane) {
+    if (lane == 0) bw::bulk_wait_group_read<1>();   // the box used two chunks ago has been read
+    __syncwarp();
+    if (ep.bias) {
+        float b[32];
+        load_bias32(ep, f0, limit, b);
+#pragma unroll
+        for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) + b[i]);
+    }
+    if (ep.act) {
+#pragma unroll
+        for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(ep_unary(ep, __uint_as_float(v[i])));
+    }
+    if (ep.tma_add == BOX_BF16) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            uint32_t w[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) w[i] = bw::pack_bf16x2(__uint_as_float(v[8 * j + 2 * i]), __uint_as_float(v[8 * j + 2 * i + 1]));
+            *reinterpret_cast<uint4*>(box + lane * 64 + ((j ^ ((lane >> 1) & 3)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
+        }
+    } else {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            uint4 q4;
+            q4.x = 4 * j + 0 < width ? v[4 * j + 0] : 0u; q4.y = 4 * j + 1 < width ? v[4 * j + 1] : 0u;
+            q4.z = 4 * j + 2 < width ? v[4 * j + 2] : 0u; q4.w = 4 * j + 3 < width ? v[4 * j + 3] : 0u;
+            *reinterpret_cast<uint4*>(box + lane * 128 + ((j ^ (lane & 7)) << 4)) = q4;
+        }
+    }
+    bw::fence_proxy_async_smem();
+    __syncwarp();
+    if (lane == 0) {
+        if (ep.tma_add == BOX_ADD) bw::tma_reduce_add_2d(map, bw::smem_u32(box), f0, row0);
+        else bw::tma_store_2d(map, bw::smem_u32(box), f0, row0);
+        bw::bulk_commit_group();
+    }
+}
+
 // SwiGLU epilogue in the normal orientation: the thread holds 32 consecutive features f0 .. f0 + 31 of
 // ONE token, f0 a multiple of 32: 16 gate sums, then the 16 up sums of the same output features.
 // It writes silu(gate) * up for those 16 features as 32 contiguous bytes.
@@ -609,33 +657,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                     emit<CH, ROPE>(ep, part, vals, token0, min(CH, b_rows - token0), ga, ga < a_rows);
                 } else if (ep.tma_add) {
                     if constexpr (CH == 32 && !ROPE) {
-                        // out += tile: the lane's row of 32 sums goes to a 128-byte-swizzled box in shared
-                        // memory, the TMA unit adds the box into out (rows and columns past the matrix are
-                        // clipped; columns past this tile's width are sent as zeros).  Two boxes per warp,
-                        // so filling one overlaps the other's way out.
-                        const int chunk = c0 / 32;
-                        uint8_t* box = (uint8_t*)staging + ((warp - 2) * 2 + (chunk & 1)) * 4096;
-                        if (lane == 0) bw::bulk_wait_group_read<1>();   // the box used two chunks ago has been read
-                        __syncwarp();
-                        if (ep.bias) {
-                            float b[32];
-                            load_bias32(ep, tile_b * BN + c0, b_rows, b);
-#pragma unroll
-                            for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) + b[i]);
-                        }
-#pragma unroll
-                        for (int j = 0; j < 8; ++j) {
-                            uint4 q4;
-                            q4.x = c0 + 4 * j + 0 < BN ? v[4 * j + 0] : 0u; q4.y = c0 + 4 * j + 1 < BN ? v[4 * j + 1] : 0u;
-                            q4.z = c0 + 4 * j + 2 < BN ? v[4 * j + 2] : 0u; q4.w = c0 + 4 * j + 3 < BN ? v[4 * j + 3] : 0u;
-                            *reinterpret_cast<uint4*>(box + lane * 128 + ((j ^ (lane & 7)) << 4)) = q4;
-                        }
-                        bw::fence_proxy_async_smem();
-                        __syncwarp();
-                        if (lane == 0) {
-                            bw::tma_reduce_add_2d(&tmC, bw::smem_u32(box), tile_b * BN + c0, tile_a * BM + quarter * 32);
-                            bw::bulk_commit_group();
-                        }
+                        // the TMA unit takes the tile out (adds it into out, or writes it), a box of 32 x 32 at a time.  Two
+                        // boxes per warp, so filling one overlaps the other's way out.
+                        uint8_t* box = (uint8_t*)staging + ((warp - 2) * 2 + ((c0 / 32) & 1)) * 4096;
+                        box_out(ep, &tmC, v, box, tile_b * BN + c0, BN - c0, b_rows, tile_a * BM + quarter * 32, lane);
                     }
                 } else if (ep.swiglu && !part) {
                     if constexpr (CH == 32 && !ROPE) {
@@ -889,28 +914,8 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
                     }
                 } else if (ep.tma_add) {
                     if constexpr (!ROPE) {
-                        const int chunk = c0 / 32;
-                        uint8_t* box = (uint8_t*)staging + ((warp - 2) * 2 + (chunk & 1)) * 4096;
-                        if (lane == 0) bw::bulk_wait_group_read<1>();
-                        __syncwarp();
-                        if (ep.bias) {
-                            float b[32];
-                            load_bias32(ep, tile_b * BN + c0, b_rows, b);
-#pragma unroll
-                            for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) + b[i]);
-                        }
-#pragma unroll
-                        for (int j = 0; j < 8; ++j) {   // columns past this tile's width go out as zeros
-                            const bool in = c0 + 4 * j < BN;   // BN is a multiple of 16: whole groups of four
-                            *reinterpret_cast<uint4*>(box + lane * 128 + ((j ^ (lane & 7)) << 4)) =
-                                in ? make_uint4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]) : make_uint4(0u, 0u, 0u, 0u);
-                        }
-                        bw::fence_proxy_async_smem();
-                        __syncwarp();
-                        if (lane == 0) {
-                            bw::tma_reduce_add_2d(&tmC, bw::smem_u32(box), tile_b * BN + c0, row0);
-                            bw::bulk_commit_group();
-                        }
+                        uint8_t* box = (uint8_t*)staging + ((warp - 2) * 2 + ((c0 / 32) & 1)) * 4096;
+                        box_out(ep, &tmC, v, box, tile_b * BN + c0, BN - c0, b_rows, row0, lane);
                     }
                 } else if (ROPE) {
                     if constexpr (ROPE) {
@@ -1077,17 +1082,17 @@ int launch_pair(const CUtensorMap& a, const CUtensorMap& b, const CUtensorMap& c
     return 0;
 }
 
-// float32 [rows, cols] with row stride ld (elements), box = 32 x 32, 128-byte swizzle: the epilogue's
-// way out for out += product
-bool make_out_map(CUtensorMap* m, void* base, long long rows, long long cols, long long ld) {
+// float32 or bfloat16 [rows, cols] with row stride ld (elements), box = 32 x 32, rows of the box swizzled over their 128 or 64
+// bytes: the epilogue's way out for whole boxes
+bool make_out_map(CUtensorMap* m, void* base, long long rows, long long cols, long long ld, bool f32) {
     EncodeTiledFn fn = encode_fn();
     if (!fn) return false;
     cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-    cuuint64_t strides[1] = {(cuuint64_t)ld * 4};
+    cuuint64_t strides[1] = {(cuuint64_t)ld * (f32 ? 4 : 2)};
     cuuint32_t box[2] = {32, 32};
     cuuint32_t estr[2] = {1, 1};
-    return fn(m, CU_TENSOR_MAP_DATA_TYPE_FLOAT32, 2, base, dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-              CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_NONE, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+    return fn(m, f32 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT32 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, base, dims, strides, box, estr,
+              CU_TENSOR_MAP_INTERLEAVE_NONE, f32 ? CU_TENSOR_MAP_SWIZZLE_128B : CU_TENSOR_MAP_SWIZZLE_64B, CU_TENSOR_MAP_L2_PROMOTION_NONE, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
 int ceil_div(long long a, long long b) { return (int)((a + b - 1) / b); }
@@ -1275,13 +1280,15 @@ static int run_gemm_tc(const void* x, const void* w, const void* bias, int bias_
     ep.rope_on = rope ? 1 : 0;
     ep.stream = stream_k ? 1 : 0;
     if (rope) ep.rope = *rope; else ep.rope = RopeOut{};
-    // out += product with many tokens and no split: the epilogue hands 32 x 32 boxes to the TMA unit
+    // many tokens and no split: the epilogue hands 32 x 32 boxes to the TMA unit
     CUtensorMap tc;
     std::memset(&tc, 0, sizeof(tc));
-    ep.tma_add = 0;
-    if (!tr && accumulate && splits == 1 && !rope && !swiglu && ((uintptr_t)out & 15) == 0 && ldo % 4 == 0) {
-        if (!make_out_map(&tc, out, M, N, ldo)) return BW_ERR_DRIVER;
-        ep.tma_add = 1;
+    ep.tma_add = BOX_NONE;
+    if (!tr && splits == 1 && !rope && !swiglu && !planes && ((uintptr_t)out & 15) == 0 && ldo % (out_type == BW_F32 ? 4 : 8) == 0) {
+        // (boxes that are written need tiles of whole boxes: 240 columns are seven and a half)
+        if (accumulate) ep.tma_add = BOX_ADD;
+        else if (use_pairs ? pbn % 32 == 0 : bn % 32 == 0) ep.tma_add = out_type == BW_F32 ? BOX_F32 : BOX_BF16;
+        if (ep.tma_add && !make_out_map(&tc, out, M, N, ldo, out_type == BW_F32)) return BW_ERR_DRIVER;
     }
     const int num_work = stream_k ? NUM_SMS : tiles_a * tiles_b * splits;
     int rc;

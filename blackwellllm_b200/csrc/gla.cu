@@ -11,7 +11,7 @@
 // portion of a prompt are the same case), from the state the steps before left in the request's slot,
 // and leaves the new state there.  A block owns (request, head, COLS value columns); its state lies in registers, a tile of
 // rows x columns per lane (common.cuh), two rows per packed instruction.  A token's S^T q is summed over a warp's row groups
-// by shuffles that nothing waits for, the warps' parts go to shared memory and are added, in warp order, after 16 tokens.
+// by shuffles that nothing waits for, the warps' parts go to shared memory and are added, in warp order, after a chunk of tokens.
 // The order of all sums depends on dk alone, never on how the tokens were cut into steps or on the batch.  The scan keeps
 // float32 throughout (as the design asks): it is bound by the issue of its packed multiply-adds and the shared-memory reads
 // that feed them, and its parallelism is requests x heads x columns / COLS.
@@ -28,7 +28,6 @@ namespace {
 #define SCAN_NARROW_BELOW 3     // quarters of the SM count: with fewer 32-column blocks than that they become 16 columns wide
 #endif
 constexpr int MAX_DK = 256;
-constexpr int TOK_CHUNK = 16;   // tokens staged in shared memory at a time
 
 struct ScanParams {
     const float* qkv;      // [T, ld]: q at q_off, k at k_off, v at v_off (head-major within each)
@@ -49,6 +48,7 @@ struct ScanParams {
     const float* k_scale;
     int scalar_decay, ones_col;
     int sld;               // floats between the state's rows (>= dv; columns from dv on stay zero)
+    int single;            // every request has one token
     int rep;               // head h reads query/key head h / rep (heads / rep of them; the plain form has rep == 1)
 };
 
@@ -77,20 +77,21 @@ gla_decay_kernel(const float* __restrict__ x, long long ldx, int x_off, const WT
     a[idx] = expf(log_sigmoid(z) * inv_tau);
 }
 
-// NW warps of 32 state rows: dk <= DKP = 32 NW.  CPT value columns a lane: COLS = 8 CPT.  In shared memory a token's q, k
+// NW warps of 32 state rows: dk <= DKP = 32 NW.  CPT value columns a lane: COLS = 8 CPT.  TOK_CHUNK tokens are staged in shared
+// memory at a time: 16, or 1 in steps of single tokens (fewer registers, more blocks side by side).  In shared memory a token's q, k
 // (and a) are padded with zeros to DKP channels (a padded channel stays at zero and adds nothing), so the inner loop has no
 // bounds.
 // MEM: the form for a matrix memory (ScanParams: one decay per head, keys times k_scale, the column of ones, query/key
 // heads shared by several heads); the plain form's code does not know of it.  What a fetch loads is not touched before it
 // is staged: a thread never waits for a load inside the fetch.  The key's scale multiplies the token's value instead, which is
 // the same product.
-template <int NW, int CPT, bool MEM>
+template <int NW, int CPT, bool MEM, int TOK_CHUNK>
 struct ScanSmem {
     static constexpr int DKP = NW * bw::TILE_WARP_ROWS, COLS = bw::TILE_CG * CPT;
     static constexpr int floats = (MEM ? 2 : 3) * TOK_CHUNK * DKP + TOK_CHUNK * COLS + 2 * TOK_CHUNK + TOK_CHUNK * NW * COLS;
 };
 
-template <int NW, int CPT, bool MEM>
+template <int NW, int CPT, bool MEM, int TOK_CHUNK>
 __global__ void __launch_bounds__(32 * NW)
 gla_scan_kernel(ScanParams p) {
     BW_PDL_TRIGGER();
@@ -102,7 +103,7 @@ gla_scan_kernel(ScanParams p) {
     float* vs = as + (MEM ? 0 : TOK_CHUNK * DKP);        // [TOK_CHUNK][COLS]
     float* gs = vs + TOK_CHUNK * COLS;                   // MEM: [TOK_CHUNK] decays, [TOK_CHUNK] scales of the keys
     float* part = gs + 2 * TOK_CHUNK;                    // [TOK_CHUNK][NW][COLS]
-    constexpr int NST = TOK_CHUNK * DKP / THREADS;       // staged values of q, k, a per thread
+    constexpr int NST = (TOK_CHUNK * DKP + THREADS - 1) / THREADS;       // staged values of q, k, a per thread
     constexpr int NSV = (TOK_CHUNK * COLS + THREADS - 1) / THREADS;
     const int r = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * COLS;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -209,13 +210,13 @@ gla_scan_kernel(ScanParams p) {
     bw::tile_store<CPT>(s, S, row0, p.dk, p.sld, c0 + cg * CPT, p.dv);
 }
 
-template <int NW, int CPT, bool MEM>
+template <int NW, int CPT, bool MEM, int TOK_CHUNK>
 int launch_scan(const ScanParams& p, int R, cudaStream_t s) {
-    constexpr int smem = ScanSmem<NW, CPT, MEM>::floats * (int)sizeof(float), COLS = bw::TILE_CG * CPT;
+    constexpr int smem = ScanSmem<NW, CPT, MEM, TOK_CHUNK>::floats * (int)sizeof(float), COLS = bw::TILE_CG * CPT;
     static bool raised[bw::MAX_DEVICES] = {};
     if (smem > 48 * 1024)
-        if (bw::allow_dynamic_smem(gla_scan_kernel<NW, CPT, MEM>, smem, raised) != cudaSuccess) return BW_ERR_DRIVER;
-    bw::launch((gla_scan_kernel<NW, CPT, MEM>), dim3(R, p.heads, (p.dv + COLS - 1) / COLS), dim3(32 * NW), smem, s, p);
+        if (bw::allow_dynamic_smem(gla_scan_kernel<NW, CPT, MEM, TOK_CHUNK>, smem, raised) != cudaSuccess) return BW_ERR_DRIVER;
+    bw::launch((gla_scan_kernel<NW, CPT, MEM, TOK_CHUNK>), dim3(R, p.heads, (p.dv + COLS - 1) / COLS), dim3(32 * NW), smem, s, p);
     BW_LAUNCH_CHECK();
     return 0;
 }
@@ -225,7 +226,8 @@ inline bool scan_narrow(int R, int heads, int dv) { return (long long)R * heads 
 
 template <int NW, bool MEM>
 int launch_scan_any(const ScanParams& p, int R, cudaStream_t s) {
-    return scan_narrow(R, p.heads, p.dv) ? launch_scan<NW, 2, MEM>(p, R, s) : launch_scan<NW, 4, MEM>(p, R, s);
+    if (p.single) return launch_scan<NW, 4, MEM, 1>(p, R, s);
+    return scan_narrow(R, p.heads, p.dv) ? launch_scan<NW, 2, MEM, 16>(p, R, s) : launch_scan<NW, 4, MEM, 16>(p, R, s);
 }
 
 // one warp per (token, head): o / sqrt(mean(o^2) + eps) * gain[c] * silu(g[c])
@@ -258,11 +260,11 @@ gla_gate_kernel(const float* __restrict__ o, const float* __restrict__ g, long l
 // decay: float32 [T, heads * dk] from bw_gla_decay; with scalar_decay [T, heads].  k_scale: float32 [T, heads] or null.
 // ones_col != 0: dv counts a last column of ones that v does not hold (state [slots, heads, dk, state_ld], o [T, heads * dv]).
 // state_ld: floats between the state's rows (0: dv); columns from dv on stay zero.
-// qk_rep: head h uses query/key head h / qk_rep (1: every head has its own).
+// qk_rep: head h uses query/key head h / qk_rep (1: every head has its own).  single != 0: one token per request.
 BW_EXPORT int bw_gla_scan(const float* qkv, long long ld, int q_off, int k_off, int v_off, const float* decay,
                           const int* cu_q, const int* state_slot, float* state, float* o, int R, int heads, int dk,
                           int dv, float q_scale, const float* k_scale, int scalar_decay, int ones_col, int state_ld,
-                          int qk_rep, void* stream) {
+                          int qk_rep, int single, void* stream) {
     if (R <= 0) return 0;
     if (heads <= 0 || dk <= 0 || dv <= 0 || (ones_col && dv < 2) || (state_ld != 0 && state_ld < dv) ||
         qk_rep <= 0 || heads % qk_rep)
@@ -273,7 +275,7 @@ BW_EXPORT int bw_gla_scan(const float* qkv, long long ld, int q_off, int k_off, 
     p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.heads = heads; p.dk = dk; p.dv = dv;
     p.q_scale = q_scale;
     p.k_scale = k_scale; p.scalar_decay = scalar_decay; p.ones_col = ones_col; p.sld = state_ld ? state_ld : dv;
-    p.rep = qk_rep;
+    p.rep = qk_rep; p.single = single;
     cudaStream_t s = (cudaStream_t)stream;
     const bool mem = k_scale || scalar_decay || ones_col || qk_rep > 1;
     if (mem && !scalar_decay) return BW_ERR_UNSUPPORTED;     // the memory's form has one decay per head

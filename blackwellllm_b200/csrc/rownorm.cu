@@ -55,7 +55,7 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float2* scratch) 
     return make_float2(bw::warp_sum(v.x), bw::warp_sum(v.y));
 }
 
-// a row of a sublayer's output: base (if there is one) plus its planes in order, four loads in flight
+// a row of a sublayer's output: base (if there is one) plus its planes in order, eight loads in flight
 template <int W>
 __device__ __forceinline__ void row_of(const float* base, const float* planes, long long stride, int n, size_t at, float* v) {
     if (base) ld<W>(base + at, v);
@@ -63,10 +63,10 @@ __device__ __forceinline__ void row_of(const float* base, const float* planes, l
 #pragma unroll
         for (int e = 0; e < W; ++e) v[e] = 0.f;
     }
-    for (int p0 = 0; p0 < n; p0 += 4) {
-        float t[4][W];
+    for (int p0 = 0; p0 < n; p0 += 8) {
+        float t[8][W];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
+        for (int j = 0; j < 8; ++j) {
             if (p0 + j < n) ld<W>(planes + (size_t)(p0 + j) * stride + at, t[j]);
             else {
 #pragma unroll
@@ -74,7 +74,7 @@ __device__ __forceinline__ void row_of(const float* base, const float* planes, l
             }
         }
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
+        for (int j = 0; j < 8; ++j)
 #pragma unroll
             for (int e = 0; e < W; ++e) v[e] += t[j][e];
     }
@@ -214,7 +214,8 @@ row_step_kernel(RowParams p) {
 template <typename OT, int W>
 int run(const RowParams& p, int n, cudaStream_t s) {
     const int units = (p.H + W - 1) / W;
-    const int nv = units <= 256 ? 1 : (units <= 2048 ? 2 : (units <= 4096 ? 4 : (units <= 8192 ? 8 : (units <= 16384 ? 16 : 0))));
+    // (few rows: as many loads in flight per row as can be; many rows: smaller blocks)
+    const int nv = units <= (n <= 64 ? 1024 : 256) ? 1 : (units <= 2048 ? 2 : (units <= 4096 ? 4 : (units <= 8192 ? 8 : (units <= 16384 ? 16 : 0))));
     if (!nv) return BW_ERR_UNSUPPORTED;
     const int threads = ((units + nv - 1) / nv + 31) / 32 * 32;
     switch (nv) {

@@ -73,6 +73,11 @@ __device__ __forceinline__ void tma_reduce_add_2d(const CUtensorMap* map, uint32
         "cp.reduce.async.bulk.tensor.2d.global.shared::cta.add.tile.bulk_group [%0, {%2, %3}], [%1];"
         :: "l"(map), "r"(smem_src), "r"(x), "r"(y) : "memory");
 }
+// the same box written to global memory (x * element size a multiple of 16 bytes, x and y not negative)
+__device__ __forceinline__ void tma_store_2d(const CUtensorMap* map, uint32_t smem_src, int x, int y) {
+    asm volatile("cp.async.bulk.tensor.2d.global.shared::cta.tile.bulk_group [%0, {%2, %3}], [%1];"
+                 :: "l"(map), "r"(smem_src), "r"(x), "r"(y) : "memory");
+}
 __device__ __forceinline__ void bulk_commit_group() { asm volatile("cp.async.bulk.commit_group;" ::: "memory"); }
 // waits until at most N of the thread's bulk groups still READ their shared-memory source
 template <int N> __device__ __forceinline__ void bulk_wait_group_read() {

@@ -1515,10 +1515,10 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torc
         raise KernelError("gla_scan: q, k or v lie outside the projection's columns")
     o = torch.empty((T, heads * dv), dtype=torch.float32, device=proj.device)
     fn = _fn("gla", "bw_gla_scan", [c_void_p, c_ll, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                    c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+                                    c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
     _check(fn(_ptr(proj), proj.stride(0), q_off, k_off, v_off, _ptr(decay), _ptr(batch.cu_q), _ptr(batch.state_slot),
               _ptr(state), _ptr(o), batch.R, heads, dk, dv, float(q_scale), _ptr(k_scale), int(scalar_decay),
-              int(ones_col), int(state.shape[3]), int(qk_rep), _stream()), "gla_scan")
+              int(ones_col), int(state.shape[3]), int(qk_rep), int(T == batch.R), _stream()), "gla_scan")
     return o
 
 
@@ -1644,9 +1644,9 @@ def delta_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: tor
     if max(q_off + hk * dk, k_off + hk * dk, v_off + heads * dv) > qkv.shape[1]:
         raise KernelError("delta_scan: q, k or v lie outside the rows")
     o = torch.empty((T, heads * dv), dtype=torch.float32, device=qkv.device)
-    fn = _fn("delta", "bw_delta_scan", [c_void_p, c_ll, c_int, c_int, c_int] + [c_void_p] * 6 + [c_int] * 5 + [c_void_p])
+    fn = _fn("delta", "bw_delta_scan", [c_void_p, c_ll, c_int, c_int, c_int] + [c_void_p] * 6 + [c_int] * 6 + [c_void_p])
     _check(fn(_ptr(qkv), qkv.stride(0), int(q_off), int(k_off), int(v_off), _ptr(decay), _ptr(beta), _ptr(batch.cu_q),
-              _ptr(batch.state_slot), _ptr(state), _ptr(o), batch.R, heads, int(qk_rep), dk, dv, _stream()), "delta_scan")
+              _ptr(batch.state_slot), _ptr(state), _ptr(o), batch.R, heads, int(qk_rep), dk, dv, int(T == batch.R), _stream()), "delta_scan")
     return o
 
 
