@@ -15,8 +15,8 @@
 // float32 FMAs.  chunk_scan_kernel walks the chunks of one request's portion: a block owns (request, head, 16 value columns)
 // and keeps S^T in mma accumulators, [16, 32] per warp, the warps splitting dk; only two small exchanges per chunk cross
 // warps.  State, decays and sums are float32; every product a b of the mma's is made as a_lo b_hi + a_hi b_lo + a_hi b_hi with
-// a_hi the value rounded to 11 bits of mantissa and a_lo the rest rounded likewise, which leaves an error of about 2^-22 of a
-// product (float32's own rounding is 2^-24), and the sums are float32.  The 32-bit path does not come here: it walks token by
+// a_hi the value rounded to 11 bits of mantissa and a_lo the rest, of which the tensor core reads the leading 11 bits; that leaves
+// an error of about 2^-21 of a product (float32's own rounding is 2^-24), and the sums are float32.  The 32-bit path does not come here: it walks token by
 // token (delta.cu, gla.cu), as do steps of single tokens.
 #include "common.cuh"
 

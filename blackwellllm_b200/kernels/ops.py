@@ -1657,7 +1657,7 @@ _chunk_row = {}        # form -> floats per (token, head) of the chunked scan's 
 def chunk_scan(delta: bool, qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torch.Tensor, second: torch.Tensor,
                batch, state: torch.Tensor, heads: int, qk_rep: int, dk: int, dv: int) -> torch.Tensor:
     """The recurrences with one decay per head for portions of prompts, 32 tokens at a time with compensated tensor-core
-    products (float32 state, sums and decays; a product's error about 2^-22 of it): ``delta``: as :func:`delta_scan` with
+    products (float32 state, sums and decays; a product's error about 2^-21 of it): ``delta``: as :func:`delta_scan` with
     beta = ``second``; else ``S <- g S + c k v^T, o = S^T q`` with c = ``second`` (as :func:`gla_scan` with ``scalar_decay``
     and ``k_scale``).  ``decay``, ``second`` float32 [T, heads]; state [slots, heads, dk, >= dv]."""
     _dev(qkv, "qkv", torch.float32); _dev(decay, "decay", torch.float32); _dev(second, "second", torch.float32)

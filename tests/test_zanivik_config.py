@@ -148,20 +148,20 @@ def test_specs_that_do_not_go_together():
 # ------------------------------------------------------------------ the plain implementation itself
 
 def test_plain_frequency_bands():
-    rot = {"base": 10000.0, "dims": 32, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 512}}
+    rot = {"base": 10000.0, "dims": 32, "scaling": {"factor": 6.0, "low": 1.5, "high": 5.0, "original": 700}}
     f = plain.frequencies(rot)
     plain_f = plain.frequencies({"base": 10000.0, "dims": 32})
     kept = mixed = divided = 0
     for a, b in zip(f, plain_f):
         wave = 2 * math.pi / b
-        if wave < 128:
+        if wave < 140:
             assert a == b
             kept += 1
-        elif wave > 512:
-            assert abs(a - b / 8) < 1e-15
+        elif wave > 700 / 1.5:
+            assert abs(a - b / 6) < 1e-15
             divided += 1
         else:
-            assert b / 8 < a < b
+            assert b / 6 < a < b
             mixed += 1
     assert kept and mixed and divided
 
