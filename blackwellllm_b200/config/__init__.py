@@ -9,3 +9,4 @@ from ..models import fuvevik as _fuvevik  # noqa: F401  (registers Fuvevik)
 from ..models import zigipel as _zigipel  # noqa: F401  (registers Zigipel)
 from ..models import vubotar as _vubotar  # noqa: F401  (registers Vubotar)
 from ..models import zanivik as _zanivik  # noqa: F401  (registers Zanivik)
+from ..models import zogulorn as _zogulorn  # noqa: F401  (registers Zogulorn)

@@ -88,6 +88,16 @@ class LayerNormSpec:
 
 
 @dataclass(frozen=True)
+class DynamicTanhSpec:
+    """tanh(alpha * x) * weight + bias: a norm that takes no statistic of the row.  ``alpha_param`` and ``bias_param`` are the
+    names of the number and of the vector, below the norm's prefix like ``param``, the weight's."""
+    param: str = "weight"
+    alpha_param: str = "alpha"
+    bias_param: str = "bias"
+    kind: str = "dynamic_tanh"
+
+
+@dataclass(frozen=True)
 class AttentionSpec:
     """Grouped-query softmax attention over a paged key/value cache.
 
@@ -155,6 +165,32 @@ class AttentionSpec:
     values_from_keys: bool = False
     head_temperature: bool = False
     output_scale: float = 1.0
+
+
+@dataclass(frozen=True)
+class DifferentialAttentionSpec:
+    """Softmax attention of two maps over the same values: a query head is [map 1, map 2] of ``head_dim`` channels each, a key
+    head likewise, a value head has ``v_head_dim``; with a1 and a2 the maps' outputs and ``lambda = exp(lq1 . lk1) - exp(lq2 . lk2) +
+    diff`` (tensors lq1, lk1, lq2, lk2 [head_dim]) a head returns ``rms_unit(a1 - lambda a2) * (1 - diff)``, the root mean square over
+    v_head_dim with ``norm_eps`` and no gain.  Queries, keys and values pass a causal convolution over time of ``conv_taps`` columns
+    per channel right after their projections (tensors q_conv, k_conv, v_conv; no bias, no activation); no position is encoded.
+    ``chunk``: a query sees no key before the start of its own block of positions (None: all).  ``gate_per_head``: a head's output
+    is multiplied by sigmoid(W_g x), one number per head, before the output projection.  ``shares_kv``: no keys and values of its
+    own; the run reads those of the schedule entry it names, as that entry cached them.  ``names``: (role, name) pairs for q, k, v,
+    q_conv, k_conv, v_conv, lq1, lk1, lq2, lk2, g, o."""
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    v_head_dim: int
+    conv_taps: int
+    diff: float
+    norm_eps: float
+    softmax_scale: float
+    chunk: Optional[int] = None
+    gate_per_head: bool = False
+    shares_kv: bool = False
+    kind: str = "differential_attention"
+    names: Tuple[Tuple[str, str], ...] = ()
 
 
 @dataclass(frozen=True)
@@ -229,7 +265,11 @@ class GatedDeltaSpec:
     key_dim ** -0.5; ``beta = sigmoid(W_b x)``, ``g = exp(-exp(A_log) softplus(W_a x + dt_bias))``, one of each per head.  Each
     head's o is RMS-normed over value_dim with a gain shared by the heads, multiplied by ``silu(W_g x)`` and projected.
     ``output_scale``: a constant the mixer's output is multiplied by.  ``names``: (role, name) pairs for q, k, v, b, a, g, o,
-    norm, q_conv, k_conv, v_conv, A_log, dt_bias."""
+    norm, q_conv, k_conv, v_conv, A_log, dt_bias.
+    ``channel_decay``: one decay per head and KEY CHANNEL, ``g = exp(-exp(A_log) softplus(W_a2 (W_a1 x) + dt_bias))`` laid out heads *
+    key_dim (tensors a1 [rank, hidden], a2 [heads * key_dim, rank] instead of a; dt_bias [heads * key_dim]), each acting on its row
+    of S.  ``lowrank_gate``: the output gate is ``sigmoid(W_g2 (W_g1 x))`` (tensors g1, g2 instead of g).  ``decay_rank``, ``gate_rank``:
+    the inner sizes (None: whatever the stored tensors have)."""
     num_heads: int
     num_kv_heads: int
     key_dim: int
@@ -239,6 +279,10 @@ class GatedDeltaSpec:
     output_scale: float = 1.0
     kind: str = "gated_delta"
     names: Tuple[Tuple[str, str], ...] = ()
+    channel_decay: bool = False
+    lowrank_gate: bool = False
+    decay_rank: Optional[int] = None
+    gate_rank: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -278,7 +322,8 @@ class SideBySideSpec:
 class RoutedFFNSpec:
     """Mixture of experts: ``num_experts`` gated feed-forwards ``down(silu(gate u) * (up u))`` without biases,
     of which each token uses the ``top_k`` with the largest router scores.  ``score``: "sigmoid" or
-    "softmax" of the float32 router logits; ``renormalize``: the chosen scores are divided by their sum;
+    "softmax" of the float32 router logits, or "softmax_chosen": the ``top_k`` largest logits are chosen and the weights are the
+    softmax over those alone; ``renormalize``: the chosen scores are divided by their sum;
     ``scale_input``: the score multiplies what the expert reads (u = s x) instead of what it returns."""
     num_experts: int
     top_k: int
@@ -295,7 +340,8 @@ class RoutedFFNSpec:
     # ``renorm_eps``: added to the sum that ``renormalize`` divides by.  ``activation``: the experts' gated
     # activation, "silu" (silu(g) u) or "clamped_swish" (g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit),
     # u' = clamp(u, -limit, limit)).  ``shared``: a dense gated feed-forward (a :class:`SwiGLUSpec`) that runs
-    # for every token and is added; its tensors lie below ``shared_prefix``.
+    # for every token and is added; its tensors lie below ``shared_prefix``.  ``activation`` "relu2" or "gelu": the experts
+    # have no gate, down(act(up u)) (:class:`DenseMLPSpec`), and no gate tensors.
     identity_experts: int = 0
     choice_bias: Optional[str] = None
     renorm_eps: float = 0.0
@@ -375,7 +421,8 @@ class LayerSpec:
     token_shift: Optional[str] = None
     # the "parallel" arrangement: the names of two vectors [hidden] ("layer scale"); the mixer's output is multiplied
     # channel by channel by the first and the feed-forward's by the second before they are added to the stream.  In the
-    # "sandwich" arrangement the outputs are multiplied after their second norms.  ``residual_mult`` ("sandwich"): a constant
+    # "sandwich" arrangement the outputs are multiplied after their second norms, in the "prenorm" arrangement as they are.
+    # ``residual_mult`` ("sandwich"): a constant
     # that multiplies both on top of that.
     layer_scale: Optional[Tuple[str, str]] = None
     residual_mult: float = 1.0

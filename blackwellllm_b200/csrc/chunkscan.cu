@@ -1,4 +1,4 @@
-// Recurrences with one decay per head and token, for portions of prompts, 32 tokens at a time on the tensor cores with
+// Recurrences with one decay per head and token (the delta rule also with one per key channel), for portions of prompts, 32 tokens at a time on the tensor cores with
 // compensated products.  Two forms over a state S [dk, dv] per head:
 //
 //   linear   S <- g_t S + c_t k_t v_t^T                                          o_t = S^T q_t
@@ -10,6 +10,12 @@
 //   delta:   U = T B,  B_t = beta_t (v_t - G_t S0^T k_t),  T = (I + L)^-1,  L_ts = beta_t D_ts k_s . k_t  (s < t)
 //   linear:  U = V, and c_s multiplies k_s below
 //   o_t = G_t S0^T q_t + sum_{s<=t} M_ts u_s,    M_ts = D_ts k_s . q_t           S = G S0 + sum_s R_s k_s u_s^T
+//
+// A third form is the delta rule with a decay per KEY CHANNEL, S <- diag(g_t) S in place of g_t S.  Then D_ts is a vector inside
+// the dot products, L_ts = beta_t sum_c k_s[c] D_ts[c] k_t[c] and M_ts likewise with q_t, and the walk reads ready-made rows
+// G_t o k_t, G_t o q_t (where it says G_t S0^T k_t, G_t S0^T q_t above) and R_s o k_s, with the chunk's G as a vector over the state's
+// rows.  chunk_rows_channel_kernel makes all of that, again with products of decays only: the vector D_ts o k_s is carried along
+// t in registers.
 //
 // chunk_rows_kernel makes the rows of T and M and the numbers G, R for every token and head, in parallel over the chunks, with
 // float32 FMAs.  chunk_scan_kernel walks the chunks of one request's portion: a block owns (request, head, 16 value columns)
@@ -37,7 +43,40 @@ struct ChunkParams {
     float* state; int sld;                 // [slots, heads, dk, sld]
     float* o;                              // [T, heads * dv]
     int T, R, heads, rep, dk, dv, vec;     // vec: 16-byte copies of q and k rows (1), of the values (2)
+    // the form with a decay per key channel: decay [T, heads, dk], and two more scratches
+    float* chan;                           // [T, heads, 3, dk]: G o k, G o q, R o k
+    float* gend;                           // [T / C + R, heads, dk]: the product of a chunk's decays (chunk_index)
 };
+
+// The number of request r's i-th chunk among all chunks of a step, a its first token: distinct for all chunks, below T / C + R.
+__device__ __forceinline__ int chunk_index(int r, int a, int i) { return a / C + r + i; }
+
+// The chunk of this block: its first token (< 0: none), its tokens and chunk_index; `number` counts the chunks of all requests.
+__device__ __forceinline__ void find_chunk(const ChunkParams& p, int number, int& t0, int& n, int& index) {
+    const int lane = threadIdx.x & 31;
+    t0 = -1; n = 0; index = 0;
+    for (int r0 = 0, before = 0; r0 < p.R; r0 += 32) {
+        const int r = r0 + lane;
+        const int a = r < p.R ? p.cu_q[r] : 0, len = r < p.R ? p.cu_q[r + 1] - a : 0;
+        int upto = (len + C - 1) / C;
+#pragma unroll
+        for (int d = 1; d < 32; d <<= 1) {
+            const int v = __shfl_up_sync(0xffffffffu, upto, d);
+            if (lane >= d) upto += v;
+        }
+        const unsigned has = __ballot_sync(0xffffffffu, before + upto > number);
+        if (has) {
+            const int l = __ffs(has) - 1;                  // the first request whose chunks reach past this one
+            const int first = number - (before + (l ? __shfl_sync(0xffffffffu, upto, l - 1) : 0));
+            const int start = __shfl_sync(0xffffffffu, a, l);
+            t0 = start + first * C;
+            n = min(C, __shfl_sync(0xffffffffu, a + len, l) - t0);
+            index = chunk_index(r0 + l, start, first);
+            return;
+        }
+        before += __shfl_sync(0xffffffffu, upto, 31);
+    }
+}
 
 // ------------------------------------------------------------------ the chunks' small matrices
 // One block per (chunk, query/key head); the grid has room for as many chunks as the requests can have, blocks behind the last
@@ -47,28 +86,8 @@ __global__ void __launch_bounds__(128)
 chunk_rows_kernel(ChunkParams p) {
     BW_PDL_TRIGGER();
     const int hk = blockIdx.y;
-    // the request that holds chunk number blockIdx.x, and the chunk's first token
-    int t0 = -1, n = 0;
-    for (int r0 = 0, before = 0; r0 < p.R; r0 += 32) {
-        const int r = r0 + (threadIdx.x & 31);
-        const int a = r < p.R ? p.cu_q[r] : 0, len = r < p.R ? p.cu_q[r + 1] - a : 0;
-        int upto = (len + C - 1) / C;
-#pragma unroll
-        for (int d = 1; d < 32; d <<= 1) {
-            const int v = __shfl_up_sync(0xffffffffu, upto, d);
-            if ((threadIdx.x & 31) >= d) upto += v;
-        }
-        const unsigned has = __ballot_sync(0xffffffffu, before + upto > (int)blockIdx.x);
-        if (has) {
-            const int l = __ffs(has) - 1;                  // the first request whose chunks reach past this one
-            const int first = (int)blockIdx.x - (before + (l ? __shfl_sync(0xffffffffu, upto, l - 1) : 0));
-            const int at = __shfl_sync(0xffffffffu, a, l) + first * C;
-            n = min(C, __shfl_sync(0xffffffffu, a + len, l) - at);
-            t0 = at;
-            break;
-        }
-        before += __shfl_sync(0xffffffffu, upto, 31);
-    }
+    int t0, n, index;
+    find_chunk(p, blockIdx.x, t0, n, index);
     if (t0 < 0) return;
     extern __shared__ __align__(16) float sm[];
     constexpr int lds = DKP + 4;
@@ -172,6 +191,139 @@ chunk_rows_kernel(ChunkParams p) {
     }
 }
 
+// The same for a decay per key channel.  One block per (chunk, head).  DKP: dk up to a multiple of 32.
+template <int DKP>
+__global__ void __launch_bounds__(128)
+chunk_rows_channel_kernel(ChunkParams p) {
+    BW_PDL_TRIGGER();
+    constexpr int lds = DKP + 4, CH = DKP / 8;             // channels of a lane
+    const int h = blockIdx.y, hk = h / p.rep;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    int t0, n, index;
+    find_chunk(p, blockIdx.x, t0, n, index);
+    if (t0 < 0) return;
+    extern __shared__ __align__(16) float sm[];
+    float* ks = sm;                        // [C][lds] each
+    float* qs = ks + C * lds;
+    float* gs = qs + C * lds;
+    float* kk = gs + C * lds;              // [C][C + 4]: sum_c k_s D_ts k_t, turned into L in place
+    float* kq = kk + C * (C + 4);          // [C][C + 4]
+    BW_PDL_WAIT();
+    if (p.vec & 1) {
+#pragma unroll 4
+        for (int idx = threadIdx.x; idx < C * DKP / 4; idx += 128) {
+            const int t = idx / (DKP / 4), i = (idx % (DKP / 4)) * 4;
+            const bool in = t < n && i < p.dk;
+            const float* src = p.qkv + (size_t)(t0 + t) * p.ld + hk * p.dk + i;
+            const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+            *reinterpret_cast<float4*>(ks + t * lds + i) = in ? *reinterpret_cast<const float4*>(src + p.k_off) : zero;
+            *reinterpret_cast<float4*>(qs + t * lds + i) = in ? *reinterpret_cast<const float4*>(src + p.q_off) : zero;
+            *reinterpret_cast<float4*>(gs + t * lds + i) = in ? *reinterpret_cast<const float4*>(p.decay + ((size_t)(t0 + t) * p.heads + h) * p.dk + i) : zero;
+        }
+    } else {
+#pragma unroll 4
+        for (int idx = threadIdx.x; idx < C * DKP; idx += 128) {
+            const int t = idx / DKP, i = idx % DKP;
+            const bool in = t < n && i < p.dk;
+            const float* src = p.qkv + (size_t)(t0 + t) * p.ld + hk * p.dk + i;
+            ks[t * lds + i] = in ? src[p.k_off] : 0.f;
+            qs[t * lds + i] = in ? src[p.q_off] : 0.f;
+            gs[t * lds + i] = in ? p.decay[((size_t)(t0 + t) * p.heads + h) * p.dk + i] : 0.f;
+        }
+    }
+    __syncthreads();
+    {
+        // Warp w has the tokens s = 8 w .. 8 w + 7, lane = 8 sl + cg two of them (8 w + 2 sl and + 1) on the channels
+        // (8 j + cg) 4 + e; z = D_ts o k_s goes along t, zero before s.
+        const int cg = lane & 7, s0 = 8 * warp + 2 * (lane >> 3);
+        bw::f32x2 z[2][CH / 2];
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+            for (int j = 0; j < CH / 2; ++j) z[u][j] = 0;              // (pairs of zeros)
+        for (int idx = threadIdx.x; idx < C * (C + 4); idx += 128) kk[idx] = kq[idx] = 0.f;
+        __syncthreads();
+        const ulonglong2 *k4 = reinterpret_cast<const ulonglong2*>(ks) + cg, *q4 = reinterpret_cast<const ulonglong2*>(qs) + cg,
+                         *g4 = reinterpret_cast<const ulonglong2*>(gs) + cg;
+        for (int t = 8 * warp; t < n; ++t) {
+            bw::f32x2 a[2] = {0, 0}, b[2] = {0, 0};
+            const bool near = t < 8 * warp + 8;                        // (uniform over the warp)
+#pragma unroll
+            for (int j = 0; j < CH / 4; ++j) {
+                const int at = t * (lds / 4) + 8 * j;
+                const ulonglong2 k = k4[at], q = q4[at], g = g4[at];
+#pragma unroll
+                for (int u = 0; u < 2; ++u) {
+                    z[u][2 * j] = bw::mul2(z[u][2 * j], g.x);
+                    z[u][2 * j + 1] = bw::mul2(z[u][2 * j + 1], g.y);
+                    if (near && t == s0 + u) { z[u][2 * j] = k.x; z[u][2 * j + 1] = k.y; }
+                    a[u] = bw::fma2(z[u][2 * j], k.x, a[u]);
+                    a[u] = bw::fma2(z[u][2 * j + 1], k.y, a[u]);
+                    b[u] = bw::fma2(z[u][2 * j], q.x, b[u]);
+                    b[u] = bw::fma2(z[u][2 * j + 1], q.y, b[u]);
+                }
+            }
+            // four sums over the eight lanes of a token pair: the lane ends with the one its bits 2 and 1 name
+            const float a0 = bw::sum2(a[0]), a1 = bw::sum2(a[1]), b0 = bw::sum2(b[0]), b1 = bw::sum2(b[1]);
+            const bool hi4 = lane & 4, hi2 = lane & 2;
+            const float x0 = (hi4 ? b0 : a0) + __shfl_xor_sync(0xffffffffu, hi4 ? a0 : b0, 4);
+            const float x1 = (hi4 ? b1 : a1) + __shfl_xor_sync(0xffffffffu, hi4 ? a1 : b1, 4);
+            float x = (hi2 ? x1 : x0) + __shfl_xor_sync(0xffffffffu, hi2 ? x0 : x1, 2);
+            x += __shfl_xor_sync(0xffffffffu, x, 1);
+            if (!(lane & 1)) (hi4 ? kq : kk)[t * (C + 4) + s0 + (hi2 ? 1 : 0)] = x;
+        }
+    }
+    __syncthreads();
+    if (warp == 0) {
+        float* base = p.rows + ((size_t)t0 * p.heads + h) * ROW_DELTA;
+        const size_t step = (size_t)p.heads * ROW_DELTA;
+        const float beta = lane < n ? p.second[(size_t)(t0 + lane) * p.heads + h] : 0.f;
+        for (int t = 0; t < n; ++t) {
+            const float bt = __shfl_sync(0xffffffffu, beta, t);
+            base[t * step + C + lane] = t >= lane ? kq[t * (C + 4) + lane] : 0.f;
+            kk[t * (C + 4) + lane] = t > lane ? bt * kk[t * (C + 4) + lane] : 0.f;
+        }
+        if (lane < n) {      // (the decays stand in the rows themselves: G and R are 1 here)
+            float* sc = base + lane * step + 2 * C;
+            sc[0] = 1.f; sc[1] = 1.f; sc[2] = beta; sc[3] = 0.f;
+        }
+        __syncwarp();
+        float x[C];                        // lane s: column s of T, row by row (rows of kk from n on are zeros)
+#pragma unroll
+        for (int t = 0; t < C; ++t) {
+            float u0 = t == lane ? 1.f : 0.f, u1 = 0.f;
+#pragma unroll
+            for (int j = 0; j < t; j += 4) {
+                const float4 l = *reinterpret_cast<const float4*>(kk + t * (C + 4) + j);
+                u0 = fmaf(-l.x, x[j], u0);
+                if (j + 1 < t) u1 = fmaf(-l.y, x[j + 1], u1);
+                if (j + 2 < t) u0 = fmaf(-l.z, x[j + 2], u0);
+                if (j + 3 < t) u1 = fmaf(-l.w, x[j + 3], u1);
+            }
+            x[t] = u0 + u1;
+            if (t < n) base[t * step + lane] = x[t];
+        }
+        return;
+    }
+    // meanwhile the other warps: the rows with the decays in them
+    const size_t step = (size_t)p.heads * 3 * p.dk;
+    for (int c = threadIdx.x - 32; c < p.dk; c += 96) {
+        float* dst = p.chan + ((size_t)t0 * p.heads + h) * 3 * p.dk + c;
+        float G = 1.f;
+        for (int t = 0; t < n; ++t) {
+            G *= gs[t * lds + c];
+            dst[t * step] = G * ks[t * lds + c];
+            dst[t * step + p.dk] = G * qs[t * lds + c];
+        }
+        p.gend[((size_t)index * p.heads + h) * p.dk + c] = G;
+        float R = 1.f;
+        for (int t = n - 1; t >= 0; --t) {
+            dst[t * step + 2 * p.dk] = R * ks[t * lds + c];
+            R *= gs[t * lds + c];
+        }
+    }
+}
+
 // ------------------------------------------------------------------ the walk through the chunks
 struct Split { uint32_t hi, lo; };
 __device__ __forceinline__ Split split(float x) {
@@ -220,25 +372,29 @@ __device__ __forceinline__ void copy4(float* dst, const float* src, bool in) {
 }
 
 // NW warps split dk (8 NB state rows each: dk <= DKP = 8 NB NW), MT groups of NW warps take 16 value columns each.
-template <bool DELTA, int NW, int NB, int MT>
+// CHAN: a decay per key channel (delta only).  The next chunk is fetched while this one is worked on where two fit.
+template <bool DELTA, bool CHAN, int NW, int NB, int MT>
 struct ChunkSmem {
     static constexpr int LDK = 8 * NB * NW + 4;                 // a token's q or k
     static constexpr int LDV = MT == 1 ? VS : 36;           // a token's values (twice it is 8 modulo 32)
     static constexpr int k0 = 0, q0 = k0 + C * LDK, v0 = q0 + C * LDK, m0 = v0 + C * LDV, t0 = m0 + C * TS, s0 = t0 + (DELTA ? C * TS : 0);
-    static constexpr int buffer = s0 + C * 4;
+    static constexpr int r0 = s0 + C * 4, g0 = r0 + (CHAN ? C * LDK : 0);
+    static constexpr int buffer = g0 + (CHAN ? 8 * NB * NW : 0);
     static constexpr int part = (DELTA ? 2 : 1) * COLS * TS;            // one warp's parts of S0^T q (and S0^T k)
-    static constexpr int floats = 2 * buffer + NW * MT * part + (DELTA ? MT * COLS * TS : 0);
+    static constexpr int tail = NW * MT * part + (DELTA ? MT * COLS * TS : 0);
+    static constexpr int buffers = (2 * buffer + tail) * 4 <= 227 * 1024 ? 2 : 1;
+    static constexpr int floats = buffers * buffer + tail;
 };
 
-template <bool DELTA, int NW, int NB, int MT>
+template <bool DELTA, bool CHAN, int NW, int NB, int MT>
 __global__ void __launch_bounds__(32 * NW * MT)
 chunk_scan_kernel(ChunkParams p) {
     BW_PDL_TRIGGER();
-    using L = ChunkSmem<DELTA, NW, NB, MT>;
+    using L = ChunkSmem<DELTA, CHAN, NW, NB, MT>;
     constexpr int THREADS = 32 * NW * MT, DKP = 8 * NB * NW, LDK = L::LDK, LDV = L::LDV;
     constexpr int ROW = DELTA ? ROW_DELTA : ROW_LINEAR;
     extern __shared__ __align__(16) float sm[];
-    float* part = sm + 2 * L::buffer;
+    float* part = sm + L::buffers * L::buffer;
     const int r = blockIdx.x, h = blockIdx.y;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, kw = warp % NW, mt = warp / NW;
     const int g = lane >> 2, t4 = lane & 3, pg = (g >> 1) + (g & 1) * 4;
@@ -254,7 +410,31 @@ chunk_scan_kernel(ChunkParams p) {
         float* b = sm + buf * L::buffer;
         const int n = min(C, te - tb);
         const float* src = p.qkv + (size_t)tb * p.ld;
-        if (p.vec & 1) {
+        if constexpr (CHAN) {
+            const float* rows = p.chan + ((size_t)tb * p.heads + h) * 3 * p.dk;
+            const size_t step = (size_t)p.heads * 3 * p.dk;
+            const float* end = p.gend + ((size_t)chunk_index(r, ta, (tb - ta) / C) * p.heads + h) * p.dk;
+            if (p.vec & 1) {
+                for (int idx = threadIdx.x; idx < C * (DKP / 4); idx += THREADS) {
+                    const int t = idx / (DKP / 4), i = (idx % (DKP / 4)) * 4;
+                    const bool in = t < n && i < p.dk;
+                    const float* s = in ? rows + t * step + i : rows;
+                    copy16(b + L::k0 + t * LDK + i, s, in);
+                    copy16(b + L::q0 + t * LDK + i, in ? s + p.dk : rows, in);
+                    copy16(b + L::r0 + t * LDK + i, in ? s + 2 * p.dk : rows, in);
+                }
+            } else {
+                for (int idx = threadIdx.x; idx < C * DKP; idx += THREADS) {
+                    const int t = idx / DKP, i = idx % DKP;
+                    const bool in = t < n && i < p.dk;
+                    const float* s = in ? rows + t * step + i : rows;
+                    copy4(b + L::k0 + t * LDK + i, s, in);
+                    copy4(b + L::q0 + t * LDK + i, in ? s + p.dk : rows, in);
+                    copy4(b + L::r0 + t * LDK + i, in ? s + 2 * p.dk : rows, in);
+                }
+            }
+            for (int i = threadIdx.x; i < DKP; i += THREADS) copy4(b + L::g0 + i, i < p.dk ? end + i : end, i < p.dk);
+        } else if (p.vec & 1) {
             for (int idx = threadIdx.x; idx < C * (DKP / 4); idx += THREADS) {
                 const int t = idx / (DKP / 4), i = (idx % (DKP / 4)) * 4;
                 const bool in = t < n && i < p.dk;
@@ -307,11 +487,11 @@ chunk_scan_kernel(ChunkParams p) {
         }
     if (ta < te) fetch(ta, 0);
     int buf = 0;
-    for (int tb = ta; tb < te; tb += C, buf ^= 1) {
+    for (int tb = ta; tb < te; tb += C, buf ^= L::buffers - 1) {
         const int n = min(C, te - tb);
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();                   // this chunk has arrived, the one before has been read
-        if (tb + C < te) fetch(tb + C, buf ^ 1);
+        if (L::buffers == 2 && tb + C < te) fetch(tb + C, buf ^ 1);
         const float* b = sm + buf * L::buffer;
         const float *ks = b + L::k0, *qs = b + L::q0, *vs = b + L::v0 + mt * COLS, *ms = b + L::m0, *ts = b + L::t0, *sc = b + L::s0;
         {   // this warp's rows of S0^T q_t (and S0^T k_t), all tokens side by side
@@ -414,11 +594,12 @@ chunk_scan_kernel(ChunkParams p) {
             }
         }
         {   // the state after the chunk
-            const float G = sc[(n - 1) * 4];
+            const float G = CHAN ? 1.f : sc[(n - 1) * 4];
+            const float *ge = b + L::g0 + k0 + t4, *ku = CHAN ? b + L::r0 : ks;       // the keys that take the decays after them in
 #pragma unroll
             for (int nb = 0; nb < NB; ++nb)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) s[nb][e] *= G;
+                for (int e = 0; e < 4; ++e) s[nb][e] *= CHAN ? ge[8 * nb + (e & 1) * 4] : G;
 #pragma unroll
             for (int kb = 0; kb < 4; ++kb) {
                 if (8 * kb >= n) break;
@@ -427,9 +608,13 @@ chunk_scan_kernel(ChunkParams p) {
                 const SplitA a = split_a(u[kb][0] * R0, u[kb][1] * R0, u[kb][2] * R1, u[kb][3] * R1);
                 float k[NB][2];
 #pragma unroll
-                for (int nb = 0; nb < NB; ++nb) { k[nb][0] = ks[t * LDK + k0 + 8 * nb + pg]; k[nb][1] = ks[(t + 1) * LDK + k0 + 8 * nb + pg]; }
+                for (int nb = 0; nb < NB; ++nb) { k[nb][0] = ku[t * LDK + k0 + 8 * nb + pg]; k[nb][1] = ku[(t + 1) * LDK + k0 + 8 * nb + pg]; }
                 mma3<NB>(s, a, k);
             }
+        }
+        if (L::buffers == 1 && tb + C < te) {
+            __syncthreads();               // the one buffer has been read
+            fetch(tb + C, 0);
         }
     }
 #pragma unroll
@@ -451,31 +636,46 @@ int launch_rows(const ChunkParams& p, cudaStream_t s) {
     return 0;
 }
 
-template <bool DELTA, int NW, int NB, int MT>
-int launch_scan(const ChunkParams& p, int R, cudaStream_t s) {
-    constexpr int smem = ChunkSmem<DELTA, NW, NB, MT>::floats * (int)sizeof(float);
-    static_assert(smem <= 227 * 1024, "shared memory budget");
+template <int DKP>
+int launch_rows_channel(const ChunkParams& p, cudaStream_t s) {
+    constexpr int smem = (3 * C * (DKP + 4) + 2 * C * (C + 4)) * (int)sizeof(float);
     static bool raised[bw::MAX_DEVICES] = {};
-    if (bw::allow_dynamic_smem(chunk_scan_kernel<DELTA, NW, NB, MT>, smem, raised) != cudaSuccess) return BW_ERR_DRIVER;
-    const int cols = COLS * MT;
-    bw::launch((chunk_scan_kernel<DELTA, NW, NB, MT>), dim3(R, p.heads, (p.dv + cols - 1) / cols), dim3(32 * NW * MT), smem, s, p);
+    if (bw::allow_dynamic_smem(chunk_rows_channel_kernel<DKP>, smem, raised) != cudaSuccess) return BW_ERR_DRIVER;
+    bw::launch((chunk_rows_channel_kernel<DKP>), dim3(p.T / C + p.R, p.heads), dim3(128), smem, s, p);
     BW_LAUNCH_CHECK();
     return 0;
 }
 
-template <bool DELTA>
+template <bool DELTA, bool CHAN, int NW, int NB, int MT>
+int launch_scan(const ChunkParams& p, int R, cudaStream_t s) {
+    constexpr int smem = ChunkSmem<DELTA, CHAN, NW, NB, MT>::floats * (int)sizeof(float);
+    static_assert(smem <= 227 * 1024, "shared memory budget");
+    static bool raised[bw::MAX_DEVICES] = {};
+    if (bw::allow_dynamic_smem(chunk_scan_kernel<DELTA, CHAN, NW, NB, MT>, smem, raised) != cudaSuccess) return BW_ERR_DRIVER;
+    const int cols = COLS * MT;
+    bw::launch((chunk_scan_kernel<DELTA, CHAN, NW, NB, MT>), dim3(R, p.heads, (p.dv + cols - 1) / cols), dim3(32 * NW * MT), smem, s, p);
+    BW_LAUNCH_CHECK();
+    return 0;
+}
+
+template <bool DELTA, bool CHAN>
 int run(const ChunkParams& p, int R, cudaStream_t s) {
     const int nw = p.dk <= 32 ? 1 : (p.dk <= 64 ? 2 : (p.dk <= 128 ? 4 : 8));
-    const int rc = nw == 1 ? launch_rows<DELTA, 32>(p, s) : (nw == 2 ? launch_rows<DELTA, 64>(p, s)
-                 : (nw == 4 ? launch_rows<DELTA, 128>(p, s) : launch_rows<DELTA, 256>(p, s)));
+    int rc;
+    if constexpr (CHAN)
+        rc = nw == 1 ? launch_rows_channel<32>(p, s) : (nw == 2 ? launch_rows_channel<64>(p, s)
+           : (nw == 4 ? launch_rows_channel<128>(p, s) : launch_rows_channel<256>(p, s)));
+    else
+        rc = nw == 1 ? launch_rows<DELTA, 32>(p, s) : (nw == 2 ? launch_rows<DELTA, 64>(p, s)
+           : (nw == 4 ? launch_rows<DELTA, 128>(p, s) : launch_rows<DELTA, 256>(p, s)));
     if (rc) return rc;
     // more blocks than fit side by side: two column groups share a block, its keys and its matrices
     const bool wide = (long long)R * p.heads * ((p.dv + COLS - 1) / COLS) > (long long)bw::num_sms() * (DELTA ? 1 : 2);
     switch (nw) {
-        case 1: return wide ? launch_scan<DELTA, 2, 2, 2>(p, R, s) : launch_scan<DELTA, 2, 2, 1>(p, R, s);
-        case 2: return wide ? launch_scan<DELTA, 4, 2, 2>(p, R, s) : launch_scan<DELTA, 4, 2, 1>(p, R, s);
-        case 4: return wide ? launch_scan<DELTA, 4, 4, 2>(p, R, s) : (DELTA ? launch_scan<DELTA, 8, 2, 1>(p, R, s) : launch_scan<DELTA, 4, 4, 1>(p, R, s));
-        default: return launch_scan<DELTA, 8, 4, 1>(p, R, s);
+        case 1: return wide ? launch_scan<DELTA, CHAN, 2, 2, 2>(p, R, s) : launch_scan<DELTA, CHAN, 2, 2, 1>(p, R, s);
+        case 2: return wide ? launch_scan<DELTA, CHAN, 4, 2, 2>(p, R, s) : launch_scan<DELTA, CHAN, 4, 2, 1>(p, R, s);
+        case 4: return wide ? launch_scan<DELTA, CHAN, 4, 4, 2>(p, R, s) : (DELTA ? launch_scan<DELTA, CHAN, 8, 2, 1>(p, R, s) : launch_scan<DELTA, CHAN, 4, 4, 1>(p, R, s));
+        default: return launch_scan<DELTA, CHAN, 8, 4, 1>(p, R, s);
     }
 }
 
@@ -487,17 +687,24 @@ BW_EXPORT int bw_chunk_row_floats(int delta) { return delta ? ROW_DELTA : ROW_LI
 // qkv: float32 rows `ld` apart with q and k (heads / rep heads of dk channels) and v (heads of dv) at the given columns;
 // decay [T, heads]; second [T, heads]: beta (delta != 0) or the keys' factor; rows: scratch float32
 // [T, heads, bw_chunk_row_floats(delta)], 16-byte aligned; state [slots, heads, dk, sld]; o [T, heads * dv].
+// delta == 2: the delta rule with decay [T, heads * dk]; chan: scratch float32 [T, heads, 3, dk], gend: scratch float32
+// [T / 32 + R, heads, dk], both 16-byte aligned (otherwise null).
 BW_EXPORT int bw_chunk_scan(int delta, const float* qkv, long long ld, int q_off, int k_off, int v_off, const float* decay,
                             const float* second, const int* cu_q, const int* state_slot, float* rows,
-                            float* state, float* o, int T, int R, int heads, int rep, int dk, int dv, int sld, void* stream) {
+                            float* chan, float* gend, float* state, float* o, int T, int R, int heads, int rep, int dk, int dv,
+                            int sld, void* stream) {
     if (T <= 0 || R <= 0) return 0;
     if (heads <= 0 || rep <= 0 || heads % rep || dk <= 0 || dv <= 0 || sld < dv || !rows || ((uintptr_t)rows & 15)) return BW_ERR_BAD_ARG;
     if (dk > 256) return BW_ERR_UNSUPPORTED;
+    if (delta == 2 && (!chan || !gend || (((uintptr_t)chan | (uintptr_t)gend) & 15))) return BW_ERR_BAD_ARG;
     ChunkParams p;
+    p.chan = chan; p.gend = gend;
     p.qkv = qkv; p.ld = ld; p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.decay = decay; p.second = second; p.cu_q = cu_q;
     p.state_slot = state_slot; p.rows = rows; p.state = state; p.sld = sld; p.o = o;
     p.T = T; p.R = R; p.heads = heads; p.rep = rep; p.dk = dk; p.dv = dv;
     const bool base = ((uintptr_t)qkv & 15) == 0 && (ld & 3) == 0;
     p.vec = (base && (dk & 3) == 0 && (q_off & 3) == 0 && (k_off & 3) == 0 ? 1 : 0) | (base && (dv & 3) == 0 && (v_off & 3) == 0 ? 2 : 0);
-    return delta ? run<true>(p, R, (cudaStream_t)stream) : run<false>(p, R, (cudaStream_t)stream);
+    if (delta == 2 && ((uintptr_t)decay & 15)) p.vec &= ~1;
+    if (delta == 2) return run<true, true>(p, R, (cudaStream_t)stream);
+    return delta ? run<true, false>(p, R, (cudaStream_t)stream) : run<false, false>(p, R, (cudaStream_t)stream);
 }

@@ -230,11 +230,11 @@ int launch_scan_any(const ScanParams& p, int R, cudaStream_t s) {
     return scan_narrow(R, p.heads, p.dv) ? launch_scan<NW, 2, MEM, 16>(p, R, s) : launch_scan<NW, 4, MEM, 16>(p, R, s);
 }
 
-// one warp per (token, head): o / sqrt(mean(o^2) + eps) * gain[c] * silu(g[c])
+// one warp per (token, head): o / sqrt(mean(o^2) + eps) * gain[c] * silu(g[c]); ready != 0: times g[c] as it is
 template <typename OT>
 __global__ void __launch_bounds__(128)
 gla_gate_kernel(const float* __restrict__ o, const float* __restrict__ g, long long g_ld, int g_off,
-                const float* __restrict__ gain, OT* __restrict__ out, int T, int heads, int dv, float eps) {
+                const float* __restrict__ gain, OT* __restrict__ out, int T, int heads, int dv, float eps, int ready) {
     BW_PDL_TRIGGER();
     BW_PDL_WAIT();
     const int item = blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -250,7 +250,7 @@ gla_gate_kernel(const float* __restrict__ o, const float* __restrict__ g, long l
     OT* dst = out + (size_t)t * heads * dv + (size_t)h * dv;
     for (int c = lane; c < dv; c += 32) {
         const float gv = grow[c];
-        const float sg = gv / (1.f + expf(-gv));
+        const float sg = ready ? gv : gv / (1.f + expf(-gv));
         dst[c] = bw::from_f32<OT>(orow[c] * r * gain[c] * sg);
     }
 }
@@ -300,16 +300,17 @@ BW_EXPORT int bw_gla_decay(const float* x, long long ldx, int x_off, const void*
     return 0;
 }
 
+// ready != 0: g holds the gate itself (whatever activation it has is in it already); 0: its silu is taken here.
 BW_EXPORT int bw_gla_gate(const float* o, const float* g, long long g_ld, int g_off, const float* gain, void* out,
-                          int out_type, int T, int heads, int dv, float eps, void* stream) {
+                          int out_type, int T, int heads, int dv, float eps, int ready, void* stream) {
     if (T <= 0) return 0;
     if (heads <= 0 || dv <= 0) return BW_ERR_BAD_ARG;
     const int items = T * heads;
     cudaStream_t s = (cudaStream_t)stream;
     if (out_type == BW_F32)
-        bw::launch((gla_gate_kernel<float>), dim3((items + 3) / 4), dim3(128), 0, s, o, g, g_ld, g_off, gain, (float*)out, T, heads, dv, eps);
+        bw::launch((gla_gate_kernel<float>), dim3((items + 3) / 4), dim3(128), 0, s, o, g, g_ld, g_off, gain, (float*)out, T, heads, dv, eps, ready);
     else if (out_type == BW_BF16)
-        bw::launch((gla_gate_kernel<bf16>), dim3((items + 3) / 4), dim3(128), 0, s, o, g, g_ld, g_off, gain, (bf16*)out, T, heads, dv, eps);
+        bw::launch((gla_gate_kernel<bf16>), dim3((items + 3) / 4), dim3(128), 0, s, o, g, g_ld, g_off, gain, (bf16*)out, T, heads, dv, eps, ready);
     else return BW_ERR_BAD_ARG;
     BW_LAUNCH_CHECK();
     return 0;

@@ -1,0 +1,220 @@
+// The second halves of projections through a small inner size, W2 (W1 x), and what a recurrent mixer makes of them:
+//
+//   decay   g[t, c] = exp(A[c / per] * softplus(z + bias[c])),  A = -exp(A_log), one per `per` neighbouring channels (a head)
+//   gate    s[t, c] = sigmoid(z)
+//
+// with z = sum_r x[t, r] W2[c, r], x being `rank` columns of the first halves' float32 result.  Several such parts share a
+// launch (blockIdx.z).  Everything is float32.  bfloat16 weights: mma.sync m16n8k16 with x split into two bfloat16 halves
+// (x = hi + lo up to 2^-17 of it) and float32 sums, the weights as they are; float32 weights: float32 multiply-adds.  The
+// order of the sums depends on the inner size alone.
+#include "common.cuh"
+
+using bf16 = __nv_bfloat16;
+
+namespace {
+
+constexpr int MAX_PARTS = 2;
+enum { PART_DECAY = 0, PART_SIGMOID = 1 };
+
+struct Part {
+    const void* w;               // [n_out, rank]
+    const float *A, *bias;       // decay: [n_out / per], [n_out]
+    float* out;                  // [T, n_out]
+    int x_off, rank, n_out, per, kind;
+};
+struct LowRankParams {
+    const float* x; long long ld;
+    int T, vec;
+    Part part[MAX_PARTS];
+};
+
+__device__ __forceinline__ float finish(const Part& q, int c, float z) {
+    if (q.kind == PART_SIGMOID) return 1.f / (1.f + expf(-z));
+    z += q.bias[c];
+    const float d = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+    return expf(q.A[c / q.per] * d);
+}
+
+// float32 weights: 32 tokens x 64 outputs a block, 32 inner values at a time
+constexpr int FT = 32, FO = 64, FK = 32;
+__global__ void __launch_bounds__(256)
+lowrank_f32_kernel(LowRankParams p) {
+    BW_PDL_TRIGGER();
+    const Part q = p.part[blockIdx.z];
+    const int t0 = blockIdx.x * FT, o0 = blockIdx.y * FO;
+    if (o0 >= q.n_out) return;
+    __shared__ float xs[FT][FK + 1], ws[FO][FK + 1];
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    const float* w = (const float*)q.w;
+    float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+    BW_PDL_WAIT();
+    for (int k0 = 0; k0 < q.rank; k0 += FK) {
+        for (int idx = threadIdx.x; idx < FT * FK; idx += 256) {
+            const int t = t0 + idx / FK, k = k0 + idx % FK;
+            xs[idx / FK][idx % FK] = (t < p.T && k < q.rank) ? p.x[(size_t)t * p.ld + q.x_off + k] : 0.f;
+        }
+        for (int idx = threadIdx.x; idx < FO * FK; idx += 256) {
+            const int o = o0 + idx / FK, k = k0 + idx % FK;
+            ws[idx / FK][idx % FK] = (o < q.n_out && k < q.rank) ? w[(size_t)o * q.rank + k] : 0.f;
+        }
+        __syncthreads();
+#pragma unroll 8
+        for (int k = 0; k < FK; ++k) {
+            const float a0 = xs[ty * 2][k], a1 = xs[ty * 2 + 1][k];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float b = ws[tx + 16 * j][k];
+                acc[0][j] = fmaf(a0, b, acc[0][j]);
+                acc[1][j] = fmaf(a1, b, acc[1][j]);
+            }
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int t = t0 + ty * 2 + i;
+        if (t >= p.T) continue;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int o = o0 + tx + 16 * j;
+            if (o < q.n_out) q.out[(size_t)t * q.n_out + o] = finish(q, o, acc[i][j]);
+        }
+    }
+}
+
+// bfloat16 weights: a block of 4 warps makes 64 tokens x 64 outputs, warp w the tokens 16 w ..; 64 inner values at a time;
+// rows of shared memory padded to 144 bytes, so that the 8 rows of an ldmatrix fall into different banks
+constexpr int MT = 64, MO = 64, MK = 64, MROW = (MK + 8) * 2;
+
+__device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// two neighbouring values as bfloat16 pairs: the rounded values, and what the rounding left
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    hi = *reinterpret_cast<const uint32_t*>(&h);
+    lo = bw::pack_bf16x2(a - __low2float(h), b - __high2float(h));
+}
+
+__global__ void __launch_bounds__(128)
+lowrank_mma_kernel(LowRankParams p) {
+    BW_PDL_TRIGGER();
+    const Part q = p.part[blockIdx.z];
+    const int t0 = blockIdx.x * MT, o0 = blockIdx.y * MO;
+    if (o0 >= q.n_out) return;
+    __shared__ __align__(16) uint8_t xh[MT * MROW], xl[MT * MROW], ws[MO * MROW];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const bf16* w = (const bf16*)q.w;
+    float acc[MO / 8][4];
+#pragma unroll
+    for (int j = 0; j < MO / 8; ++j) { acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f; }
+    const int srow = threadIdx.x >> 1, scol = (threadIdx.x & 1) * 32;       // this thread stages 32 inner values of a row of each
+    const int t = t0 + srow, o = o0 + srow;
+    const bool vec = (p.vec >> blockIdx.z) & 1;
+    BW_PDL_WAIT();
+    for (int k0 = 0; k0 < q.rank; k0 += MK) {
+        const float* src = p.x + (size_t)(t < p.T ? t : 0) * p.ld + q.x_off + k0 + scol;
+        const bf16* wsrc = w + (size_t)(o < q.n_out ? o : 0) * q.rank + k0 + scol;
+#pragma unroll
+        for (int c = 0; c < 32; c += 8) {
+            float v[8];
+            uint4 wv = make_uint4(0, 0, 0, 0);
+            if (vec) {           // (the inner size is a multiple of 8: a stretch of eight is inside or outside)
+                const bool in = k0 + scol + c < q.rank;
+                const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+                const float4 a = in && t < p.T ? *reinterpret_cast<const float4*>(src + c) : zero;
+                const float4 b = in && t < p.T ? *reinterpret_cast<const float4*>(src + c + 4) : zero;
+                v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+                if (in && o < q.n_out) wv = __ldg(reinterpret_cast<const uint4*>(wsrc + c));
+            } else {
+                bf16 we[8];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    const bool ok = k0 + scol + c + i < q.rank;
+                    v[i] = (ok && t < p.T) ? src[c + i] : 0.f;
+                    we[i] = (ok && o < q.n_out) ? wsrc[c + i] : __float2bfloat16_rn(0.f);
+                }
+                wv = *reinterpret_cast<const uint4*>(we);
+            }
+            uint4 hi, lo;
+            split2(v[0], v[1], hi.x, lo.x); split2(v[2], v[3], hi.y, lo.y); split2(v[4], v[5], hi.z, lo.z); split2(v[6], v[7], hi.w, lo.w);
+            *reinterpret_cast<uint4*>(xh + srow * MROW + (scol + c) * 2) = hi;
+            *reinterpret_cast<uint4*>(xl + srow * MROW + (scol + c) * 2) = lo;
+            *reinterpret_cast<uint4*>(ws + srow * MROW + (scol + c) * 2) = wv;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int ks = 0; ks < MK / 16; ++ks) {
+            if (k0 + ks * 16 >= q.rank) break;
+            uint32_t ah[4], al[4];
+            const int at = (warp * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * MROW + 16 * (lane >> 4) + ks * 32;
+            ldsm_x4(smem_addr(xh) + at, ah);
+            ldsm_x4(smem_addr(xl) + at, al);
+#pragma unroll
+            for (int nb = 0; nb < MO / 16; ++nb) {
+                uint32_t b[4];
+                ldsm_x4(smem_addr(ws) + (nb * 16 + (lane & 7) + 8 * (lane >> 4)) * MROW + 16 * ((lane >> 3) & 1) + ks * 32, b);
+                mma_bf16(acc[2 * nb], al, b[0], b[1]);
+                mma_bf16(acc[2 * nb + 1], al, b[2], b[3]);
+                mma_bf16(acc[2 * nb], ah, b[0], b[1]);
+                mma_bf16(acc[2 * nb + 1], ah, b[2], b[3]);
+            }
+        }
+        __syncthreads();
+    }
+    const bool pairs = (q.n_out & 1) == 0 && ((uintptr_t)q.out & 7) == 0;
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const int row = t0 + warp * 16 + (lane >> 2) + 8 * half;
+        if (row >= p.T) continue;
+        float* dst = q.out + (size_t)row * q.n_out;
+#pragma unroll
+        for (int j = 0; j < MO / 8; ++j) {
+            const int c = o0 + j * 8 + 2 * (lane & 3);
+            if (pairs && c + 1 < q.n_out)
+                *reinterpret_cast<float2*>(dst + c) = make_float2(finish(q, c, acc[j][2 * half]), finish(q, c + 1, acc[j][2 * half + 1]));
+            else {
+                if (c < q.n_out) dst[c] = finish(q, c, acc[j][2 * half]);
+                if (c + 1 < q.n_out) dst[c + 1] = finish(q, c + 1, acc[j][2 * half + 1]);
+            }
+        }
+    }
+}
+
+}  // namespace
+
+// x: float32 [T, .], rows `ld` apart.  n parts (1 or 2), each: the column x_off of its inner values, rank, w [n_out, rank] of
+// w_type, kind (0 decay, 1 sigmoid), A [n_out / per] and bias [n_out] float32 (decay), out float32 [T, n_out].
+BW_EXPORT int bw_lowrank_gates(const float* x, long long ld, int w_type, int T, int n, const int* x_off, const int* rank,
+                               const int* n_out, const int* kind, const int* per, const void* const* w,
+                               const float* const* A, const float* const* bias, float* const* out, void* stream) {
+    if (T <= 0) return 0;
+    if (n < 1 || n > MAX_PARTS) return BW_ERR_BAD_ARG;
+    LowRankParams p;
+    p.x = x; p.ld = ld; p.T = T; p.vec = 0;
+    int widest = 0;
+    for (int i = 0; i < n; ++i) {
+        Part& q = p.part[i];
+        q.w = w[i]; q.A = A[i]; q.bias = bias[i]; q.out = out[i];
+        q.x_off = x_off[i]; q.rank = rank[i]; q.n_out = n_out[i]; q.per = per[i]; q.kind = kind[i];
+        if (q.rank <= 0 || q.n_out <= 0 || q.x_off < 0 || !q.w || !q.out || q.kind < 0 || q.kind > PART_SIGMOID || ld < q.x_off + q.rank ||
+            (q.kind == PART_DECAY && (!q.A || !q.bias || q.per <= 0 || q.n_out % q.per)))
+            return BW_ERR_BAD_ARG;
+        if (q.rank % 8 == 0 && ld % 4 == 0 && (((uintptr_t)(x + q.x_off) | (uintptr_t)q.w) & 15) == 0) p.vec |= 1 << i;
+        if (q.n_out > widest) widest = q.n_out;
+    }
+    for (int i = n; i < MAX_PARTS; ++i) p.part[i] = p.part[0];
+    cudaStream_t s = (cudaStream_t)stream;
+    if (w_type == BW_F32)
+        bw::launch((lowrank_f32_kernel), dim3((T + FT - 1) / FT, (widest + FO - 1) / FO, n), dim3(256), 0, s, p);
+    else if (w_type == BW_BF16)
+        bw::launch((lowrank_mma_kernel), dim3((T + MT - 1) / MT, (widest + MO - 1) / MO, n), dim3(128), 0, s, p);
+    else return BW_ERR_BAD_ARG;
+    BW_LAUNCH_CHECK();
+    return 0;
+}

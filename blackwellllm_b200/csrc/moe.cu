@@ -6,14 +6,16 @@
 //
 //   moe_route    one warp per token: score = sigmoid(logit) (or softmax), the `top` largest scores
 //                (lowest index on ties), optionally renormalised to sum 1; float32 throughout.  With a bias
-//                per router output the CHOICE goes by score + bias while the weights stay the scores.
+//                per router output the CHOICE goes by score + bias while the weights stay the scores.  softmax == 2: the
+//                choice goes by the logits and the weights are exp(logit - largest), to be renormalised: a softmax over the
+//                chosen logits alone
 //                The router may have more outputs than there are experts: outputs from `E` (the experts
 //                that have weights) up to `E_total` stand for experts that return their input; their rows
 //                take no part in the regrouping and the products, and moe_combine adds weight * x for them
 //   moe_plan     one block: rows per expert, each expert's stretch padded to whole tiles (64 rows here, 128 in moe_tc.cu),
 //                the place of every (token, choice) row, and the expert of every tile
 //   moe_scatter  the regrouped operand: row (token, choice) = weight * x[token] (input scaling) or x[token]
-//   moe_gemm     C[row, :] = A[row, :] W[expert of row]^T, optionally as silu(A Wg^T) * (A Wu^T);
+//   moe_gemm     C[row, :] = A[row, :] W[expert of row]^T, optionally as silu(A Wg^T) * (A Wu^T), or with an activation;
 //                float32 sums on the CUDA cores from float32 or bfloat16 operands (the true 32-bit path, and
 //                bfloat16 sizes that the tcgen05 kernel of moe_tc.cu does not take)
 //   moe_combine  out[token] = sum over choices (in order) of (weight *) C[row of (token, choice)], written,
@@ -64,8 +66,11 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, in
     if (softmax) {
         for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, z[e]);
         zmax = bw::warp_max(zmax);
-        for (int e = lane; e < E; e += 32) zsum += expf(z[e] - zmax);
-        zsum = bw::warp_sum(zsum);
+        if (softmax == 2) zsum = 1.f;
+        else {
+            for (int e = lane; e < E; e += 32) zsum += expf(z[e] - zmax);
+            zsum = bw::warp_sum(zsum);
+        }
     }
     float total = 0.f;
     int last = -1; float last_s = INFINITY;   // choices are taken in order of (choice score descending, index ascending)
@@ -73,7 +78,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, in
         float best = -INFINITY, best_w = 0.f; int bi = 0x7fffffff;
         for (int e = lane; e < E; e += 32) {
             const float w = softmax ? expf(z[e] - zmax) / zsum : 1.f / (1.f + expf(-z[e]));
-            const float s = bias ? w + bias[e] : w;
+            const float s = softmax == 2 ? z[e] : (bias ? w + bias[e] : w);
             const bool after = (s < last_s) || (s == last_s && e > last);   // not chosen yet
             if (after && (s > best || (s == best && e < bi))) { best = s; best_w = w; bi = e; }
         }
@@ -243,6 +248,7 @@ moe_gemm_kernel(const AT* __restrict__ A, const AT* __restrict__ W, const AT* __
             if (n >= N) continue;
             float v = acc[i][j];
             if constexpr (GATED) v = bw::glu(act, v, acc2[i][j], limit, alpha);
+            else v = bw::unary_act(act, v);
             C[(size_t)(row0 + ty * 4 + i) * N + n] = bw::from_f32<CT>(v);
         }
 }

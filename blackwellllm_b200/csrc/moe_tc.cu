@@ -6,7 +6,8 @@
 //
 // One CTA per (tile of 128 rows, 128 weight rows): warp 0 feeds a ring of TMA stages (128-byte swizzle),
 // warp 1 owns the tensor memory and issues the MMAs (M = 128, N = 128, K = 16), warps 2..5 read the
-// accumulator (TMEM lane quarter = warp % 4) and write the result: either plain (float32 or bfloat16), or,
+// accumulator (TMEM lane quarter = warp % 4) and write the result: either plain (float32 or bfloat16, the latter also with
+// an activation of one input: experts without a gate), or,
 // for a gate/up weight whose rows alternate in blocks of 16 (16 gate features, the same 16 up features),
 // silu(gate) * up as bfloat16.  Three stages of 32 KB leave room for two CTAs on an SM.
 // Every wait is bounded; a wait that gives up sets the status word and the roles fall through to the exit.
@@ -125,7 +126,28 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ C
                     }
                 } else {
                     CT* dst = C + row * N + n0 + c0;
-                    if (n0 + c0 + 32 <= N && (N & 3) == 0 && sizeof(CT) == 4) {
+                    if constexpr (sizeof(CT) == 2) {
+                        if (act == BW_ACT_RELU2) {
+#pragma unroll
+                            for (int j = 0; j < 32; ++j) {
+                                const float z = fmaxf(__uint_as_float(v[j]), 0.f);
+                                v[j] = __float_as_uint(z * z);
+                            }
+                        } else if (act == BW_ACT_GELU) {
+#pragma unroll
+                            for (int j = 0; j < 32; ++j) v[j] = __float_as_uint(bw::gelu_fast(__uint_as_float(v[j])));
+                        }
+                    }
+                    if (sizeof(CT) == 2 && n0 + c0 + 32 <= N && (N & 7) == 0) {
+#pragma unroll
+                        for (int j = 0; j < 4; ++j) {
+                            uint32_t w[4];
+#pragma unroll
+                            for (int e = 0; e < 4; ++e)
+                                w[e] = bw::pack_bf16x2(__uint_as_float(v[8 * j + 2 * e]), __uint_as_float(v[8 * j + 2 * e + 1]));
+                            reinterpret_cast<uint4*>(dst)[j] = make_uint4(w[0], w[1], w[2], w[3]);
+                        }
+                    } else if (n0 + c0 + 32 <= N && (N & 3) == 0 && sizeof(CT) == 4) {
 #pragma unroll
                         for (int j = 0; j < 8; ++j)
                             reinterpret_cast<uint4*>(dst)[j] = make_uint4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
@@ -171,7 +193,8 @@ BW_EXPORT int bw_moe_tc_supported(const void* A, const void* W, int N, int K, in
 
 // A: bfloat16 [max_tiles * 128, K]; W: bfloat16 [E, N, K]; tile_expert: int32 [max_tiles].
 // gated: W's rows alternate 16 gate / 16 up and C is bfloat16 [rows, N / 2] = glu(gate, up) with the gated
-// activation `act` of common.cuh and its limit and alpha (BW_ACT_SILU: silu(gate) * up); else C is [rows, N] of c_type.
+// activation `act` of common.cuh and its limit and alpha (BW_ACT_SILU: silu(gate) * up); else C is [rows, N] of c_type, and a
+// bfloat16 C gets the activation `act` where it is BW_ACT_RELU2 or BW_ACT_GELU (0: none).
 BW_EXPORT int bw_moe_gemm_tc(const void* A, const void* W, int gated, const int* tile_expert, void* C, int c_type,
                              int max_tiles, int E, int N, int K, int act, float limit, float alpha, void* stream) {
     if (max_tiles <= 0) return 0;
@@ -182,8 +205,9 @@ BW_EXPORT int bw_moe_gemm_tc(const void* A, const void* W, int gated, const int*
     cudaStream_t s = (cudaStream_t)stream;
     if (gated && act != BW_ACT_SILU && act != BW_ACT_CLAMPED_SWISH) return BW_ERR_BAD_ARG;
     if (gated) return launch<true, bf16>(ta, tb, tile_expert, C, max_tiles, N, K, act, limit, alpha, s);
+    if (act != 0 && (c_type != BW_BF16 || (act != BW_ACT_RELU2 && act != BW_ACT_GELU))) return BW_ERR_BAD_ARG;
     if (c_type == BW_F32) return launch<false, float>(ta, tb, tile_expert, C, max_tiles, N, K, 0, 0.f, 1.f, s);
-    if (c_type == BW_BF16) return launch<false, bf16>(ta, tb, tile_expert, C, max_tiles, N, K, 0, 0.f, 1.f, s);
+    if (c_type == BW_BF16) return launch<false, bf16>(ta, tb, tile_expert, C, max_tiles, N, K, act, 0.f, 1.f, s);
     return BW_ERR_BAD_ARG;
 }
 

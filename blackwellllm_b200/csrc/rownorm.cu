@@ -2,7 +2,8 @@
 //
 //   y   = what the sublayer left: one float32 row, or the mean of two rows that are RMS-normed with a gain each
 //   x  += post(y) * gp                    post: layer norm, RMS norm or nothing; gp may hold further constants
-//   h   = next(x) * gn                    next: the norm before the next sublayer (or none)
+//   h   = next(x) * gn                    next: the norm before the next sublayer (or none), which may also be
+//                                         tanh(alpha x) * gn + bn, a norm without any statistic of the row
 //
 // in one pass over the stream.  A row of y may come as planes of a matrix product that its kernel left unsummed; they are
 // added (in plane order) while they are read.  One block per row; a row's values stay in registers from the first load to
@@ -13,8 +14,9 @@ using bf16 = __nv_bfloat16;
 
 namespace {
 
-// what a norm does to a row: 0 nothing, 1 x / sqrt(mean(x^2) + eps), 2 (x - mean) / sqrt(mean((x - mean)^2) + eps)
-enum { NORM_NONE = 0, NORM_RMS = 1, NORM_LAYER = 2 };
+// what a norm does to a row: 0 nothing, 1 x / sqrt(mean(x^2) + eps), 2 (x - mean) / sqrt(mean((x - mean)^2) + eps), 3 (only as the
+// next norm) tanh(alpha x), with a bias after the gain
+enum { NORM_NONE = 0, NORM_RMS = 1, NORM_LAYER = 2, NORM_TANH = 3 };
 
 struct RowParams {
     float* x;                // the stream [T, H]
@@ -27,6 +29,7 @@ struct RowParams {
     int pair, has_y;
     const float* gp; float post_eps; int post;
     const float* gn; float next_eps; int next;
+    const float* bn; float alpha;   // NORM_TANH: the bias after the gain [H] or null, the factor inside the tanh
     const int* rows;         // only these rows, and x stays as it is
     void* out; int H;
 };
@@ -186,7 +189,7 @@ row_step_kernel(RowParams p) {
             for (int e = 0; e < W; ++e) s += x[i][e];
         mean = block_sum2(s, 0.f, scratch).x * inv_h;
     }
-    if (p.next != NORM_NONE) {
+    if (p.next == NORM_RMS || p.next == NORM_LAYER) {
         float s = 0.f;
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
@@ -203,8 +206,17 @@ row_step_kernel(RowParams p) {
         if (c < H) {
             float g[W], o[W];
             if (p.gn) ld<W>(p.gn + c, g);
+            if (p.next == NORM_TANH) {
+                float b[W];
 #pragma unroll
-            for (int e = 0; e < W; ++e) { o[e] = (x[i][e] - mean) * r; if (p.gn) o[e] *= g[e]; }
+                for (int e = 0; e < W; ++e) b[e] = 0.f;
+                if (p.bn) ld<W>(p.bn + c, b);
+#pragma unroll
+                for (int e = 0; e < W; ++e) o[e] = fmaf(tanhf(p.alpha * x[i][e]), p.gn ? g[e] : 1.f, b[e]);
+            } else {
+#pragma unroll
+                for (int e = 0; e < W; ++e) { o[e] = (x[i][e] - mean) * r; if (p.gn) o[e] *= g[e]; }
+            }
             if constexpr (W == 4) st4(out + c, o);
             else st(out + c, o[0]);
         }
@@ -236,23 +248,24 @@ int run(const RowParams& p, int n, cudaStream_t s) {
 // x: float32 [T, H], updated in place unless `rows` names the rows to make (then out is dense [n, H]).  has_y == 0: no
 // sublayer output, only the next norm.  y / z: float32 [T, H] or null where the planes are all of it; planes: n of them,
 // `stride` floats apart, each [T, H].  pair: z counts, both rows are RMS-normed (pair_eps) times gy / gz and averaged.
-// post / next: 0 none, 1 RMS norm, 2 layer norm; gp / gn: float32 [H] or null.  out: null, or the next norm's result.
+// post / next: 0 none, 1 RMS norm, 2 layer norm, next also 3 tanh(alpha x); gp / gn: float32 [H] or null; bn: float32 [H] or null,
+// added after gn where next is 3.  out: null, or the next norm's result.
 BW_EXPORT int bw_row_step(float* x, int has_y, const float* y, const float* y_planes, long long y_stride, int y_n,
                           int pair, const float* z, const float* z_planes, long long z_stride, int z_n,
                           const float* gy, const float* gz, float pair_eps, int post, const float* gp, float post_eps,
-                          int next, const float* gn, float next_eps, const int* rows, void* out, int out_type, int n, int H,
+                          int next, const float* gn, float next_eps, const float* bn, float alpha, const int* rows, void* out, int out_type, int n, int H,
                           void* stream) {
     if (n <= 0) return 0;
-    if (H <= 0 || post < 0 || post > 2 || next < 0 || next > 2 || (pair && (!gy || !gz || !has_y)) || y_n < 0 || z_n < 0 ||
+    if (H <= 0 || post < 0 || post > 2 || next < 0 || next > 3 || (bn && next != 3) || (pair && (!gy || !gz || !has_y)) || y_n < 0 || z_n < 0 ||
         (has_y && !y && y_n == 0) || (pair && !z && z_n == 0) || (y_n && !y_planes) || (z_n && !z_planes))
         return BW_ERR_BAD_ARG;
     RowParams p;
     p.x = x; p.has_y = has_y; p.y = y; p.y_planes = y_planes; p.y_stride = y_stride; p.y_n = y_n;
     p.pair = pair; p.z = z; p.z_planes = z_planes; p.z_stride = z_stride; p.z_n = z_n;
     p.gy = gy; p.gz = gz; p.pair_eps = pair_eps; p.post = post; p.gp = gp; p.post_eps = post_eps;
-    p.next = next; p.gn = gn; p.next_eps = next_eps; p.rows = rows; p.out = out; p.H = H;
+    p.next = next; p.gn = gn; p.next_eps = next_eps; p.bn = bn; p.alpha = alpha; p.rows = rows; p.out = out; p.H = H;
     const uintptr_t all = (uintptr_t)x | (uintptr_t)y | (uintptr_t)y_planes | (uintptr_t)z | (uintptr_t)z_planes | (uintptr_t)gy |
-                          (uintptr_t)gz | (uintptr_t)gp | (uintptr_t)gn | (uintptr_t)out;
+                          (uintptr_t)gz | (uintptr_t)gp | (uintptr_t)gn | (uintptr_t)bn | (uintptr_t)out;
     const bool vec = (H & 3) == 0 && (all & 15) == 0 && (y_stride & 3) == 0 && (z_stride & 3) == 0;
     cudaStream_t s = (cudaStream_t)stream;
     if (out_type == BW_F32) return vec ? run<float, 4>(p, n, s) : run<float, 1>(p, n, s);

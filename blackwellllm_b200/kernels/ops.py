@@ -8,7 +8,7 @@ from __future__ import annotations
 import ctypes
 import math
 import os
-from typing import Optional
+from typing import List, Optional
 
 import torch
 
@@ -1523,17 +1523,18 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torc
 
 
 def gla_gate(o: torch.Tensor, proj: torch.Tensor, g_off: int, gain: torch.Tensor, heads: int, dv: int, eps: float,
-             out_dtype: torch.dtype) -> torch.Tensor:
-    """Per token and head ``o / rms(o) * gain * silu(g)`` with g at column ``g_off`` of ``proj``."""
+             out_dtype: torch.dtype, ready: bool = False) -> torch.Tensor:
+    """Per token and head ``o / rms(o) * gain * silu(g)`` with g at column ``g_off`` of ``proj``; ``ready``: g is the gate itself
+    and multiplies as it is."""
     _dev(o, "o", torch.float32); _dev(proj, "proj", torch.float32, contiguous=False); _dev(gain, "gain", torch.float32)
     T = o.shape[0]
     if o.shape[1] != heads * dv or gain.numel() != dv or proj.stride(1) != 1 or g_off + heads * dv > proj.shape[1]:
         raise KernelError("gla_gate: o must be [T, heads * dv], the gain [dv], the gate inside the projection")
     out = torch.empty((T, heads * dv), dtype=out_dtype, device=o.device)
     fn = _fn("gla", "bw_gla_gate", [c_void_p, c_void_p, c_ll, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                    c_float, c_void_p])
+                                    c_float, c_int, c_void_p])
     _check(fn(_ptr(o), _ptr(proj), proj.stride(0), g_off, _ptr(gain), _ptr(out), _code(out, "out"), T, heads, dv,
-              float(eps), _stream()), "gla_gate")
+              float(eps), int(ready), _stream()), "gla_gate")
     return out
 
 
@@ -1585,7 +1586,8 @@ def short_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], s
     ``state`` float32 [slots, taps, C]: the earlier inputs of the requests, position p at entry p mod taps; it takes the
     step's last inputs.  ``segments``: (heads, size, scale) per stretch of channels; a stretch with a scale that is not None
     has every head divided by sqrt(sum + ``unit_eps``) and multiplied by the scale.  ``gates`` = (z, column, column of the
-    second gate or None, A [heads], dt_bias [heads]): in the same kernel decay = exp(A d), d = softplus(z + dt_bias).
+    second gate or None, A [heads], dt_bias [heads]): in the same kernel decay = exp(A d), d = softplus(z + dt_bias);
+    (z, None, column of the second gate, heads, None): the second gate alone.
     Returns (float32 [T, C], decay, second) where second is sigmoid of the second gate, or d without one."""
     _dev(x, "x", torch.float32, contiguous=False); _dev(w, "w", torch.float32); _dev(state, "state", torch.float32)
     T = x.shape[0]
@@ -1603,12 +1605,18 @@ def short_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], s
     z_off, z2_off, heads = 0, -1, 0
     if gates is not None:
         z, z_off, z2, A, dtb = gates
-        _dev(z, "z", torch.float32, contiguous=False); _dev(A, "A", torch.float32); _dev(dtb, "dt_bias", torch.float32)
-        heads = A.numel()
+        _dev(z, "z", torch.float32, contiguous=False)
         z2_off = -1 if z2 is None else int(z2)
-        if dtb.numel() != heads or z.shape[0] != T or z.stride(1) != 1 or max(z_off, z2_off) + heads > z.shape[1]:
+        if z_off is None:
+            z_off, heads, A, dtb = -1, int(A), None, None
+            if z2_off < 0:
+                raise KernelError("short_conv: gates without a decay need the second gate's column")
+        else:
+            _dev(A, "A", torch.float32); _dev(dtb, "dt_bias", torch.float32)
+            heads = A.numel()
+        if (dtb is not None and dtb.numel() != heads) or z.shape[0] != T or z.stride(1) != 1 or max(z_off, z2_off) + heads > z.shape[1]:
             raise KernelError("short_conv: the gates' columns lie outside the projections")
-        decay = torch.empty((T, heads), dtype=torch.float32, device=x.device)
+        decay = torch.empty((T, heads), dtype=torch.float32, device=x.device) if z_off >= 0 else None
         second = torch.empty((T, heads), dtype=torch.float32, device=x.device)
     n = len(segments)
     heads_c, size_c = (c_int * n)(*[s[0] for s in segments]), (c_int * n)(*[s[1] for s in segments])
@@ -1623,6 +1631,88 @@ def short_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], s
     return out, decay, second
 
 
+LOWRANK_DECAY, LOWRANK_SIGMOID = 0, 1
+
+
+def lowrank_gates(proj: torch.Tensor, parts) -> List[torch.Tensor]:
+    """What a mixer makes of projections through a small inner size, z = W2 (W1 x): ``proj`` (float32 rows, possibly a range of
+    columns) holds the first halves' results.  ``parts``: one or two of (column, W2 [n_out, rank], kind, A, bias):
+    LOWRANK_DECAY: exp(A[c // per] * softplus(z + bias[c])) with A float32 [n_out / per], bias float32 [n_out];
+    LOWRANK_SIGMOID: sigmoid(z).  Returns one float32 [T, n_out] per part.  All in one kernel, float32 throughout (bfloat16
+    weights run on the tensor cores with the rows split into two bfloat16 parts)."""
+    _dev(proj, "proj", torch.float32, contiguous=False)
+    n, T = len(parts), proj.shape[0]
+    if not 1 <= n <= 2 or proj.dim() != 2 or proj.stride(1) != 1:
+        raise KernelError("lowrank_gates: one or two parts, proj [T, columns] with contiguous rows")
+    ws = [_dev(p[1], "w", parts[0][1].dtype) for p in parts]
+    outs = [torch.empty((T, w.shape[0]), dtype=torch.float32, device=proj.device) for w in ws]
+    per = [1] * n
+    for i, (col, w, kind, A, bias) in enumerate(parts):
+        if col < 0 or col + w.shape[1] > proj.shape[1]:
+            raise KernelError("lowrank_gates: a part's inner values lie outside the rows")
+        if kind == LOWRANK_DECAY:
+            _dev(A, "A", torch.float32); _dev(bias, "bias", torch.float32)
+            if w.shape[0] % A.numel() or bias.numel() != w.shape[0]:
+                raise KernelError("lowrank_gates: A must have one entry per head, the bias one per output")
+            per[i] = w.shape[0] // A.numel()
+    ints = lambda v: (c_int * n)(*[int(e) for e in v])
+    ptrs = lambda v: (c_void_p * n)(*[0 if t is None else t.data_ptr() for t in v])
+    fn = _fn("lowrank", "bw_lowrank_gates", [c_void_p, c_ll, c_int, c_int, c_int] + [c_void_p] * 10)
+    _check(fn(_ptr(proj), proj.stride(0), _code(ws[0], "w"), T, n, ints(p[0] for p in parts), ints(w.shape[1] for w in ws),
+              ints(w.shape[0] for w in ws), ints(p[2] for p in parts), ints(per), ptrs(ws), ptrs(p[3] for p in parts),
+              ptrs(p[4] for p in parts), ptrs(outs), _stream()), "lowrank_gates")
+    return outs
+
+
+def conv_heads(x: torch.Tensor, w: torch.Tensor, state: torch.Tensor, batch, block_table: torch.Tensor, k_pages: torch.Tensor,
+               v_pages: torch.Tensor, nq: int, d: int, maps: int, nkv: int, dv: int, has_kv: bool = True) -> torch.Tensor:
+    """A causal convolution over time per channel (no bias, no activation) of an attention's projections ``x`` float32 [T, >= C],
+    C = nq d + nkv (maps d + dv): ``nq`` query heads of ``d`` channels, ``nkv`` key heads of ``maps * d`` and value heads of ``dv``;
+    with ``has_kv`` False the queries alone.  ``w`` float32 [taps, C] (the last row is the current token's), ``state`` float32
+    [slots, taps, C] as in :func:`short_conv`.  The keys and values go to the pages [num_pages, nkv, page_size, dpad] of the
+    tokens' positions; returned are the queries [T, nq * dpad] in the pages' dtype, head h's channels at offset
+    (h mod maps) d of its row and zeros around them, so that query head h meets map h mod maps of its key head's row."""
+    _dev(x, "x", torch.float32, contiguous=False); _dev(w, "w", torch.float32); _dev(state, "state", torch.float32)
+    _dev(block_table, "block_table", torch.int32); _dev(k_pages, "k_pages"); _dev(v_pages, "v_pages", k_pages.dtype)
+    T = x.shape[0]
+    taps, C = w.shape
+    num_pages, pk, page_size, dpad = k_pages.shape
+    if C != nq * d + (nkv * (maps * d + dv) if has_kv else 0) or pk != nkv or nq % (maps * nkv) or dpad < max(maps * d, dv):
+        raise KernelError("conv_heads: w [taps, nq d (+ nkv (maps d + dv))], pages [num_pages, nkv, page, >= maps d and dv]")
+    if x.dim() != 2 or x.stride(1) != 1 or x.shape[1] < C or T != batch.T or state.dim() != 3 or tuple(state.shape[1:]) != (taps, C):
+        raise KernelError("conv_heads: x [T, >= C] with contiguous rows, state [slots, taps, C]")
+    q = torch.empty((T, nq * dpad), dtype=k_pages.dtype, device=x.device)
+    fn = _fn("shortconv", "bw_conv_heads", [c_void_p, c_ll] + [c_void_p] * 7 + [c_int] + [c_void_p] * 3 + [c_int] * 14 + [c_void_p])
+    _check(fn(_ptr(x), x.stride(0), _ptr(w), _ptr(state), _ptr(batch.positions), _ptr(batch.req_of_token), _ptr(batch.cu_q),
+              _ptr(batch.state_slot), _ptr(block_table), block_table.shape[1], _ptr(q), _ptr(k_pages), _ptr(v_pages),
+              _code(k_pages, "pages"), T, batch.R, taps, int(T == batch.R), nq, d, maps, nkv, dv, dpad, int(has_kv), page_size,
+              num_pages, _stream()), "conv_heads")
+    return q
+
+
+def diff_combine(a: torch.Tensor, heads: int, dv: int, lam: torch.Tensor, eps: float, scale: float,
+                 gate: Optional[torch.Tensor], out_dtype: torch.dtype) -> torch.Tensor:
+    """Differential attention's two maps made one: ``a`` [T, heads * 2 * dpad] holds head h's maps at 2 h and 2 h + 1 (channels from
+    ``dv`` on are padding); o = a1 - lam a2, divided by its root mean square over the dv channels, times ``scale`` and, with
+    ``gate`` (float32 [T, heads], possibly a range of columns), sigmoid(gate[t, h]).  ``lam``: one float32 number on the device.
+    Returns [T, heads * dpad]."""
+    _dev(a, "a"); _dev(lam, "lam", torch.float32)
+    T = a.shape[0]
+    if a.shape[1] % (2 * heads):
+        raise KernelError("diff_combine: a must be [T, 2 heads * dpad]")
+    dpad = a.shape[1] // (2 * heads)
+    if gate is not None:
+        _dev(gate, "gate", torch.float32, contiguous=False)
+        if gate.shape != (T, heads) or gate.stride(1) != 1:
+            raise KernelError("diff_combine: the gate must be float32 [T, heads] with contiguous rows")
+    out = torch.empty((T, heads * dpad), dtype=out_dtype, device=a.device)
+    fn = _fn("diffattn", "bw_diff_combine", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_float,
+                                             c_void_p, c_ll, c_void_p])
+    _check(fn(_ptr(a), _code(a, "a"), _ptr(out), _code(out, "out"), T, heads, dv, dpad, _ptr(lam), float(eps), float(scale),
+              _ptr(gate), gate.stride(0) if gate is not None else 0, _stream()), "diff_combine")
+    return out
+
+
 DELTA_MAX_KEY_DIM = 256
 
 
@@ -1630,27 +1720,31 @@ def delta_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: tor
                state: torch.Tensor, heads: int, qk_rep: int, dk: int, dv: int) -> torch.Tensor:
     """The gated delta rule ``S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q`` over the step's tokens, request by
     request in order, from and into ``state`` [slots, heads, dk, dv] (float32).  ``qkv`` float32 [T, ld] holds q and k
-    (``heads / qk_rep`` heads) and v (``heads`` heads) at the given columns; ``decay`` (g), ``beta`` float32 [T, heads].
+    (``heads / qk_rep`` heads) and v (``heads`` heads) at the given columns; ``decay`` (g), ``beta`` float32 [T, heads]; a
+    ``decay`` of [T, heads * dk] decays every key channel's row of the state by its own number.
     Returns o float32 [T, heads * dv]."""
     _dev(qkv, "qkv", torch.float32); _dev(decay, "decay", torch.float32); _dev(beta, "beta", torch.float32)
     _dev(state, "state", torch.float32)
     T = qkv.shape[0]
     if dk > DELTA_MAX_KEY_DIM:
         raise KernelError(f"delta_scan: key size {dk} exceeds {DELTA_MAX_KEY_DIM}")
-    if (qk_rep < 1 or heads % qk_rep or decay.shape != (T, heads) or beta.shape != (T, heads) or state.dim() != 4
+    channel = dk > 1 and decay.shape == (T, heads * dk)
+    if (qk_rep < 1 or heads % qk_rep or (not channel and decay.shape != (T, heads)) or beta.shape != (T, heads) or state.dim() != 4
             or tuple(state.shape[1:]) != (heads, dk, dv)):
-        raise KernelError("delta_scan: decay and beta [T, heads], state [slots, heads, dk, dv], heads a multiple of qk_rep")
+        raise KernelError("delta_scan: decay [T, heads] or [T, heads * dk], beta [T, heads], state [slots, heads, dk, dv], heads a multiple of qk_rep")
     hk = heads // qk_rep
     if max(q_off + hk * dk, k_off + hk * dk, v_off + heads * dv) > qkv.shape[1]:
         raise KernelError("delta_scan: q, k or v lie outside the rows")
     o = torch.empty((T, heads * dv), dtype=torch.float32, device=qkv.device)
-    fn = _fn("delta", "bw_delta_scan", [c_void_p, c_ll, c_int, c_int, c_int] + [c_void_p] * 6 + [c_int] * 6 + [c_void_p])
+    fn = _fn("delta", "bw_delta_scan", [c_void_p, c_ll, c_int, c_int, c_int] + [c_void_p] * 6 + [c_int] * 7 + [c_void_p])
     _check(fn(_ptr(qkv), qkv.stride(0), int(q_off), int(k_off), int(v_off), _ptr(decay), _ptr(beta), _ptr(batch.cu_q),
-              _ptr(batch.state_slot), _ptr(state), _ptr(o), batch.R, heads, int(qk_rep), dk, dv, int(T == batch.R), _stream()), "delta_scan")
+              _ptr(batch.state_slot), _ptr(state), _ptr(o), batch.R, heads, int(qk_rep), dk, dv, int(channel), int(T == batch.R),
+              _stream()), "delta_scan")
     return o
 
 
 CHUNK_MAX_KEY_DIM = 256
+CHUNK_TOKENS = 32       # tokens of a chunk
 _chunk_row = {}        # form -> floats per (token, head) of the chunked scan's scratch
 
 
@@ -1659,13 +1753,15 @@ def chunk_scan(delta: bool, qkv: torch.Tensor, q_off: int, k_off: int, v_off: in
     """The recurrences with one decay per head for portions of prompts, 32 tokens at a time with compensated tensor-core
     products (float32 state, sums and decays; a product's error about 2^-21 of it): ``delta``: as :func:`delta_scan` with
     beta = ``second``; else ``S <- g S + c k v^T, o = S^T q`` with c = ``second`` (as :func:`gla_scan` with ``scalar_decay``
-    and ``k_scale``).  ``decay``, ``second`` float32 [T, heads]; state [slots, heads, dk, >= dv]."""
+    and ``k_scale``).  ``decay``, ``second`` float32 [T, heads]; state [slots, heads, dk, >= dv].  With ``delta`` the decay may be
+    [T, heads * dk], one number per key channel."""
     _dev(qkv, "qkv", torch.float32); _dev(decay, "decay", torch.float32); _dev(second, "second", torch.float32)
     _dev(state, "state", torch.float32)
     T = qkv.shape[0]
     if dk > CHUNK_MAX_KEY_DIM:
         raise KernelError(f"chunk_scan: key size {dk} exceeds {CHUNK_MAX_KEY_DIM}")
-    if (qk_rep < 1 or heads % qk_rep or decay.shape != (T, heads) or second.shape != (T, heads) or state.dim() != 4
+    channel = delta and dk > 1 and decay.shape == (T, heads * dk)
+    if (qk_rep < 1 or heads % qk_rep or (not channel and decay.shape != (T, heads)) or second.shape != (T, heads) or state.dim() != 4
             or tuple(state.shape[1:3]) != (heads, dk) or state.shape[3] < dv or T != batch.T):
         raise KernelError("chunk_scan: decay and second [T, heads], state [slots, heads, dk, >= dv], heads a multiple of qk_rep")
     hk = heads // qk_rep
@@ -1676,10 +1772,14 @@ def chunk_scan(delta: bool, qkv: torch.Tensor, q_off: int, k_off: int, v_off: in
         n = _chunk_row[bool(delta)] = int(_fn("chunkscan", "bw_chunk_row_floats", [c_int])(int(delta)))
     rows = torch.empty((T, heads, n), dtype=torch.float32, device=qkv.device)
     o = torch.empty((T, heads * dv), dtype=torch.float32, device=qkv.device)
-    fn = _fn("chunkscan", "bw_chunk_scan", [c_int, c_void_p, c_ll, c_int, c_int, c_int] + [c_void_p] * 7 + [c_int] * 7 + [c_void_p],
-             tag=("delta" if delta else "linear") if _timings is not None else None)
-    _check(fn(int(delta), _ptr(qkv), qkv.stride(0), int(q_off), int(k_off), int(v_off), _ptr(decay), _ptr(second), _ptr(batch.cu_q),
-              _ptr(batch.state_slot), _ptr(rows), _ptr(state), _ptr(o), T, batch.R, heads, int(qk_rep),
+    chan = gend = None
+    if channel:
+        chan = torch.empty((T, heads, 3, dk), dtype=torch.float32, device=qkv.device)
+        gend = torch.empty((T // CHUNK_TOKENS + batch.R, heads, dk), dtype=torch.float32, device=qkv.device)
+    fn = _fn("chunkscan", "bw_chunk_scan", [c_int, c_void_p, c_ll, c_int, c_int, c_int] + [c_void_p] * 9 + [c_int] * 7 + [c_void_p],
+             tag=("channel" if channel else "delta" if delta else "linear") if _timings is not None else None)
+    _check(fn(2 if channel else int(delta), _ptr(qkv), qkv.stride(0), int(q_off), int(k_off), int(v_off), _ptr(decay), _ptr(second), _ptr(batch.cu_q),
+              _ptr(batch.state_slot), _ptr(rows), _ptr(chan), _ptr(gend), _ptr(state), _ptr(o), T, batch.R, heads, int(qk_rep),
               dk, dv, int(state.shape[3]), _stream()), "chunk_scan")
     return o
 
@@ -1705,7 +1805,7 @@ def ssd_out(y: torch.Tensor, x: torch.Tensor, z: torch.Tensor, D: torch.Tensor, 
 
 # ------------------------------------------------------------------ the seam between two sublayers
 
-NORM_NONE, NORM_RMS, NORM_LAYER = 0, 1, 2    # what a norm does to a row (csrc/rownorm.cu)
+NORM_NONE, NORM_RMS, NORM_LAYER, NORM_TANH = 0, 1, 2, 3    # what a norm does to a row (csrc/rownorm.cu)
 
 
 class NormedPair:
@@ -1739,7 +1839,8 @@ def row_step(stream: torch.Tensor, branch=None, post: Optional[tuple] = None, th
     """One pass over the stream (float32 [T, H]): ``stream += post(branch)`` and then ``then(stream)``, the next sublayer's
     input, which is returned.  ``branch``: a float32 tensor [T, H] (a sum that is outstanding for it is added while it is
     read) or a :class:`NormedPair`; None: nothing is added.  ``post``, ``then`` = (kind, gain, eps): kind NORM_NONE, NORM_RMS
-    or NORM_LAYER, gain float32 [H] or None; without ``then`` nothing is returned.  ``rows`` (int32): only these rows are
+    or NORM_LAYER, gain float32 [H] or None; ``then`` may also be (NORM_TANH, gain, alpha, bias): tanh(alpha x) gain + bias; without
+    ``then`` nothing is returned.  ``rows`` (int32): only these rows are
     made, and the stream is left as it is (the model's last norm on the rows whose logits are wanted)."""
     T, H = stream.shape
     y = z = (None, None, 0, 0)
@@ -1761,8 +1862,11 @@ def row_step(stream: torch.Tensor, branch=None, post: Optional[tuple] = None, th
         y = _row_source(branch, T, H, "branch")
     _dev(stream, "stream", torch.float32)
     p_kind, p_gain, p_eps = post if post is not None else (NORM_NONE, None, 0.0)
-    n_kind, n_gain, n_eps = then if then is not None else (NORM_NONE, None, 0.0)
-    for g in (p_gain, n_gain):
+    n_kind, n_gain, n_eps, *more = then if then is not None else (NORM_NONE, None, 0.0)
+    n_bias, alpha = (more[0], n_eps) if n_kind == NORM_TANH else (None, 0.0)
+    if p_kind == NORM_TANH:
+        raise KernelError("row_step: the tanh norm stands before a sublayer, not after one")
+    for g in (p_gain, n_gain, n_bias):
         if g is not None:
             _dev(g, "gain", torch.float32)
             if g.numel() != H:
@@ -1774,10 +1878,10 @@ def row_step(stream: torch.Tensor, branch=None, post: Optional[tuple] = None, th
     out = torch.empty((n, H), dtype=out_dtype or torch.float32, device=stream.device) if then is not None else None
     fn = _fn("rownorm", "bw_row_step", [c_void_p, c_int, c_void_p, c_void_p, c_ll, c_int, c_int, c_void_p, c_void_p, c_ll, c_int,
                                         c_void_p, c_void_p, c_float, c_int, c_void_p, c_float, c_int, c_void_p, c_float,
-                                        c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+                                        c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
     _check(fn(_ptr(stream), int(branch is not None), _ptr(y[0]), _ptr(y[1]), y[2], y[3], int(pair), _ptr(z[0]), _ptr(z[1]), z[2],
               z[3], _ptr(gy), _ptr(gz), pair_eps, int(p_kind), _ptr(p_gain), float(p_eps), int(n_kind), _ptr(n_gain), float(n_eps),
-              _ptr(rows), _ptr(out), _code(out, "out") if out is not None else F32, n, H, _stream()), "row_step")
+              _ptr(n_bias), float(alpha), _ptr(rows), _ptr(out), _code(out, "out") if out is not None else F32, n, H, _stream()), "row_step")
     return out
 
 
@@ -1810,10 +1914,10 @@ def moe_tc_tile_rows() -> int:
     return _moe_tc_tile
 
 
-def moe_gemm_tc_supports(H: int, F: int) -> bool:
+def moe_gemm_tc_supports(H: int, F: int, gated: bool = True) -> bool:
     """Whether the tcgen05 grouped products take an expert of size F on width H (bfloat16): inner sizes that
     are multiples of 8 (TMA rows), gate/up rows interleaved in blocks of 16.  BW_MOE_TC=0 keeps the CUDA cores."""
-    return os.environ.get("BW_MOE_TC", "1") != "0" and H % 8 == 0 and F % 16 == 0
+    return os.environ.get("BW_MOE_TC", "1") != "0" and H % 8 == 0 and F % (16 if gated else 8) == 0
 
 
 def moe_gemm_tc(a: torch.Tensor, w: torch.Tensor, tile_expert: torch.Tensor, gated: bool = False,
@@ -1821,7 +1925,8 @@ def moe_gemm_tc(a: torch.Tensor, w: torch.Tensor, tile_expert: torch.Tensor, gat
     """The grouped product on the tensor cores: a bfloat16 [tiles * 128, K], w bfloat16 [E, N, K]; row r gets
     ``a[r] @ w[e].T`` with e the expert of r's tile.  ``gated``: w's rows alternate 16 gate rows / 16 up rows
     (:func:`interleave_gate_up` per expert) and the result is bfloat16 [rows, N / 2] = silu(gate) * up, or the
-    gated activation ``act`` with its ``limit`` and ``alpha`` (:func:`glu`)."""
+    gated activation ``act`` with its ``limit`` and ``alpha`` (:func:`glu`).  Without ``gated`` a bfloat16 result may have an activation
+    of one input, ``act`` = ACT_RELU2 or ACT_GELU (ACT_SILU, the default, stands for none)."""
     _dev(a, "a", torch.bfloat16); _dev(w, "w", torch.bfloat16); _dev(tile_expert, "tile_expert", torch.int32)
     rows, K = a.shape
     E, N, K2 = w.shape
@@ -1846,10 +1951,11 @@ def moe_route(logits: torch.Tensor, top: int, softmax: bool = False, renormalize
     """float32 router logits [T, E] -> (chosen experts int32 [T, top], their weights float32 [T, top]):
     scores are sigmoid(logit) (or the softmax over the experts), the ``top`` largest are chosen (lowest
     index on ties) in falling order, optionally renormalised to sum 1 (divided by their sum + ``renorm_eps``).
+    ``softmax`` = 2 (with ``renormalize``, without a bias): the ``top`` largest logits, the weights their softmax among themselves.
     ``bias`` (float32 [E]): the choice goes by score + bias, the weights stay the scores."""
     _dev(logits, "logits", torch.float32)
     T, E = logits.shape
-    _check_route_bias(bias, E)
+    _check_route_bias(bias, E, softmax, renormalize)
     sel = torch.empty((T, top), dtype=torch.int32, device=logits.device)
     wt = torch.empty((T, top), dtype=torch.float32, device=logits.device)
     fn = _fn("moe", "bw_moe_route", [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p])
@@ -1858,7 +1964,9 @@ def moe_route(logits: torch.Tensor, top: int, softmax: bool = False, renormalize
     return sel, wt
 
 
-def _check_route_bias(bias: Optional[torch.Tensor], E: int) -> None:
+def _check_route_bias(bias: Optional[torch.Tensor], E: int, softmax: int = 0, renormalize: bool = False) -> None:
+    if int(softmax) == 2 and (bias is not None or not renormalize):
+        raise KernelError("moe_route: a softmax over the chosen logits is renormalised and takes no bias")
     if bias is not None:
         _dev(bias, "bias", torch.float32)
         if bias.numel() != E:
@@ -1878,7 +1986,7 @@ def moe_route_plan_scatter(logits: torch.Tensor, x: torch.Tensor, top: int, tile
     _dev(logits, "logits", torch.float32); _dev(x, "x")
     T, E_total = logits.shape
     E = E_total if experts is None else int(experts)
-    _check_route_bias(bias, E_total)
+    _check_route_bias(bias, E_total, softmax, renormalize)
     H = x.shape[1]
     n = T * top
     if n > MOE_FUSED_FRONT_MAX_ROWS or x.shape[0] != T:
@@ -1930,7 +2038,8 @@ def moe_scatter(x: torch.Tensor, pos_of: torch.Tensor, wt: torch.Tensor, rows: i
 def moe_gemm(a: torch.Tensor, w: torch.Tensor, tile_expert: torch.Tensor, w2: Optional[torch.Tensor] = None,
              out_dtype: Optional[torch.dtype] = None, act: int = ACT_SILU, limit: float = 0.0, alpha: float = 1.0) -> torch.Tensor:
     """Row r of the result is ``a[r] @ w[e].T`` with e the expert of r's tile; with ``w2`` it is
-    ``silu(a[r] @ w[e].T) * (a[r] @ w2[e].T)``, or the gated activation ``act`` (:func:`glu`) of the two.
+    ``silu(a[r] @ w[e].T) * (a[r] @ w2[e].T)``, or the gated activation ``act`` (:func:`glu`) of the two; without ``w2`` the
+    activation ``act`` of one input (ACT_RELU2, ACT_GELU; ACT_SILU, the default, stands for none).
     a [rows, K], w (w2) [E, N, K]."""
     _dev(a, "a"); _dev(w, "w", a.dtype); _dev(tile_expert, "tile_expert", torch.int32)
     if w2 is not None:

@@ -22,7 +22,7 @@ import torch
 
 from ..config.specs import ModelConfig
 from ..kernels import ops
-from ..parts import BuildContext, FixedStateRequest, ParamSpec, build_block, build_norm
+from ..parts import BorrowedCache, BuildContext, FixedStateRequest, ParamSpec, build_block, build_norm
 from ..parts.block import flush_hyper_write, flush_open_sums
 from ..parts.linear import Linear
 
@@ -47,6 +47,7 @@ class DecoderModel:
             if e.cache_of is not None:
                 if not 0 <= e.cache_of < pos or config.schedule[e.cache_of].cache_of is not None:
                     raise ValueError(f"schedule entry {pos}: cache_of must name an earlier entry that owns its cache")
+        self._own_requests = [self.blocks[e.layer].borrower_request() if e.cache_of is not None else None for e in config.schedule]
         self.embed: Optional[torch.Tensor] = None
         self.head: Optional[Linear] = None
         self.bigram = config.bigram_embedding
@@ -120,12 +121,14 @@ class DecoderModel:
 
     # ------------------------------------------------------------ caches
     def cache_requests(self) -> List[object]:
-        """Per schedule entry: what cache that run owns (None if it owns none; a tuple if the block keeps something
+        """Per schedule entry: what cache that run owns (None if it owns none; a run that reads another run's cache owns what its
+        block still keeps by itself; a tuple if the block keeps something
         beside its mixer's).  A model that keeps something per request itself (the previous token, for the hashed second
         embedding table) asks for it in one more entry behind the schedule's."""
         out = []
         for e in self.config.schedule:
-            out.append(None if e.cache_of is not None else self.blocks[e.layer].cache_request())
+            blk = self.blocks[e.layer]
+            out.append(blk.cache_request() if e.cache_of is None else blk.borrower_request())
         if self.bigram is not None:
             out.append(FixedStateRequest((1,), torch.int32))
         return out
@@ -148,7 +151,10 @@ class DecoderModel:
             h = ops.embed_gather(self.embed, batch.token_ids, scale=c.embedding_multiplier)
         h0 = h.clone() if self._keeps_embedding else None   # the embedding's output, for repeated passes
         for pos, e in enumerate(self.config.schedule):
-            cache = caches[e.cache_of if e.cache_of is not None else pos]
+            cache = caches[pos]
+            if e.cache_of is not None:
+                shared = caches[e.cache_of]
+                cache = shared if self._own_requests[pos] is None else BorrowedCache(shared, cache)
             blk = self.blocks[e.layer]
             if not blk.takes_pending or e.add_embedding or e.pass_input is not None:
                 ops.resolve_pending()   # the block before may have left its last sum to the next reader

@@ -80,6 +80,13 @@ class FixedStateRequest:
     dtype: torch.dtype = torch.float32
 
 
+@dataclass(frozen=True)
+class BorrowedCache:
+    """The cache view of a run that reads another run's cache and keeps something itself."""
+    shared: Any    # the other run's view
+    own: Any       # what the run asked for with ``borrower_request``
+
+
 def flatten_cache_requests(request) -> tuple:
     """A run's cache request as a tuple of single needs: a run may ask for several things at once (pages for its
     mixer and a state for the block around it) by returning a tuple; None: nothing."""
@@ -152,6 +159,11 @@ class Mixer(Part):
     #   take_projection()    hands that Linear's weight over: a wider product makes its rows from now on,
     #   from_projection(proj, batch, cache, owns_cache)   from those rows (float32) to what its output projection ``o`` reads.
 
+    def borrower_request(self):
+        """What a run that reads another run's cache (``ScheduleEntry.cache_of``) still keeps of its own; None: nothing.  With
+        something of its own, the run's cache view is a :class:`BorrowedCache`."""
+        return None
+
 
 class FeedForward(Part):
     def forward(self, x, residual, batch) -> None:
@@ -168,6 +180,11 @@ class Block(Part):
         """What a run of this block owns in the cache manager: the mixer's need, or a tuple of needs when the block
         keeps something of its own per request (the run's cache view is then a tuple in the same order)."""
         return self.mixer.cache_request()
+
+    def borrower_request(self):
+        """What a run of this block still owns when it reads another run's cache (see :class:`BorrowedCache`)."""
+        fn = getattr(self.mixer, "borrower_request", None)
+        return fn() if fn is not None else None
 
     def forward(self, residual, batch, cache, owns_cache: bool = True) -> None:
         raise NotImplementedError

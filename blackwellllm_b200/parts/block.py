@@ -17,8 +17,20 @@ from .base import (Block, BuildContext, ParamSpec, build_ffn, build_mixer, build
 
 
 class PreNormBlock(Block):
+    """``x += mixer(norm(x))``, ``x += ffn(norm(x))``.
+
+    With the layer's ``layer_scale`` (two vectors s1, s2) the outputs are multiplied channel by channel, ``x += s1 * mixer(..)``,
+    ``x += s2 * ffn(..)``, and the seams between the sublayers are one kernel each (``ops.row_step``): the scaled sum into the stream and the
+    norm before the next sublayer.  The seam behind the block's last sublayer is left to whoever reads the stream next
+    (``batch.extras["post_sum"]`` holds the output and what it is multiplied by until then): the next such block, the model's last
+    norm on the wanted rows, or :func:`flush_open_sums`.  A sublayer's output may come with its last product open, or as a pair of
+    outputs (``forward_open``): the seam's kernel takes either."""
+    seams = False
+
     def __init__(self, layer_spec, hidden_size: int, ctx: BuildContext):
         self.spec = layer_spec
+        self.hidden_size = hidden_size
+        self.ctx = ctx
         self.mixer_norm = build_norm(layer_spec.mixer_norm, hidden_size, ctx)
         self.mixer = build_mixer(layer_spec.mixer, hidden_size, ctx)
         self.ffn = None
@@ -26,6 +38,20 @@ class PreNormBlock(Block):
         if layer_spec.ffn is not None:
             self.ffn_norm = build_norm(layer_spec.ffn_norm, hidden_size, ctx)
             self.ffn = build_ffn(layer_spec.ffn, hidden_size, ctx)
+        self.scale_names = getattr(layer_spec, "layer_scale", None)
+        self.posts = []        # with seams: (kind, gain or scale, eps) after the mixer, after the feed-forward
+        if self.scale_names is not None and layer_spec.block == "prenorm":
+            self._use_seams()
+
+    def _use_seams(self) -> None:
+        if not all(hasattr(n, "row_norm") for n in self._norms()):
+            raise ValueError("a layer scale or a constant on the sublayers' outputs needs norms that describe themselves (row_norm)")
+        self.seams = True
+        self.takes_pending = True
+        self.takes_open = ("post_sum",)
+
+    def _norms(self) -> list:
+        return [n for n in (self.mixer_norm, self.ffn_norm) if n is not None]
 
     def _children(self):
         s = self.spec
@@ -34,16 +60,35 @@ class PreNormBlock(Block):
             kids += [(s.ffn_norm_prefix, self.ffn_norm), (s.ffn_prefix, self.ffn)]
         return kids
 
+    def _unused_params(self) -> List[ParamSpec]:
+        """A layer without a feed-forward may still store the second scale and the norms around it: taken and not used."""
+        s, out = self.spec, []
+        if self.ffn is None:
+            for norm, prefix in ((s.ffn_norm, s.ffn_norm_prefix), (s.ffn_post_norm, s.ffn_post_norm_prefix)):
+                if norm is not None:
+                    out += [ParamSpec(prefix + p.name, p.shape, p.role, p.init, True)
+                            for p in build_norm(norm, self.hidden_size, self.ctx).param_specs()]
+        return out
+
+    def _scale_params(self) -> List[ParamSpec]:
+        return [ParamSpec(name, (self.hidden_size,), role="gain", init="ones", optional=k == 1 and self.ffn is None)
+                for k, name in enumerate((self.scale_names or ())[:2])]
+
     def param_specs(self) -> List[ParamSpec]:
         out = []
         for prefix, part in self._children():
             for p in part.param_specs():
                 out.append(ParamSpec(prefix + p.name, p.shape, p.role, p.init, p.optional))
+        if self.spec.block == "prenorm":
+            out += self._scale_params() + self._unused_params()
         return out
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         for prefix, part in self._children():
             part.bind({k[len(prefix):]: v for k, v in tensors.items() if k.startswith(prefix)})
+        if self.seams:
+            self.posts = [(ops.NORM_NONE, tensors[name].float().contiguous(), 0.0)
+                          for name in self.scale_names[:1 if self.ffn is None else 2]]
 
     takes_pending = True
 
@@ -56,11 +101,30 @@ class PreNormBlock(Block):
         return norm.forward(residual)
 
     def forward(self, residual, batch, cache, owns_cache: bool = True) -> None:
+        if self.seams:
+            return self._forward_seams(residual, batch, cache, owns_cache)
         x = self._normed(self.mixer_norm, residual)
         self.mixer.forward(x, residual, batch, cache, owns_cache)
         if self.ffn is not None:
             x = self._normed(self.ffn_norm, residual)
             self.ffn.forward(x, residual, batch)
+
+    def _forward_seams(self, residual, batch, cache, owns_cache) -> None:
+        dtype = self.ctx.dtype
+        branch, post = batch.extras.pop("post_sum", (None, None))      # what the block before left
+        x = ops.row_step(residual, branch, post, then=self.mixer_norm.row_norm(), out_dtype=dtype)
+        if hasattr(self.mixer, "forward_open"):
+            y = self.mixer.forward_open(x, batch, cache, owns_cache)
+        else:
+            y = torch.empty_like(residual)
+            self.mixer.forward(x, y, batch, cache, owns_cache, accumulate=None)
+        post = self.posts[0]
+        if self.ffn is not None:
+            x = ops.row_step(residual, y, post, then=self.ffn_norm.row_norm(), out_dtype=dtype)
+            y = torch.empty_like(residual)
+            self.ffn.forward(x, y, batch, accumulate=None)
+            post = self.posts[1]
+        batch.extras["post_sum"] = (y, post)
 
 
 class SandwichBlock(PreNormBlock):
@@ -69,13 +133,9 @@ class SandwichBlock(PreNormBlock):
     it and adds the result to the stream in one kernel.  A feed-forward with ``forward_post`` does the
     second norm inside its own last kernel.
 
-    With the layer's ``layer_scale`` (two vectors), a ``residual_mult`` other than 1 or layer norms, the arrangement is
-    ``x += mult * s1 * post(mixer(pre(x)))`` and so on, and the seams between the sublayers are one kernel each
-    (``ops.row_step``): the norm of a sublayer's output with scale and constant in its gain, the sum into the stream, and the
-    norm before the next sublayer.  The seam behind the block's last sublayer is left to whoever reads the stream next
-    (``batch.extras["post_sum"]`` holds the output and its norm until then): the next such block, the model's last norm on
-    the wanted rows, or :func:`flush_open_sums`.  A sublayer's output may come with its last product open, or as a pair of
-    outputs (``forward_open``): the seam's kernel takes either."""
+    With the layer's ``layer_scale``, a ``residual_mult`` other than 1 or layer norms, the arrangement is
+    ``x += mult * s1 * post(mixer(pre(x)))`` and so on, with the seams of :class:`PreNormBlock`: the norm of a sublayer's output, with
+    scale and constant in its gain, runs in the seam's kernel too."""
     takes_pending = False
 
     def __init__(self, layer_spec, hidden_size: int, ctx: BuildContext):
@@ -87,19 +147,13 @@ class SandwichBlock(PreNormBlock):
         for norm in (self.mixer_post, self.ffn_post):
             if norm is not None and not hasattr(norm, "add_to"):
                 raise ValueError(f"{type(norm).__name__} cannot follow a sublayer (it has no add_to)")
-        self.hidden_size = hidden_size
-        self.ctx = ctx
-        self.scale_names = getattr(layer_spec, "layer_scale", None)
         self.mult = float(getattr(layer_spec, "residual_mult", 1.0))
         from .norm import LayerNorm
-        norms = [n for n in (self.mixer_norm, self.mixer_post, self.ffn_norm, self.ffn_post) if n is not None]
-        self.seams = self.scale_names is not None or self.mult != 1.0 or any(isinstance(n, LayerNorm) for n in norms)
-        self.posts = []        # with seams: (kind, gain with layer scale and constant, eps) after the mixer, after the feed-forward
-        if self.seams:
-            if not all(hasattr(n, "row_norm") for n in norms):
-                raise ValueError("a layer scale or a constant on the sublayers' outputs needs norms that describe themselves (row_norm)")
-            self.takes_pending = True
-            self.takes_open = ("post_sum",)
+        if self.scale_names is not None or self.mult != 1.0 or any(isinstance(n, LayerNorm) for n in self._norms()):
+            self._use_seams()
+
+    def _norms(self) -> list:
+        return super()._norms() + [n for n in (self.mixer_post, self.ffn_post) if n is not None]
 
     def _children(self):
         s = self.spec
@@ -109,21 +163,11 @@ class SandwichBlock(PreNormBlock):
         return kids
 
     def param_specs(self) -> List[ParamSpec]:
-        out = super().param_specs()
-        if self.scale_names is not None:
-            for k, name in enumerate(self.scale_names[:2]):
-                # (a layer without a feed-forward may still store the second vector, and the norms: taken and not used)
-                out.append(ParamSpec(name, (self.hidden_size,), role="gain", init="ones", optional=k == 1 and self.ffn is None))
-        if self.ffn is None:
-            s = self.spec
-            for norm, prefix in ((s.ffn_norm, s.ffn_norm_prefix), (s.ffn_post_norm, s.ffn_post_norm_prefix)):
-                if norm is not None:
-                    out.append(ParamSpec(prefix + getattr(norm, "param", "weight"), (self.hidden_size,), role="gain", init="ones",
-                                         optional=True))
-        return out
+        return super().param_specs() + self._scale_params() + self._unused_params()
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
-        super().bind(tensors)
+        for prefix, part in self._children():
+            part.bind({k[len(prefix):]: v for k, v in tensors.items() if k.startswith(prefix)})
         if self.seams:
             self.posts = []
             for k, norm in enumerate((self.mixer_post, self.ffn_post)):
@@ -154,23 +198,6 @@ class SandwichBlock(PreNormBlock):
             else:
                 self.ffn.forward(x, branch, batch, accumulate=False)
                 self.ffn_post.add_to(branch, residual)
-
-    def _forward_seams(self, residual, batch, cache, owns_cache) -> None:
-        dtype = self.ctx.dtype
-        branch, post = batch.extras.pop("post_sum", (None, None))      # what the block before left
-        x = ops.row_step(residual, branch, post, then=self.mixer_norm.row_norm(), out_dtype=dtype)
-        if hasattr(self.mixer, "forward_open"):
-            y = self.mixer.forward_open(x, batch, cache, owns_cache)
-        else:
-            y = torch.empty_like(residual)
-            self.mixer.forward(x, y, batch, cache, owns_cache, accumulate=None)
-        post = self.posts[0]
-        if self.ffn is not None:
-            x = ops.row_step(residual, y, post, then=self.ffn_norm.row_norm(), out_dtype=dtype)
-            y = torch.empty_like(residual)
-            self.ffn.forward(x, y, batch, accumulate=None)
-            post = self.posts[1]
-        batch.extras["post_sum"] = (y, post)
 
 
 register_block("prenorm", PreNormBlock)

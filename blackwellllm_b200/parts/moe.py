@@ -1,6 +1,7 @@
 """Routed feed-forward (mixture of experts).
 
     z = W_r x (float32)      s = sigmoid(z) or softmax(z)      the top_k largest s are chosen
+                             (or: the top_k largest z, s their softmax among themselves)
     y = sum over chosen e of  s_e * expert_e(x)      or, with scale_input,  expert_e(s_e * x)
     expert(u) = W_down (silu(W_gate u) * (W_up u))
 
@@ -18,7 +19,7 @@ the renormalising sum (``renorm_eps``); router outputs beyond the experts that s
 their input (``identity_experts``: such a choice takes no row in the regrouping, the summing kernel adds
 weight * x for it); another gated activation for the experts (``activation``, run in the first product's
 epilogue like the default); and a shared expert (``shared``: a dense gated feed-forward that every token runs
-through and whose result is added).
+through and whose result is added); and experts without a gate, down(act(up u)), act the squared positive part or gelu.
 """
 from __future__ import annotations
 
@@ -36,10 +37,10 @@ class RoutedFFN(FeedForward):
         self.E, self.top, self.F = int(spec.num_experts), int(spec.top_k), int(spec.expert_size)
         if not 0 < self.top <= self.E + int(getattr(spec, "identity_experts", 0) or 0):
             raise ValueError(f"top_k {self.top} must be in 1..{self.E} (plus the experts that return their input)")
-        if spec.score not in ("sigmoid", "softmax"):
+        if spec.score not in ("sigmoid", "softmax", "softmax_chosen"):
             raise ValueError(f"unknown router score {spec.score!r}")
-        self.softmax = spec.score == "softmax"
-        self.renormalize, self.scale_input = bool(spec.renormalize), bool(spec.scale_input)
+        self.softmax = {"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}[spec.score]
+        self.renormalize, self.scale_input = bool(spec.renormalize) or self.softmax == 2, bool(spec.scale_input)
         self.hidden_size = hidden_size
         self.ctx = ctx
         self.router_name = spec.router_name
@@ -51,9 +52,13 @@ class RoutedFFN(FeedForward):
         self.bias_name = getattr(spec, "choice_bias", None)
         self.renorm_eps = float(getattr(spec, "renorm_eps", 0.0))
         activation = getattr(spec, "activation", "silu")
-        if activation not in ops.GATED_ACTIVATIONS:
-            raise ValueError(f"unknown gated activation {activation!r}; known: {sorted(ops.GATED_ACTIVATIONS)}")
-        self.act = ops.GATED_ACTIVATIONS[activation]
+        self.gated = activation not in ops.UNARY_ACTIVATIONS
+        known = {**ops.GATED_ACTIVATIONS, **ops.UNARY_ACTIVATIONS}
+        if activation not in known:
+            raise ValueError(f"unknown activation {activation!r}; known: {sorted(known)}")
+        if self.softmax == 2 and self.bias_name:
+            raise ValueError("a softmax over the chosen logits goes without a bias on the choice")
+        self.act = known[activation]
         self.limit, self.alpha = float(getattr(spec, "act_limit", 0.0)), float(getattr(spec, "act_alpha", 1.0))
         self.shared = None
         self.shared_prefix = getattr(spec, "shared_prefix", "shared.")
@@ -77,8 +82,8 @@ class RoutedFFN(FeedForward):
         if self.shared is not None:
             specs += [ParamSpec(self.shared_prefix + p.name, p.shape, p.role, p.init, p.optional) for p in self.shared.param_specs()]
         for e in range(self.E):
-            specs += [ParamSpec(self._expert(e, self.gate_name), (F, H)), ParamSpec(self._expert(e, self.up_name), (F, H)),
-                      ParamSpec(self._expert(e, self.down_name), (H, F))]
+            specs += ([ParamSpec(self._expert(e, self.gate_name), (F, H))] if self.gated else []) + [
+                ParamSpec(self._expert(e, self.up_name), (F, H)), ParamSpec(self._expert(e, self.down_name), (H, F))]
         return specs
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
@@ -91,8 +96,10 @@ class RoutedFFN(FeedForward):
         stack = lambda which: torch.stack([tensors[self._expert(e, which)] for e in range(self.E)]).contiguous()
         self.w_down = stack(self.down_name)
         self.tc = (self.w_down.dtype == torch.bfloat16 and self.w_down.is_cuda
-                   and ops.moe_gemm_tc_supports(self.hidden_size, self.F))
-        if self.tc:   # one gate/up tensor whose rows alternate in blocks of 16: the activation runs in the product's epilogue
+                   and ops.moe_gemm_tc_supports(self.hidden_size, self.F, self.gated))
+        if not self.gated:
+            self.w_up = stack(self.up_name)
+        elif self.tc:   # one gate/up tensor whose rows alternate in blocks of 16: the activation runs in the product's epilogue
             self.w_gate_up = torch.stack([ops.interleave_gate_up(tensors[self._expert(e, self.gate_name)],
                                                                  tensors[self._expert(e, self.up_name)])
                                           for e in range(self.E)]).contiguous()
@@ -111,7 +118,11 @@ class RoutedFFN(FeedForward):
             sel, wt = ops.moe_route(logits, self.top, self.softmax, self.renormalize, self.bias, self.renorm_eps)
             pos_of, tile_expert = ops.moe_plan(sel, self.E, tile)
             xs = ops.moe_scatter(x, pos_of, wt, tile_expert.numel() * tile, self.scale_input)
-        if self.tc:
+        if not self.gated:
+            product = ops.moe_gemm_tc if self.tc else ops.moe_gemm
+            a = product(xs, self.w_up, tile_expert, act=self.act)
+            y = product(a, self.w_down, tile_expert, out_dtype=torch.float32)
+        elif self.tc:
             a = ops.moe_gemm_tc(xs, self.w_gate_up, tile_expert, gated=True, act=self.act, limit=self.limit, alpha=self.alpha)
             y = ops.moe_gemm_tc(a, self.w_down, tile_expert, out_dtype=torch.float32)
         else:

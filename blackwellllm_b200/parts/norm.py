@@ -8,8 +8,10 @@ positions whose logits are wanted, src/core/engine.cpp:1029-1035).  With the spe
 
 :class:`LayerNorm`: (x - mean) / sqrt(mean((x - mean)^2) + eps) * w, no bias, everything float32.
 
-Both describe themselves to kernels that norm a row inside another pass over it (``row_norm``: the kind, the float32
-gain and eps, as ``ops.row_step`` takes them).
+:class:`DynamicTanh`: tanh(alpha x) * w + b with a number alpha and a vector b stored beside the weight; no statistic of the row.
+
+All describe themselves to kernels that norm a row inside another pass over it (``row_norm``: the kind, the float32
+gain and eps, or for the last one (kind, gain, alpha, bias), as ``ops.row_step`` takes them).
 """
 from __future__ import annotations
 
@@ -91,5 +93,32 @@ class LayerNorm(Norm):
         return ops.row_step(x, then=self.row_norm(), rows=rows, out_dtype=self.ctx.dtype)
 
 
+class DynamicTanh(Norm):
+    def __init__(self, spec, hidden_size: int, ctx: BuildContext):
+        self.hidden_size = hidden_size
+        self.ctx = ctx
+        self.names = (spec.param, spec.alpha_param, spec.bias_param)
+        self.gain: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+        self.alpha = 1.0
+
+    def param_specs(self) -> List[ParamSpec]:
+        w, alpha, b = self.names
+        return [ParamSpec(w, (self.hidden_size,), role="gain", init="ones"), ParamSpec(alpha, (), role="gain", init="ones"),
+                ParamSpec(b, (self.hidden_size,), role="bias", init="bias_normal")]
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        w, alpha, b = self.names
+        self.gain, self.bias = tensors[w].float().contiguous(), tensors[b].float().contiguous()
+        self.alpha = float(tensors[alpha])
+
+    def row_norm(self) -> tuple:
+        return ops.NORM_TANH, self.gain, self.alpha, self.bias
+
+    def forward(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        return ops.row_step(x, then=self.row_norm(), rows=rows, out_dtype=self.ctx.dtype)
+
+
 register_norm("rmsnorm", RMSNorm)
 register_norm("layernorm", LayerNorm)
+register_norm("dynamic_tanh", DynamicTanh)
