@@ -438,9 +438,42 @@ ZANIVIK_SHAPES = {
     "2k": (2048, 16, 4, 128, 1024, 16, 8, 128, 128, 64, 64, 128, 4, 8192, (16, 128, 128), 32000, 2),
     "4k": (4096, 32, 8, 128, 1024, 32, 16, 128, 128, 128, 64, 128, 8, 16384, (32, 128, 128), 32000, 2),
 }
+
+
+def _zogulorn_shape(width, heads, kv, hd, block, d_heads, d_kv, d_dk, d_dv, rank, a_heads, a_kv, a_dim, a_vdim, ff, experts, top, e_ff, vocab,
+                    like):
+    """Four layers: twice rotary attention in blocks beside the delta rule with a decay per key channel, twice differential
+    attention with short convolutions, the second reading the first one's keys and values; a dense gated and a routed
+    feed-forward in turn.  Beside it the dense decoder of equal width, depth and heads with the dense feed-forward, and the
+    closest designs the engine had before: Zanivik (attention and the delta rule side by side, a kernel per seam) and Gafulix
+    (block-masked attention, a recurrence with a decay per key channel, experts) at the same heads and state sizes."""
+    mask = {"size": block}
+    par = {"left": {"heads": heads, "kv_heads": kv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": mask,
+                    "rot": {"base": 10000.0, "dims": hd}},
+           "right": {"heads": d_heads, "kv_heads": d_kv, "dim": d_dk, "vdim": d_dv, "conv": 4, "decay_rank": rank, "gate_rank": rank},
+           "left_scale": 0.7, "right_scale": 0.6}
+    att = {"heads": a_heads, "kv_heads": a_kv, "dim": a_dim, "vdim": a_vdim, "scale": a_dim ** -0.5, "mask": mask, "conv": 4, "diff": 0.6}
+    mlp = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": e_ff}, "router": {"experts": experts, "top": top}}
+    design = {"architecture": "Zogulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+              "layers": [{"type": "parallel", "mixer": par, "mlp": mlp}, {"type": "parallel", "mixer": par, "mlp": moe},
+                         {"type": "attention", "mixer": att, "mlp": mlp},
+                         {"type": "attention", "mixer": dict(att, kv_from=2), "mlp": moe}]}
+    zanivik, dense, more = _zanivik_shape(*ZANIVIK_SHAPES[like])
+    dense["intermediate_size"] = ff
+    gafulix, _ = _gafulix_shape(width, heads, kv, hd, d_heads, d_dk, d_dv, experts, top, e_ff * 2 // 3 // 64 * 64, block, vocab, 2)
+    return design, dense, {"zanivik": zanivik, "gafulix": gafulix}
+
+
+ZOGULORN_SHAPES = {
+    # width, left: heads, kv heads, head size, block of positions; right: heads, query/key heads, key size, value size, inner size;
+    # differential attention: heads, kv heads, size of a map, value size; feed-forward size, experts, top, expert size, vocab
+    "2k": (2048, 16, 4, 128, 1024, 16, 8, 128, 128, 128, 16, 4, 64, 128, 5632, 16, 2, 2048, 32000, "2k"),
+    "4k": (4096, 32, 8, 128, 1024, 32, 16, 128, 128, 128, 32, 8, 64, 128, 11008, 8, 2, 5632, 32000, "4k"),
+}
 DESIGNS = {"gafulix": (_gafulix_shape, DESIGN_SHAPES), "fuvevik": (_fuvevik_shape, FUVEVIK_SHAPES),
            "zigipel": (_zigipel_shape, ZIGIPEL_SHAPES), "vubotar": (_vubotar_shape, VUBOTAR_SHAPES),
-           "zanivik": (_zanivik_shape, ZANIVIK_SHAPES)}
+           "zanivik": (_zanivik_shape, ZANIVIK_SHAPES), "zogulorn": (_zogulorn_shape, ZOGULORN_SHAPES)}
 
 
 def design_comparison(args):

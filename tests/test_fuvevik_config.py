@@ -205,4 +205,4 @@ def test_routed_feed_forward_options_are_checked():
     with pytest.raises(ValueError):
         build_ffn(RoutedFFNSpec(4, 2, 16, identity_experts=2, scale_input=True), 32, ctx)
     with pytest.raises(ValueError):
-        build_ffn(RoutedFFNSpec(4, 2, 16, activation="gelu"), 32, ctx)
+        build_ffn(RoutedFFNSpec(4, 2, 16, activation="softsign"), 32, ctx)
