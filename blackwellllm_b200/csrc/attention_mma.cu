@@ -64,6 +64,7 @@ struct Params {
     // own position writes the rotated key and the value to the cache.  Every request has one token.
     const float* qkv; long long qkv_plane_stride; const float* rope_table;
     int qkv_planes, rd, append;
+    bw::DiffHeads diff;           // diff.lam != null: pairs of query heads become one head (G even; the gate has one number per head)
 };
 
 // The sink's term of a row's denominator, in the units of the running sums (powers of two, maximum M taken off).
@@ -395,6 +396,32 @@ attn_rows_kernel(Params p, int toks_per_tile) {
         l += __shfl_xor_sync(0xffffffffu, l, 1);
         l += __shfl_xor_sync(0xffffffffu, l, 2);
         const int row = warp * 16 + (lane >> 2) + 8 * h;
+        if (p.diff.lam) {
+            // the maps of a head are neighbouring rows: lanes four apart; each writes half of the head's channels
+            const bool odd = row & 1;
+            const float mine = bw::diff_weight(p.diff, odd, l > 0.f ? 1.f / l : 0.f);
+            const int tok = row / p.G, head = (g * p.G + row - tok * p.G) >> 1;
+            const size_t token = (size_t)(p.cu_q[r] + tok0 + tok);
+            float ss = 0.f;
+#pragma unroll
+            for (int j = 0; j < HD / 8; ++j)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const float own = o[j][2 * h + e] * mine;
+                    o[j][2 * h + e] = own + __shfl_xor_sync(0xffffffffu, own, 4);
+                    ss = fmaf(o[j][2 * h + e], o[j][2 * h + e], ss);
+                }
+            ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+            ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+            if (row >= n_rows) continue;
+            const float f = bw::diff_factor(p.diff, ss, p.gate, p.gate_ld, token, head);
+            bf16* dst = p.out + (token * (p.nh >> 1) + head) * HD + 2 * (lane & 3);
+#pragma unroll
+            for (int j = 0; j < HD / 8; ++j)
+                if ((j & 1) == odd)
+                    *reinterpret_cast<__nv_bfloat162*>(dst + j * 8) = __floats2bfloat162_rn(o[j][2 * h] * f, o[j][2 * h + 1] * f);
+            continue;
+        }
         if (row >= n_rows) continue;
         const int tok = row / p.G, hg = row - tok * p.G;
         l += sink_term(p, g * p.G + hg, st.m[h]);
@@ -409,6 +436,50 @@ attn_rows_kernel(Params p, int toks_per_tile) {
                 __floats2bfloat162_rn(o[j][2 * h] * inv * bw::out_gate(p.gate, p.gate_ld, p.gate_dv, token, head, c),
                                       o[j][2 * h + 1] * inv * bw::out_gate(p.gate, p.gate_ld, p.gate_dv, token, head, c + 1));
         }
+    }
+}
+
+// The end of a key-slice CTA that has a request's only slice, where pairs of query heads become one (bw::DiffHeads): a warp per head.
+__device__ __forceinline__ void finish_pairs(const Params& p, const float* ms, const float* ls, const float* os, int r, int g, int n_rows) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    constexpr int PER = (HD + 31) / 32;
+    for (int pair = warp; 2 * pair < n_rows; pair += NWARPS) {
+        float o[PER];
+#pragma unroll
+        for (int i = 0; i < PER; ++i) o[i] = 0.f;
+#pragma unroll
+        for (int which = 0; which < 2; ++which) {
+            const int row = 2 * pair + which;
+            float M = -INFINITY, L = 0.f, f[NWARPS];
+#pragma unroll
+            for (int wv = 0; wv < NWARPS; ++wv) M = fmaxf(M, ms[wv * 16 + row]);
+#pragma unroll
+            for (int wv = 0; wv < NWARPS; ++wv) {
+                f[wv] = ms[wv * 16 + row] == -INFINITY ? 0.f : exp2f(ms[wv * 16 + row] - M);
+                L += ls[wv * 16 + row] * f[wv];
+            }
+            const float mine = bw::diff_weight(p.diff, which, L > 0.f ? 1.f / L : 0.f);
+#pragma unroll
+            for (int i = 0; i < PER; ++i) {
+                const int c = lane + 32 * i;
+                if (c >= HD) break;
+                float acc = 0.f;
+#pragma unroll
+                for (int wv = 0; wv < NWARPS; ++wv) acc += os[((size_t)(wv * 16 + row)) * HD + c] * f[wv];
+                o[i] = fmaf(acc, mine, o[i]);
+            }
+        }
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) ss = fmaf(o[i], o[i], ss);
+        ss = bw::warp_sum(ss);
+        const int tok = 2 * pair / p.G, head = (g * p.G + 2 * pair - tok * p.G) >> 1;
+        const size_t token = (size_t)(p.cu_q[r] + tok);
+        const float f = bw::diff_factor(p.diff, ss, p.gate, p.gate_ld, token, head);
+        bf16* dst = p.out + (token * (p.nh >> 1) + head) * HD;
+#pragma unroll
+        for (int i = 0; i < PER; ++i)
+            if (lane + 32 * i < HD) dst[lane + 32 * i] = __float2bfloat16_rn(o[i] * f);
     }
 }
 
@@ -436,6 +507,10 @@ __device__ __forceinline__ void finish_keys(const Params& p, const RowState& st,
         }
     }
     sync_compute_warps();
+    if (p.diff.lam && n_slices == 1) {
+        finish_pairs(p, ms, ls, os, r, g, n_rows);
+        return;
+    }
     for (int idx = threadIdx.x; idx < n_rows * HD; idx += THREADS) {
         const int row = idx / HD, c = idx - row * HD;
         float M = -INFINITY;
@@ -954,6 +1029,87 @@ attn_merge_few_kernel(Params p, const int* merge_items) {
     *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
 }
 
+// The merge where pairs of query heads become one (bw::DiffHeads): grid (sliced items, nkv, 8 pairs), half a CTA per row of the pair,
+// the slices of a row summed as in attn_merge_kernel; then one warp makes the head of the two.
+constexpr int PAIR_THREADS = 128;
+constexpr int PAIR_GROUPS = PAIR_THREADS / MERGE_QUADS < MAX_SLICES ? PAIR_THREADS / MERGE_QUADS : MAX_SLICES;
+__global__ void __launch_bounds__(2 * PAIR_THREADS)
+attn_merge_pairs_kernel(Params p, const int* merge_items) {
+    BW_PDL_TRIGGER();
+    const int4 w = reinterpret_cast<const int4*>(merge_items)[blockIdx.x];
+    const int r = w.x, n_slices = w.z, item = w.w, g = blockIdx.y, pair = blockIdx.z;
+    BW_PDL_WAIT();
+    const int n_rows = (p.cu_q[r + 1] - p.cu_q[r]) * p.G;
+    if (2 * pair >= n_rows) return;
+    __shared__ float sm_m[2][MAX_SLICES], sm_l[2][MAX_SLICES];
+    __shared__ float4 red[2][PAIR_GROUPS][MERGE_QUADS];
+    const int which = threadIdx.x / PAIR_THREADS, tid = threadIdx.x % PAIR_THREADS;
+    const size_t base0 = ((size_t)item * p.nkv + (size_t)g * n_slices) * 16 + 2 * pair + which;
+    const int quad = tid % MERGE_QUADS, group = tid / MERGE_QUADS;
+    constexpr int AHEAD = 8;
+    float4 part[AHEAD];       // the first loads do not wait for the maxima
+    if (group < PAIR_GROUPS) {
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+            const int sl = group + i * PAIR_GROUPS;
+            part[i] = sl < n_slices ? reinterpret_cast<const float4*>(p.part_o + (base0 + (size_t)sl * 16) * HD)[quad]
+                                    : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    }
+    if (tid < n_slices) {
+        const float2 ml = reinterpret_cast<const float2*>(p.part_ml)[base0 + (size_t)tid * 16];
+        sm_m[which][tid] = ml.x; sm_l[which][tid] = ml.y;
+    }
+    __syncthreads();
+    float M = -INFINITY, L = 0.f;
+    for (int sl = 0; sl < n_slices; ++sl) M = fmaxf(M, sm_m[which][sl]);
+    auto factor = [&](int sl) { return sm_m[which][sl] == -INFINITY ? 0.f : exp2f(sm_m[which][sl] - M); };
+    for (int sl = 0; sl < n_slices; ++sl) L += sm_l[which][sl] * factor(sl);
+    const float mine = bw::diff_weight(p.diff, which, L > 0.f ? 1.f / L : 0.f);
+    if (group < PAIR_GROUPS) {
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+        auto add = [&](const float4& v, int sl) {
+            const float f = factor(sl);
+            acc.x += v.x * f; acc.y += v.y * f; acc.z += v.z * f; acc.w += v.w * f;
+        };
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i)
+            if (group + i * PAIR_GROUPS < n_slices) add(part[i], group + i * PAIR_GROUPS);
+        for (int sl = group + AHEAD * PAIR_GROUPS; sl < n_slices; sl += PAIR_GROUPS)
+            add(reinterpret_cast<const float4*>(p.part_o + (base0 + (size_t)sl * 16) * HD)[quad], sl);
+        red[which][group][quad] = make_float4(acc.x * mine, acc.y * mine, acc.z * mine, acc.w * mine);
+    }
+    __syncthreads();
+    if (threadIdx.x >= 32) return;
+    constexpr int PER = (MERGE_QUADS + 31) / 32;
+    float4 o[PER];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int q = threadIdx.x + 32 * i;
+        o[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (q < MERGE_QUADS) {
+            for (int m = 0; m < 2; ++m)
+                for (int j = 0; j < PAIR_GROUPS; ++j) {
+                    const float4 v = red[m][j][q];
+                    o[i].x += v.x; o[i].y += v.y; o[i].z += v.z; o[i].w += v.w;
+                }
+        }
+        ss = fmaf(o[i].x, o[i].x, ss); ss = fmaf(o[i].y, o[i].y, ss); ss = fmaf(o[i].z, o[i].z, ss); ss = fmaf(o[i].w, o[i].w, ss);
+    }
+    ss = bw::warp_sum(ss);
+    const int tok = 2 * pair / p.G, head = (g * p.G + 2 * pair - tok * p.G) >> 1;
+    const size_t token = (size_t)(p.cu_q[r] + tok);
+    const float f = bw::diff_factor(p.diff, ss, p.gate, p.gate_ld, token, head);
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int q = threadIdx.x + 32 * i;
+        if (q < MERGE_QUADS)
+            *reinterpret_cast<uint2*>(p.out + (token * (p.nh >> 1) + head) * HD + q * 4) =
+                make_uint2(pack_bf16(o[i].x * f, o[i].y * f), pack_bf16(o[i].z * f, o[i].w * f));
+    }
+}
+
 constexpr int SMEM_ROWS = (BN + 4 * BN) * ROW_BYTES;     // q tile of 64 rows + 2 stages of K and V
 constexpr int SMEM_KEYS_LOOP = (16 + 4 * BN) * ROW_BYTES;
 constexpr int SMEM_KEYS_MERGE = SMEM_KEYS_MERGE_BYTES;
@@ -974,7 +1130,8 @@ BW_EXPORT int bw_attention_head_dim() { return HD; }
 // rope_table float32 [tokens][rd] (cosines, then sines); append != 0: key and value also go to the cache.
 // sink: float32 [nh] or null; gate: float32 [tokens, >= nh * gate_dv] with rows gate_ld apart, or null (see Params);
 // gate_dv < 0: one gate number per head (bw::out_gate).  dist: float32 [2][nh] or null; keep_first: see Params.
-// softcap (> 0: on), rel, rel_len: see Params; not together with dist, nor with qkv.
+// softcap (> 0: on), rel, rel_len: see Params; not together with dist, nor with qkv.  lam != null: pairs of query heads become one
+// (bw::DiffHeads: one float32 number on the device, diff_eps, diff_scale, diff_dv; no sink); out is then [tokens, nh / 2 * HD].
 // qkv only where the TMA key-slice kernel runs (head size a multiple of 64, pages of 8 to 64 tokens);
 // BW_ERR_UNSUPPORTED otherwise, and nothing was launched.
 BW_EXPORT int bw_attention_mma(const void* q, const void* k_pages, const void* v_pages, void* out, const int* cu_q,
@@ -985,7 +1142,7 @@ BW_EXPORT int bw_attention_mma(const void* q, const void* k_pages, const void* v
                                const float* qkv, int qkv_planes, long long qkv_plane_stride, const float* rope_table,
                                int rd, int append, int merge_max_slices, const float* sink, const float* gate, long long gate_ld,
                                int gate_dv, const float* dist, int keep_first, float softcap, const float* rel, int rel_len,
-                               void* stream) {
+                               const float* lam, float diff_eps, float diff_scale, int diff_dv, void* stream) {
     if (nkv <= 0 || nh % nkv != 0) return BW_ERR_BAD_ARG;
     if ((rel && rel_len <= 0) || ((rel || softcap > 0.f) && (dist || qkv))) return BW_ERR_UNSUPPORTED;
     const int G = nh / nkv;
@@ -1013,7 +1170,9 @@ BW_EXPORT int bw_attention_mma(const void* q, const void* k_pages, const void* v
     p.dist = dist; p.keep_first = (keep_first > 0 && window > 0) ? keep_first : 0;
     p.softcap = softcap > 0.f ? softcap : 0.f; p.rel = rel; p.rel_len = rel_len;
     if (qkv && (dist || p.keep_first)) return BW_ERR_UNSUPPORTED;
-    if (gate && gate_dv < 0 ? (-gate_dv > HD || gate_ld < (long long)nh)
+    if (lam && (G % 2 || diff_dv <= 0 || diff_dv > HD || (gate && gate_dv >= 0) || sink || qkv)) return BW_ERR_BAD_ARG;
+    p.diff.lam = lam; p.diff.eps = diff_eps; p.diff.scale = diff_scale; p.diff.dv = diff_dv;
+    if (gate && gate_dv < 0 ? (-gate_dv > HD || gate_ld < (long long)(lam ? nh / 2 : nh))
                             : gate && (gate_dv <= 0 || gate_dv > HD || gate_ld < (long long)nh * gate_dv)) return BW_ERR_BAD_ARG;
     p.gate = gate; p.gate_ld = gate_ld; p.gate_dv = gate_dv;
     p.qkv = qkv; p.qkv_plane_stride = qkv_plane_stride; p.rope_table = rope_table;
@@ -1048,7 +1207,9 @@ BW_EXPORT int bw_attention_mma(const void* q, const void* k_pages, const void* v
         }
         if (n_merge_items > 0) {
             // merge_max_slices: the most slices of any merge item (0: unknown)
-            if (merge_max_slices > 0 && merge_max_slices <= MERGE_FEW && 16 * MERGE_QUADS <= 1024)
+            if (lam)
+                bw::launch((attn_merge_pairs_kernel), dim3(n_merge_items, nkv, 8), dim3(2 * PAIR_THREADS), 0, s, p, merge_work);
+            else if (merge_max_slices > 0 && merge_max_slices <= MERGE_FEW && 16 * MERGE_QUADS <= 1024)
                 bw::launch((attn_merge_few_kernel), dim3(n_merge_items, nkv), dim3(16 * MERGE_QUADS), 0, s, p, merge_work);
             else
                 bw::launch((attn_merge_kernel), dim3(n_merge_items, nkv, 16), dim3(MERGE_THREADS), 0, s, p, merge_work);

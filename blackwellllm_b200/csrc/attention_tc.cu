@@ -66,6 +66,7 @@ struct Params {
     // softcap > 0: the scaled score s becomes softcap * tanh(s / softcap) before a bias is added.  rel != null: float32
     // [nh][rel_len], rel[query head][min(i - j, rel_len - 1)] is added to the score.  (Not together with dist.)
     float softcap; const float* rel; int rel_len;
+    bw::DiffHeads diff;   // diff.lam != null: pairs of query heads become one head (G even; the gate has one number per head)
 };
 
 // 2^x and log2(x), one MUFU instruction each
@@ -398,6 +399,47 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
             bw::tc_fence_after();
             if (p.sink) l += exp2f(p.sink[g * p.G + hg] * 1.4426950408889634f - m);   // m: the maximum that l is counted from
             const float inv = l > 0.f ? 1.f / l : 0.f;
+            if (p.diff.lam) {
+                // The maps of a head are neighbouring rows, so neighbouring lanes (G is even).  Of 32 channels the even lane makes the
+                // first 16 of the head, the odd lane the others: each sends the half that the other makes.  Two passes over O: the
+                // sum of squares, then the result.
+                const bool odd = lane & 1;
+                const float mine = bw::diff_weight(p.diff, odd, inv);
+                const size_t token = (size_t)(p.cu_q[r] + tok0 + tok);
+                const int head = (g * p.G + hg) >> 1;
+                bf16* dst = p.out + (token * (p.nh >> 1) + head) * HD + (odd ? 16 : 0);
+                float ss = 0.f, f = 0.f;
+#pragma unroll 1
+                for (int pass = 0; pass < 2; ++pass) {
+#pragma unroll 1
+                    for (int c0 = 0; c0 < HD; c0 += 32) {
+                        uint32_t v[32];
+                        bw::tmem_ld_32x32(tmem_O + lane_base + c0, v);
+                        bw::tmem_ld_wait();
+                        float o[16];
+#pragma unroll
+                        for (int c = 0; c < 16; ++c) {
+                            const float lo = __uint_as_float(v[c]) * mine, hi = __uint_as_float(v[16 + c]) * mine;
+                            const float other = __shfl_xor_sync(0xffffffffu, odd ? lo : hi, 1);
+                            o[c] = (odd ? hi : lo) + other;
+                        }
+                        if (pass == 0) {
+#pragma unroll
+                            for (int c = 0; c < 16; ++c) ss = fmaf(o[c], o[c], ss);
+                        } else if (row_ok) {
+#pragma unroll
+                            for (int c = 0; c < 16; c += 8)
+                                *reinterpret_cast<uint4*>(dst + c0 + c) =
+                                    make_uint4(pack_bf16(o[c] * f, o[c + 1] * f), pack_bf16(o[c + 2] * f, o[c + 3] * f),
+                                               pack_bf16(o[c + 4] * f, o[c + 5] * f), pack_bf16(o[c + 6] * f, o[c + 7] * f));
+                        }
+                    }
+                    if (pass == 0) {
+                        ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+                        if (row_ok) f = bw::diff_factor(p.diff, ss, p.gate, p.gate_ld, token, head);
+                    }
+                }
+            } else {
             bf16* dst = p.out + ((size_t)(p.cu_q[r] + tok0 + tok) * p.nh + g * p.G + hg) * HD;
 #pragma unroll
             for (int c0 = 0; c0 < HD; c0 += 32) {
@@ -438,6 +480,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
                                        pack_bf16(__uint_as_float(v[c + 6]) * inv, __uint_as_float(v[c + 7]) * inv));
                     }
                 }
+            }
             }
         }
     }
@@ -487,13 +530,14 @@ BW_EXPORT int bw_attention_tc_supported(int nh, int nkv, int page_size) {
 
 // work: n_items int4 (request, first token of the 128-row tile within the request's segment, 0, 0);
 // a tile holds 128 / G tokens.  q, out: [T, nh * HD] bf16; pages: [num_pages, nkv, page_size, HD] bf16.
-// dist: float32 [2][nh] or null; keep_first: see Params.  softcap (> 0: on), rel, rel_len: see Params.
+// dist: float32 [2][nh] or null; keep_first: see Params.  softcap (> 0: on), rel, rel_len: see Params.  lam != null: pairs of query heads
+// become one (bw::DiffHeads: one float32 number on the device, diff_eps, diff_scale, diff_dv); out is then [T, nh / 2 * HD].
 BW_EXPORT int bw_attention_tc(const void* q, const void* k_pages, const void* v_pages, void* out, const int* cu_q,
                               const int* q_start, const int* kv_len, const int* block_table, int max_blocks,
                               const int* work, int n_items, int T, int nh, int nkv, int page_size, int num_pages,
                               int window, int chunk, float scale, const float* sink, const float* gate, long long gate_ld,
                               int gate_dv, const float* dist, int keep_first, float softcap, const float* rel, int rel_len,
-                              void* stream) {
+                              const float* lam, float diff_eps, float diff_scale, int diff_dv, void* stream) {
     if (n_items <= 0) return 0;
     if ((rel && rel_len <= 0) || ((rel || softcap > 0.f) && dist)) return BW_ERR_UNSUPPORTED;
     if (!bw_attention_tc_supported(nh, nkv, page_size) || !(scale > 0.f)) return BW_ERR_UNSUPPORTED;
@@ -520,7 +564,9 @@ BW_EXPORT int bw_attention_tc(const void* q, const void* k_pages, const void* v_
     p.window = window > 0 ? window : 0; p.chunk = chunk > 0 ? chunk : 0; p.tpt = tpt;
     p.scale_log2 = scale * 1.4426950408889634f;
     p.sink = sink;
-    if (gate && gate_dv < 0 ? (-gate_dv > HD || gate_ld < (long long)nh)
+    if (lam && (G % 2 || sink || diff_dv <= 0 || diff_dv > HD || (gate && gate_dv >= 0))) return BW_ERR_BAD_ARG;
+    p.diff.lam = lam; p.diff.eps = diff_eps; p.diff.scale = diff_scale; p.diff.dv = diff_dv;
+    if (gate && gate_dv < 0 ? (-gate_dv > HD || gate_ld < (long long)(lam ? nh / 2 : nh))
                             : gate && (gate_dv <= 0 || gate_dv > HD || gate_ld < (long long)nh * gate_dv)) return BW_ERR_BAD_ARG;
     p.gate = gate; p.gate_ld = gate_ld; p.gate_dv = gate_dv;
     p.dist = dist; p.keep_first = (keep_first > 0 && p.window > 0) ? keep_first : 0;

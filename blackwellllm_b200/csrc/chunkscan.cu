@@ -12,10 +12,11 @@
 //   o_t = G_t S0^T q_t + sum_{s<=t} M_ts u_s,    M_ts = D_ts k_s . q_t           S = G S0 + sum_s R_s k_s u_s^T
 //
 // A third form is the delta rule with a decay per KEY CHANNEL, S <- diag(g_t) S in place of g_t S.  Then D_ts is a vector inside
-// the dot products, L_ts = beta_t sum_c k_s[c] D_ts[c] k_t[c] and M_ts likewise with q_t, and the walk reads ready-made rows
-// G_t o k_t, G_t o q_t (where it says G_t S0^T k_t, G_t S0^T q_t above) and R_s o k_s, with the chunk's G as a vector over the state's
-// rows.  chunk_rows_channel_kernel makes all of that, again with products of decays only: the vector D_ts o k_s is carried along
-// t in registers.
+// the dot products, L_ts = beta_t sum_c k_s[c] D_ts[c] k_t[c] and M_ts likewise with q_t; G_t and R_t multiply q_t and k_t channel by
+// channel, and the chunk's G is a vector over the state's rows.  Since U = T beta V - (T beta (G o K)) S0, the part of U that does not
+// know S0 and the rows W = T beta (G o K) are made beforehand too, so that the walk needs no T: U = U0 - W S0.
+// chunk_rows_channel_kernel makes all of that, again with products of decays only: the vector D_ts o k_s is carried along t in
+// registers.
 //
 // chunk_rows_kernel makes the rows of T and M and the numbers G, R for every token and head, in parallel over the chunks, with
 // float32 FMAs.  chunk_scan_kernel walks the chunks of one request's portion: a block owns (request, head, 16 value columns)
@@ -31,6 +32,7 @@ namespace {
 constexpr int C = 32;             // tokens of a chunk
 constexpr int ROW_DELTA = 68;     // floats per (token, head): T row, M row, G, R, beta, 0
 constexpr int ROW_LINEAR = 36;    // M row (with c_s in it), G, c R, 0, 0
+constexpr int ROW_CHANNEL = 32;   // M row
 constexpr int TS = 40;            // floats between rows of 32 in shared memory: 8-byte reads of (row g, column 2 t) hit 32 banks
 constexpr int VS = 20;            // floats between tokens' 16 values
 constexpr int COLS = 16;
@@ -44,7 +46,8 @@ struct ChunkParams {
     float* o;                              // [T, heads * dv]
     int T, R, heads, rep, dk, dv, vec;     // vec: 16-byte copies of q and k rows (1), of the values (2)
     // the form with a decay per key channel: decay [T, heads, dk], and two more scratches
-    float* chan;                           // [T, heads, 3, dk]: G o k, G o q, R o k
+    float* chan;                           // [T, heads, 3, dk]: W, G o q, R o k
+    float* u0;                             // [T, heads, dv]: U0
     float* gend;                           // [T / C + R, heads, dk]: the product of a chunk's decays (chunk_index)
 };
 
@@ -275,17 +278,13 @@ chunk_rows_channel_kernel(ChunkParams p) {
     }
     __syncthreads();
     if (warp == 0) {
-        float* base = p.rows + ((size_t)t0 * p.heads + h) * ROW_DELTA;
-        const size_t step = (size_t)p.heads * ROW_DELTA;
+        float* base = p.rows + ((size_t)t0 * p.heads + h) * ROW_CHANNEL;
+        const size_t step = (size_t)p.heads * ROW_CHANNEL;
         const float beta = lane < n ? p.second[(size_t)(t0 + lane) * p.heads + h] : 0.f;
         for (int t = 0; t < n; ++t) {
             const float bt = __shfl_sync(0xffffffffu, beta, t);
-            base[t * step + C + lane] = t >= lane ? kq[t * (C + 4) + lane] : 0.f;
+            base[t * step + lane] = t >= lane ? kq[t * (C + 4) + lane] : 0.f;
             kk[t * (C + 4) + lane] = t > lane ? bt * kk[t * (C + 4) + lane] : 0.f;
-        }
-        if (lane < n) {      // (the decays stand in the rows themselves: G and R are 1 here)
-            float* sc = base + lane * step + 2 * C;
-            sc[0] = 1.f; sc[1] = 1.f; sc[2] = beta; sc[3] = 0.f;
         }
         __syncwarp();
         float x[C];                        // lane s: column s of T, row by row (rows of kk from n on are zeros)
@@ -301,25 +300,52 @@ chunk_rows_channel_kernel(ChunkParams p) {
                 if (j + 3 < t) u1 = fmaf(-l.w, x[j + 3], u1);
             }
             x[t] = u0 + u1;
-            if (t < n) base[t * step + lane] = x[t];
         }
-        return;
+        __syncwarp();
+#pragma unroll
+        for (int t = 0; t < C; ++t) kk[t * (C + 4) + lane] = x[t] * beta;        // T beta in place of L (zero columns from n on)
+    } else {
+        // meanwhile the other warps: the rows with the decays in them; G o k stays here
+        const size_t step = (size_t)p.heads * 3 * p.dk;
+        for (int c = threadIdx.x - 32; c < p.dk; c += 96) {
+            float* dst = p.chan + ((size_t)t0 * p.heads + h) * 3 * p.dk + c;
+            float R = 1.f;
+            for (int t = n - 1; t >= 0; --t) {
+                dst[t * step + 2 * p.dk] = R * ks[t * lds + c];
+                R *= gs[t * lds + c];
+            }
+            float G = 1.f;
+            for (int t = 0; t < n; ++t) {
+                G *= gs[t * lds + c];
+                ks[t * lds + c] *= G;
+                dst[t * step + p.dk] = G * qs[t * lds + c];
+            }
+            p.gend[((size_t)index * p.heads + h) * p.dk + c] = G;
+        }
     }
-    // meanwhile the other warps: the rows with the decays in them
-    const size_t step = (size_t)p.heads * 3 * p.dk;
-    for (int c = threadIdx.x - 32; c < p.dk; c += 96) {
-        float* dst = p.chan + ((size_t)t0 * p.heads + h) * 3 * p.dk + c;
-        float G = 1.f;
-        for (int t = 0; t < n; ++t) {
-            G *= gs[t * lds + c];
-            dst[t * step] = G * ks[t * lds + c];
-            dst[t * step + p.dk] = G * qs[t * lds + c];
-        }
-        p.gend[((size_t)index * p.heads + h) * p.dk + c] = G;
-        float R = 1.f;
-        for (int t = n - 1; t >= 0; --t) {
-            dst[t * step + 2 * p.dk] = R * ks[t * lds + c];
-            R *= gs[t * lds + c];
+    __syncthreads();
+    // W = T beta (G o K) and U0 = T beta V: a thread per column, which it keeps in registers
+    const int cols = p.dk + p.dv;
+    for (int c = threadIdx.x; c < cols; c += 128) {
+        const bool is_k = c < p.dk;
+        float x[C];
+        const float* v = p.qkv + (size_t)t0 * p.ld + p.v_off + h * p.dv + (c - p.dk);
+#pragma unroll
+        for (int t = 0; t < C; ++t) x[t] = is_k ? ks[t * lds + c] : (t < n ? v[(size_t)t * p.ld] : 0.f);
+        float* dst = is_k ? p.chan + ((size_t)t0 * p.heads + h) * 3 * p.dk + c : p.u0 + ((size_t)t0 * p.heads + h) * p.dv + (c - p.dk);
+        const size_t step = (size_t)p.heads * (is_k ? 3 * p.dk : p.dv);
+#pragma unroll
+        for (int t = 0; t < C; ++t) {
+            float a0 = 0.f, a1 = 0.f;
+#pragma unroll
+            for (int j = 0; j <= t; j += 4) {
+                const float4 m = *reinterpret_cast<const float4*>(kk + t * (C + 4) + j);     // (zeros above the diagonal)
+                a0 = fmaf(m.x, x[j], a0);
+                a1 = fmaf(m.y, x[j + 1], a1);
+                a0 = fmaf(m.z, x[j + 2], a0);
+                a1 = fmaf(m.w, x[j + 3], a1);
+            }
+            if (t < n) dst[t * step] = a0 + a1;
         }
     }
 }
@@ -377,8 +403,8 @@ template <bool DELTA, bool CHAN, int NW, int NB, int MT>
 struct ChunkSmem {
     static constexpr int LDK = 8 * NB * NW + 4;                 // a token's q or k
     static constexpr int LDV = MT == 1 ? VS : 36;           // a token's values (twice it is 8 modulo 32)
-    static constexpr int k0 = 0, q0 = k0 + C * LDK, v0 = q0 + C * LDK, m0 = v0 + C * LDV, t0 = m0 + C * TS, s0 = t0 + (DELTA ? C * TS : 0);
-    static constexpr int r0 = s0 + C * 4, g0 = r0 + (CHAN ? C * LDK : 0);
+    static constexpr int k0 = 0, q0 = k0 + C * LDK, v0 = q0 + C * LDK, m0 = v0 + C * LDV, t0 = m0 + C * TS, s0 = t0 + (DELTA && !CHAN ? C * TS : 0);
+    static constexpr int r0 = s0 + (CHAN ? 0 : C * 4), g0 = r0 + (CHAN ? C * LDK : 0);
     static constexpr int buffer = g0 + (CHAN ? 8 * NB * NW : 0);
     static constexpr int part = (DELTA ? 2 : 1) * COLS * TS;            // one warp's parts of S0^T q (and S0^T k)
     static constexpr int tail = NW * MT * part + (DELTA ? MT * COLS * TS : 0);
@@ -392,7 +418,7 @@ chunk_scan_kernel(ChunkParams p) {
     BW_PDL_TRIGGER();
     using L = ChunkSmem<DELTA, CHAN, NW, NB, MT>;
     constexpr int THREADS = 32 * NW * MT, DKP = 8 * NB * NW, LDK = L::LDK, LDV = L::LDV;
-    constexpr int ROW = DELTA ? ROW_DELTA : ROW_LINEAR;
+    constexpr int ROW = CHAN ? ROW_CHANNEL : (DELTA ? ROW_DELTA : ROW_LINEAR);
     extern __shared__ __align__(16) float sm[];
     float* part = sm + L::buffers * L::buffer;
     const int r = blockIdx.x, h = blockIdx.y;
@@ -451,17 +477,19 @@ chunk_scan_kernel(ChunkParams p) {
                 copy4(b + L::q0 + t * LDK + i, in ? s + p.q_off : src, in);
             }
         }
+        const float* vals = CHAN ? p.u0 + ((size_t)tb * p.heads + h) * p.dv + cb : src + p.v_off + h * p.dv + cb;
+        const size_t v_step = CHAN ? (size_t)p.heads * p.dv : (size_t)p.ld;
         if (p.vec & 2) {
             for (int idx = threadIdx.x; idx < C * 4 * MT; idx += THREADS) {
                 const int t = idx / (4 * MT), c = (idx % (4 * MT)) * 4;
                 const bool in = t < n && cb + c < p.dv;
-                copy16(b + L::v0 + t * LDV + c, in ? src + (size_t)t * p.ld + p.v_off + h * p.dv + cb + c : src, in);
+                copy16(b + L::v0 + t * LDV + c, in ? vals + t * v_step + c : src, in);
             }
         } else {
             for (int idx = threadIdx.x; idx < C * COLS * MT; idx += THREADS) {
                 const int t = idx / (COLS * MT), c = idx % (COLS * MT);
                 const bool in = t < n && cb + c < p.dv;
-                copy4(b + L::v0 + t * LDV + c, in ? src + (size_t)t * p.ld + p.v_off + h * p.dv + cb + c : src, in);
+                copy4(b + L::v0 + t * LDV + c, in ? vals + t * v_step + c : src, in);
             }
         }
         for (int idx = threadIdx.x; idx < C * (ROW / 4); idx += THREADS) {
@@ -469,7 +497,8 @@ chunk_scan_kernel(ChunkParams p) {
             const bool in = t < n;
             const float* s = in ? p.rows + ((size_t)(tb + t) * p.heads + h) * ROW + u * 4 : p.rows;
             float* dst;
-            if constexpr (DELTA) dst = u < 8 ? b + L::t0 + t * TS + u * 4 : (u < 16 ? b + L::m0 + t * TS + (u - 8) * 4 : b + L::s0 + t * 4);
+            if constexpr (CHAN) dst = b + L::m0 + t * TS + u * 4;
+            else if constexpr (DELTA) dst = u < 8 ? b + L::t0 + t * TS + u * 4 : (u < 16 ? b + L::m0 + t * TS + (u - 8) * 4 : b + L::s0 + t * 4);
             else dst = u < 8 ? b + L::m0 + t * TS + u * 4 : b + L::s0 + t * 4;
             copy16(dst, s, in);
         }
@@ -535,7 +564,20 @@ chunk_scan_kernel(ChunkParams p) {
             }
             return v;
         };
-        if constexpr (DELTA) {
+        if constexpr (CHAN) {
+            // U = U0 - W S0, a thread per column and pair of tokens (zeros behind the portion's end)
+            for (int i = threadIdx.x % (32 * NW); i < COLS * (C / 2); i += 32 * NW) {
+                const int row = i / (C / 2), t = i % (C / 2) * 2;
+                float2 y = make_float2(0.f, 0.f);
+#pragma unroll
+                for (int w = 0; w < NW; ++w) {
+                    const float2 e = *reinterpret_cast<const float2*>(group + (size_t)w * L::part + (COLS + row) * TS + t);
+                    y.x += e.x; y.y += e.y;
+                }
+                *reinterpret_cast<float2*>(us + row * TS + t) = make_float2(vs[t * LDV + row] - y.x, vs[(t + 1) * LDV + row] - y.y);
+            }
+            __syncthreads();
+        } else if constexpr (DELTA) {
             for (int tk = kw; 8 * tk < n; tk += NW) {          // U of this warp's eight tokens
                 float u[1][4] = {{0.f, 0.f, 0.f, 0.f}};
                 for (int kb = 0; kb <= tk; ++kb) {
@@ -581,7 +623,7 @@ chunk_scan_kernel(ChunkParams p) {
             }
             const int t = 8 * tk + 2 * t4;
             const float2 p0 = total(g, tk), p1 = total(g + 8, tk);
-            const float G0 = sc[t * 4], G1 = sc[t * 4 + 4];
+            const float G0 = CHAN ? 1.f : sc[t * 4], G1 = CHAN ? 1.f : sc[t * 4 + 4];
             float* dst = p.o + ((size_t)(tb + t) * p.heads + h) * p.dv + c0 + g;
             const size_t ldo = (size_t)p.heads * p.dv;
             if (t < n) {
@@ -604,7 +646,7 @@ chunk_scan_kernel(ChunkParams p) {
             for (int kb = 0; kb < 4; ++kb) {
                 if (8 * kb >= n) break;
                 const int t = 8 * kb + 2 * t4;
-                const float R0 = sc[t * 4 + 1], R1 = sc[t * 4 + 5];
+                const float R0 = CHAN ? 1.f : sc[t * 4 + 1], R1 = CHAN ? 1.f : sc[t * 4 + 5];
                 const SplitA a = split_a(u[kb][0] * R0, u[kb][1] * R0, u[kb][2] * R1, u[kb][3] * R1);
                 float k[NB][2];
 #pragma unroll
@@ -682,29 +724,30 @@ int run(const ChunkParams& p, int R, cudaStream_t s) {
 }  // namespace
 
 // floats per (token, head) of the scratch that bw_chunk_scan takes
-BW_EXPORT int bw_chunk_row_floats(int delta) { return delta ? ROW_DELTA : ROW_LINEAR; }
+BW_EXPORT int bw_chunk_row_floats(int delta) { return delta == 2 ? ROW_CHANNEL : (delta ? ROW_DELTA : ROW_LINEAR); }
 
 // qkv: float32 rows `ld` apart with q and k (heads / rep heads of dk channels) and v (heads of dv) at the given columns;
 // decay [T, heads]; second [T, heads]: beta (delta != 0) or the keys' factor; rows: scratch float32
 // [T, heads, bw_chunk_row_floats(delta)], 16-byte aligned; state [slots, heads, dk, sld]; o [T, heads * dv].
-// delta == 2: the delta rule with decay [T, heads * dk]; chan: scratch float32 [T, heads, 3, dk], gend: scratch float32
-// [T / 32 + R, heads, dk], both 16-byte aligned (otherwise null).
+// delta == 2: the delta rule with decay [T, heads * dk]; scratches float32, 16-byte aligned (otherwise null): chan [T, heads, 3, dk],
+// u0 [T, heads, dv], gend [T / 32 + R, heads, dk].
 BW_EXPORT int bw_chunk_scan(int delta, const float* qkv, long long ld, int q_off, int k_off, int v_off, const float* decay,
                             const float* second, const int* cu_q, const int* state_slot, float* rows,
-                            float* chan, float* gend, float* state, float* o, int T, int R, int heads, int rep, int dk, int dv,
+                            float* chan, float* u0, float* gend, float* state, float* o, int T, int R, int heads, int rep, int dk, int dv,
                             int sld, void* stream) {
     if (T <= 0 || R <= 0) return 0;
     if (heads <= 0 || rep <= 0 || heads % rep || dk <= 0 || dv <= 0 || sld < dv || !rows || ((uintptr_t)rows & 15)) return BW_ERR_BAD_ARG;
     if (dk > 256) return BW_ERR_UNSUPPORTED;
-    if (delta == 2 && (!chan || !gend || (((uintptr_t)chan | (uintptr_t)gend) & 15))) return BW_ERR_BAD_ARG;
+    if (delta == 2 && (!chan || !u0 || !gend || (((uintptr_t)chan | (uintptr_t)u0 | (uintptr_t)gend) & 15))) return BW_ERR_BAD_ARG;
     ChunkParams p;
-    p.chan = chan; p.gend = gend;
+    p.chan = chan; p.u0 = u0; p.gend = gend;
     p.qkv = qkv; p.ld = ld; p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.decay = decay; p.second = second; p.cu_q = cu_q;
     p.state_slot = state_slot; p.rows = rows; p.state = state; p.sld = sld; p.o = o;
     p.T = T; p.R = R; p.heads = heads; p.rep = rep; p.dk = dk; p.dv = dv;
     const bool base = ((uintptr_t)qkv & 15) == 0 && (ld & 3) == 0;
     p.vec = (base && (dk & 3) == 0 && (q_off & 3) == 0 && (k_off & 3) == 0 ? 1 : 0) | (base && (dv & 3) == 0 && (v_off & 3) == 0 ? 2 : 0);
-    if (delta == 2 && ((uintptr_t)decay & 15)) p.vec &= ~1;
+    if (delta == 2) p.vec = (((uintptr_t)decay & 15) ? p.vec & ~1 : p.vec) & ~2;
+    if (delta == 2 && (dv & 3) == 0) p.vec |= 2;           // (the values come from the scratch)
     if (delta == 2) return run<true, true>(p, R, (cudaStream_t)stream);
     return delta ? run<true, false>(p, R, (cudaStream_t)stream) : run<false, false>(p, R, (cudaStream_t)stream);
 }

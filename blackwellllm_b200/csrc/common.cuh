@@ -208,6 +208,23 @@ __device__ __forceinline__ float out_gate(const float* __restrict__ gate, long l
     return 1.f / (1.f + expf(-gate[token * (size_t)ld + (size_t)head * dv + c]));
 }
 
+// Differential attention in the attention kernels' epilogues: query heads 2 h and 2 h + 1 are the two maps a1, a2 of head h, and what is
+// written is  o / sqrt(mean(o^2) + eps) * scale * gate_h,  o = a1 - *lam a2,  over dv channels (those beyond are zeros), as head h of
+// half as many heads.  lam == null: every query head is written by itself.
+struct DiffHeads {
+    const float* lam;
+    float eps, scale;
+    int dv;
+};
+// What map `which` of a pair counts with, `inv` the inverse of its softmax's denominator.
+__device__ __forceinline__ float diff_weight(const DiffHeads& d, int which, float inv) { return which ? -__ldg(d.lam) * inv : inv; }
+// The factor of a head's o from its sum of squares; the gate: one number per head, or none.
+__device__ __forceinline__ float diff_factor(const DiffHeads& d, float ss, const float* __restrict__ gate, long long ld, size_t token, int head) {
+    float f = rsqrtf(ss / (float)d.dv + d.eps) * d.scale;
+    if (gate) f *= 1.f / (1.f + expf(-gate[token * (size_t)ld + (size_t)head]));
+    return f;
+}
+
 // Two float32 operations in one instruction (sm_100: the packed form of fma and mul); a pair is a 64-bit register, the first
 // value in the low half.
 typedef unsigned long long f32x2;

@@ -117,7 +117,7 @@ head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __
                       const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps,
                       float q_coef, float q_every,
                       OT* __restrict__ q_out, OT* __restrict__ k_pages, OT* __restrict__ v_pages,
-                      int nh, int nkv, int dq, int dv, int dpad, int page_size, int num_pages, int has_kv, int vec, int vec2, int vec_v,
+                      int nh, int nkv, int dq, int dv, int dpad, int page_size, int num_pages, int has_kv, int vec, int vec2, int pairs, int vec_v,
                       float v_eps, const float* __restrict__ v_first, long long v_first_ld, const float* __restrict__ v_lam,
                       const float* __restrict__ q_head_mult, int v_col, float v_scale) {
     BW_PDL_TRIGGER();
@@ -144,7 +144,7 @@ head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __
         const float* src = is_q ? row + (size_t)h * dq : row + nq + (size_t)(h - nh) * dq;
         const float* gain = is_q ? q_gain : k_gain;
         float r = 1.f;
-        if (gain && !vec2) {
+        if (gain && !vec2 && !pairs) {
             float ss = 0.f;
             for (int c = lane; c < dq; c += 32) { const float v = src[c]; ss = fmaf(v, v, ss); }
             r = rsqrtf(bw::warp_sum(ss) / (float)dq + eps);
@@ -203,6 +203,28 @@ head_norm_rope_kernel(const float* __restrict__ qkv, long long ld, const int* __
                     const float2 g = (gain && c < dq) ? *reinterpret_cast<const float2*>(gain + c) : make_float2(1.f, 1.f);
                     put2(dst + c, q[i].x * r2 * g.x, q[i].y * r2 * g.y);
                 }
+            }
+            continue;
+        }
+        if (pairs) {
+            // rotation of neighbours, even sizes up to 256, aligned rows: a lane keeps whole pairs in registers
+            float2 a[4];
+            float ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int c = i * 64 + lane * 2;
+                a[i] = c < dq ? *reinterpret_cast<const float2*>(src + c) : make_float2(0.f, 0.f);
+                ss = fmaf(a[i].x, a[i].x, ss); ss = fmaf(a[i].y, a[i].y, ss);
+            }
+            const float r2 = (gain ? rsqrtf(bw::warp_sum(ss) / (float)dq + eps) : 1.f) * mult;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int c = i * 64 + lane * 2;
+                if (c >= dpad) break;
+                const float2 g = (gain && c < dq) ? *reinterpret_cast<const float2*>(gain + c) : make_float2(1.f, 1.f);
+                const float x = a[i].x * r2 * g.x, y = a[i].y * r2 * g.y;
+                const float cs = c < rotary_dim ? tab[c >> 1] : 1.f, sn = c < rotary_dim ? tab[half + (c >> 1)] : 0.f;
+                put2(dst + c, x * cs - y * sn, y * cs + x * sn);
             }
             continue;
         }
@@ -290,11 +312,13 @@ BW_EXPORT int bw_head_norm_rope_append(const float* qkv, long long ld, const int
     const int vec2 = rotary_dim > 0 && !interleaved && (rotary_dim & 3) == 0 && (dq & 1) == 0 && (dpad & 1) == 0 && dpad <= 256 &&
                      (ld & 1) == 0 && (((uintptr_t)qkv | (uintptr_t)q_gain | (uintptr_t)k_gain | (uintptr_t)table | (uintptr_t)q_out |
                                         (uintptr_t)k_pages) & 7) == 0;
+    const int pairs = rotary_dim > 0 && interleaved && (dq & 1) == 0 && (dpad & 1) == 0 && dpad <= 256 && (ld & 1) == 0 &&
+                      (((uintptr_t)qkv | (uintptr_t)q_gain | (uintptr_t)k_gain | (uintptr_t)q_out | (uintptr_t)k_pages) & 7) == 0;
     const int vec_v = (dv & 3) == 0 && (dpad & 3) == 0 && (ld & 3) == 0 && (v_col & 3) == 0 &&
                       (((uintptr_t)qkv | (uintptr_t)v_pages) & 15) == 0;
 #define BW_HN(OT) bw::launch((head_norm_rope_kernel<OT>), dim3(T), dim3(256), 0, s, qkv, ld, positions, req_of_token, block_table, \
         max_blocks, table, rotary_dim, interleaved, q_gain, k_gain, eps, q_coef, q_every, (OT*)q_out, (OT*)k_pages, (OT*)v_pages, \
-        nh, nkv, dq, dv, dpad, page_size, num_pages, has_kv, vec, vec2, vec_v, v_eps, v_first, v_first_ld, v_lam, \
+        nh, nkv, dq, dv, dpad, page_size, num_pages, has_kv, vec, vec2, pairs, vec_v, v_eps, v_first, v_first_ld, v_lam, \
         q_head_mult, v_col, v_scale)
     if (out_type == BW_F32) BW_HN(float);
     else if (out_type == BW_BF16) BW_HN(bf16);

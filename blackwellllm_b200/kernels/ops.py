@@ -860,7 +860,7 @@ def paged_attention(q, k_pages: torch.Tensor, v_pages: torch.Tensor, batch,
                     chunk: Optional[int] = None, sink: Optional[torch.Tensor] = None,
                     gate: Optional[tuple] = None, dist: Optional[torch.Tensor] = None,
                     keep_first: int = 0, softcap: Optional[float] = None,
-                    rel: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    rel: Optional[torch.Tensor] = None, diff: Optional[tuple] = None) -> torch.Tensor:
     """Causal attention of the batch's tokens over the paged cache (which already
     holds this step's keys and values, unless ``q`` is an :class:`UnrotatedQKV`).  float32: the
     CUDA-core kernel; bfloat16: the tensor-core kernel built for this head size.  A query sees the keys
@@ -873,7 +873,18 @@ def paged_attention(q, k_pages: torch.Tensor, v_pages: torch.Tensor, batch,
     the score of query position i and key position j.  ``keep_first``: the first so many keys of a sequence stay
     visible beyond the window.  ``softcap``: the scaled score s becomes softcap * tanh(s / softcap) before any bias.
     ``rel`` (float32 [nh, n]): rel[head, min(i - j, n - 1)] is added to the score (a learned bias per distance, its last
-    entry standing for every larger distance; :func:`distance_bucket_table` says which distances share a learned row)."""
+    entry standing for every larger distance; :func:`distance_bucket_table` says which distances share a learned row).  ``diff`` =
+    (lam: one float32 number on the device, eps, scale, dv): differential attention, query heads 2 h and 2 h + 1 are the two maps of
+    head h and become one as in :func:`diff_combine`, in the tensor-core kernels' epilogues; a gate then is ``(g [T, nh / 2], dv, "head")``,
+    there is no sink, and the result is [T, nh / 2 * head size]."""
+    if diff is not None and (isinstance(q, UnrotatedQKV) or sink is not None or nh // k_pages.shape[1] % 2
+                             or (gate is not None and (len(gate) != 3 or gate[0].shape[1] != nh // 2))):
+        raise KernelError("attention: differential heads come in pairs per kv head, with finished queries, no sink, a gate per head")
+    if diff is not None and (q.dtype == torch.float32 or nh // k_pages.shape[1] > MAX_GROUP_BF16 or k_pages.shape[3] > 256):
+        a = attention_simt(q, k_pages, v_pages, batch.positions, batch.req_of_token, block_table, nh, window, scale, chunk=chunk,
+                           dist=dist, keep_first=keep_first, softcap=softcap, rel=rel)
+        lam, eps, factor, dv = diff
+        return diff_combine(a, nh // 2, dv, lam, eps, factor, None if gate is None else gate[0], a.dtype)
     if (softcap or rel is not None) and isinstance(q, UnrotatedQKV):
         q = q.materialise()
     if isinstance(q, UnrotatedQKV):
@@ -891,13 +902,13 @@ def paged_attention(q, k_pages: torch.Tensor, v_pages: torch.Tensor, batch,
                               window, scale, chunk=chunk, sink=sink, gate=gate, dist=dist, keep_first=keep_first,
                               softcap=softcap, rel=rel)
     return attention_mma(q, k_pages, v_pages, batch, block_table, nh, window, scale, chunk, sink, gate, dist, keep_first,
-                         softcap, rel)
+                         softcap, rel, diff)
 
 
 _ATTN_MMA_ARGS = [c_void_p] * 8 + [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                    c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                                    c_void_p, c_int, c_ll, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_ll, c_int,
-                                   c_void_p, c_int, c_float, c_void_p, c_int, c_void_p]
+                                   c_void_p, c_int, c_float, c_void_p, c_int, c_void_p, c_float, c_float, c_int, c_void_p]
 
 
 _sm_counts = {}
@@ -988,7 +999,7 @@ def attention_mma(q, k_pages: torch.Tensor, v_pages: torch.Tensor, batch, block_
                   nh: int, window: Optional[int], scale: float, chunk: Optional[int] = None,
                   sink: Optional[torch.Tensor] = None, gate: Optional[tuple] = None,
                   dist: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: Optional[float] = None,
-                  rel: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  rel: Optional[torch.Tensor] = None, diff: Optional[tuple] = None) -> torch.Tensor:
     _dev(k_pages, "k_pages", torch.bfloat16); _dev(v_pages, "v_pages", torch.bfloat16)
     _check_sink(sink, nh)
     _check_dist(dist, nh)
@@ -997,7 +1008,10 @@ def attention_mma(q, k_pages: torch.Tensor, v_pages: torch.Tensor, batch, block_
         raise KernelError("attention: a soft cap on the scores does not go with the logarithmic distance bias")
     rel_len = rel.shape[1] if rel is not None else 0
     keep_first = int(keep_first or 0) if window else 0
-    g, g_ld, g_dv = _gate_args(gate, batch.T, nh, k_pages.shape[3])
+    g, g_ld, g_dv = _gate_args(gate, batch.T, nh // 2 if diff is not None else nh, k_pages.shape[3])
+    lam, d_eps, d_scale, d_dv = diff if diff is not None else (None, 0.0, 0.0, 0)
+    if lam is not None:
+        _dev(lam, "lam", torch.float32)
     _dev(block_table, "block_table", torch.int32)
     num_pages, nkv, page_size, hd = k_pages.shape
     raw = q if isinstance(q, UnrotatedQKV) else None
@@ -1019,7 +1033,7 @@ def attention_mma(q, k_pages: torch.Tensor, v_pages: torch.Tensor, batch, block_
         _dev(q, "q", torch.bfloat16)
         if q.shape[1] != nh * hd or nh % nkv:
             raise KernelError("attention: q must be [T, nh * head_dim] with nh a multiple of the kv heads")
-        out = torch.empty_like(q)
+        out = torch.empty_like(q) if diff is None else torch.empty((q.shape[0], nh // 2 * hd), dtype=q.dtype, device=q.device)
     G = nh // nkv
     check_attention_supported(torch.bfloat16, hd, G)
     if hd > 256:
@@ -1039,7 +1053,8 @@ def attention_mma(q, k_pages: torch.Tensor, v_pages: torch.Tensor, batch, block_
         _check(tc(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(batch.cu_q), _ptr(batch.q_start),
                   _ptr(batch.kv_len), _ptr(block_table), block_table.shape[1], _ptr(rows_w), n_rows, q.shape[0],
                   nh, nkv, page_size, num_pages, int(window or 0), int(chunk or 0), float(scale), _ptr(sink), _ptr(g), g_ld, g_dv,
-                  _ptr(dist), keep_first, float(softcap or 0.0), _ptr(rel), rel_len, _stream()), "attention_tc")
+                  _ptr(dist), keep_first, float(softcap or 0.0), _ptr(rel), rel_len, _ptr(lam), float(d_eps), float(d_scale), int(d_dv),
+                  _stream()), "attention_tc")
         n_rows = 0
         if not n_keys:
             return out
@@ -1052,12 +1067,13 @@ def attention_mma(q, k_pages: torch.Tensor, v_pages: torch.Tensor, batch, block_
               raw.planes.stride(0) if raw is not None else 0, _ptr(raw.table if raw is not None else None),
               raw.rotary_dim if raw is not None else 0, int(raw.append) if raw is not None else 0, merge_max,
               _ptr(sink), _ptr(g), g_ld, g_dv, _ptr(dist), keep_first, float(softcap or 0.0), _ptr(rel), rel_len,
-              _stream()), "attention_mma")
+              _ptr(lam), float(d_eps), float(d_scale), int(d_dv), _stream()), "attention_mma")
     return out
 
 
 _ATTN_TC_ARGS = [c_void_p] * 8 + [c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p,
-                                  c_void_p, c_ll, c_int, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p]
+                                  c_void_p, c_ll, c_int, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p, c_float, c_float, c_int,
+                                  c_void_p]
 
 
 def attention_tc_supports(hd: int, G: int, page_size: int) -> bool:
@@ -1767,19 +1783,21 @@ def chunk_scan(delta: bool, qkv: torch.Tensor, q_off: int, k_off: int, v_off: in
     hk = heads // qk_rep
     if max(q_off + hk * dk, k_off + hk * dk, v_off + heads * dv) > qkv.shape[1]:
         raise KernelError("chunk_scan: q, k or v lie outside the rows")
-    n = _chunk_row.get(bool(delta))
+    form = 2 if channel else int(delta)
+    n = _chunk_row.get(form)
     if n is None:
-        n = _chunk_row[bool(delta)] = int(_fn("chunkscan", "bw_chunk_row_floats", [c_int])(int(delta)))
+        n = _chunk_row[form] = int(_fn("chunkscan", "bw_chunk_row_floats", [c_int])(form))
     rows = torch.empty((T, heads, n), dtype=torch.float32, device=qkv.device)
     o = torch.empty((T, heads * dv), dtype=torch.float32, device=qkv.device)
-    chan = gend = None
+    chan = u0 = gend = None
     if channel:
         chan = torch.empty((T, heads, 3, dk), dtype=torch.float32, device=qkv.device)
+        u0 = torch.empty((T, heads, dv), dtype=torch.float32, device=qkv.device)
         gend = torch.empty((T // CHUNK_TOKENS + batch.R, heads, dk), dtype=torch.float32, device=qkv.device)
-    fn = _fn("chunkscan", "bw_chunk_scan", [c_int, c_void_p, c_ll, c_int, c_int, c_int] + [c_void_p] * 9 + [c_int] * 7 + [c_void_p],
+    fn = _fn("chunkscan", "bw_chunk_scan", [c_int, c_void_p, c_ll, c_int, c_int, c_int] + [c_void_p] * 10 + [c_int] * 7 + [c_void_p],
              tag=("channel" if channel else "delta" if delta else "linear") if _timings is not None else None)
-    _check(fn(2 if channel else int(delta), _ptr(qkv), qkv.stride(0), int(q_off), int(k_off), int(v_off), _ptr(decay), _ptr(second), _ptr(batch.cu_q),
-              _ptr(batch.state_slot), _ptr(rows), _ptr(chan), _ptr(gend), _ptr(state), _ptr(o), T, batch.R, heads, int(qk_rep),
+    _check(fn(form, _ptr(qkv), qkv.stride(0), int(q_off), int(k_off), int(v_off), _ptr(decay), _ptr(second), _ptr(batch.cu_q),
+              _ptr(batch.state_slot), _ptr(rows), _ptr(chan), _ptr(u0), _ptr(gend), _ptr(state), _ptr(o), T, batch.R, heads, int(qk_rep),
               dk, dv, int(state.shape[3]), _stream()), "chunk_scan")
     return o
 

@@ -10,7 +10,8 @@ No position is encoded; a query may be kept from looking out of its own block of
 A key row of the cache is [k1, k2] of one key head, so keys and values are kept once.  The attention kernels see two query heads
 per head: the first is [q1, 0], the second [0, q2], and both meet the key row in a plain product; any of the framework's attention
 kernels serves.  ``ops.conv_heads`` makes these rows, keys and values in one kernel from the float32 projections (the gate's
-columns ride in the same product), ``ops.diff_combine`` the heads from the maps.
+columns ride in the same product); the maps become heads in the attention kernels' epilogues (bfloat16) or in
+``ops.diff_combine``.
 
 The convolution's earlier inputs live in the request's slot of the cache manager's fixed-size state (position p at entry
 p mod taps).  A run that reads another run's keys and values (``shares_kv``) has a query projection and convolution of its own and
@@ -108,9 +109,9 @@ class DifferentialAttention(Mixer):
         table = batch.block_tables[pages.group]
         q = ops.conv_heads(rows, self.conv, inputs.state, batch, table, pages.k_pages, pages.v_pages, MAPS * self.nh, self.hd, MAPS,
                            self.nkv, self.dv, has_kv=owns_cache)
-        a = ops.paged_attention(q, pages.k_pages, pages.v_pages, batch, table, MAPS * self.nh, None, self.scale, self.chunk)
-        gate = rows[:, self.C:self.C + self.nh] if self.gated else None
-        return ops.diff_combine(a, self.nh, self.dv, self.lam, self.eps, 1.0 - self.diff, gate, self.ctx.dtype)
+        gate = (rows[:, self.C:self.C + self.nh], self.dv, "head") if self.gated else None
+        return ops.paged_attention(q, pages.k_pages, pages.v_pages, batch, table, MAPS * self.nh, None, self.scale, self.chunk,
+                                   gate=gate, diff=(self.lam, self.eps, 1.0 - self.diff, self.dv))
 
     def forward(self, x, residual, batch, cache, owns_cache: bool = True, accumulate: bool = True) -> None:
         y = self.from_projection(self.proj(x, out_dtype=torch.float32), batch, cache, owns_cache)
