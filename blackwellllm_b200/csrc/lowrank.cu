@@ -29,7 +29,7 @@ struct LowRankParams {
 };
 
 __device__ __forceinline__ float finish(const Part& q, int c, float z) {
-    if (q.kind == PART_SIGMOID) return 1.f / (1.f + expf(-z));
+    if (q.kind == PART_SIGMOID) return __fdividef(1.f, 1.f + expf(-z));      // (z < -87: the quotient's flush to zero is the sigmoid's)
     z += q.bias[c];
     const float d = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
     return expf(q.A[c / q.per] * d);
@@ -82,10 +82,8 @@ lowrank_f32_kernel(LowRankParams p) {
     }
 }
 
-// bfloat16 weights: a block of 4 warps makes 64 tokens x 64 outputs, warp w the tokens 16 w ..; 64 inner values at a time;
-// rows of shared memory padded to 144 bytes, so that the 8 rows of an ldmatrix fall into different banks
-constexpr int MT = 64, MO = 64, MK = 64, MROW = (MK + 8) * 2;
-
+// bfloat16 weights.  Both forms add, per 16 inner values in rising order, the low half's product and then the high half's, so a row's
+// result is the same in either.
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
@@ -100,89 +98,171 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
     hi = *reinterpret_cast<const uint32_t*>(&h);
     lo = bw::pack_bf16x2(a - __low2float(h), b - __high2float(h));
 }
+__device__ __forceinline__ void store_pair(const Part& q, int row, int c, float z0, float z1) {
+    float* dst = q.out + (size_t)row * q.n_out;
+    if (c + 1 < q.n_out && (((uintptr_t)(dst + c)) & 7) == 0)
+        *reinterpret_cast<float2*>(dst + c) = make_float2(finish(q, c, z0), finish(q, c + 1, z1));
+    else {
+        if (c < q.n_out) dst[c] = finish(q, c, z0);
+        if (c + 1 < q.n_out) dst[c + 1] = finish(q, c + 1, z1);
+    }
+}
 
+// Up to 16 tokens: a warp makes 8 outputs, operands straight into registers, no barrier; the weights are requested before the wait
+// for the kernels before.
+constexpr int FEW = 16, KR = 128;      // inner values at a time
 __global__ void __launch_bounds__(128)
+lowrank_few_kernel(LowRankParams p) {
+    BW_PDL_TRIGGER();
+    const Part q = p.part[blockIdx.z];
+    const int lane = threadIdx.x & 31, o0 = (blockIdx.x * 4 + (threadIdx.x >> 5)) * 8;
+    if (o0 >= q.n_out) return;
+    const bf16* w = (const bf16*)q.w;
+    const int o = o0 + (lane >> 2), k = 2 * (lane & 3);
+    const bool vec = (p.vec >> blockIdx.z) & 1;
+    float acc[1][4] = {{0.f, 0.f, 0.f, 0.f}};
+    for (int k0 = 0; k0 < q.rank; k0 += KR) {
+        uint32_t b[KR / 16][2];
+#pragma unroll
+        for (int ks = 0; ks < KR / 16; ++ks)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int kk = k0 + ks * 16 + e * 8 + k;
+                const bf16* src = w + (size_t)o * q.rank + kk;
+                if (vec) b[ks][e] = (o < q.n_out && kk < q.rank) ? __ldg(reinterpret_cast<const uint32_t*>(src)) : 0u;
+                else {
+                    const float lo = (o < q.n_out && kk < q.rank) ? __bfloat162float(src[0]) : 0.f;
+                    const float hi = (o < q.n_out && kk + 1 < q.rank) ? __bfloat162float(src[1]) : 0.f;
+                    b[ks][e] = bw::pack_bf16x2(lo, hi);
+                }
+            }
+        if (k0 == 0) BW_PDL_WAIT();
+        float2 x[KR / 16][4];
+#pragma unroll
+        for (int ks = 0; ks < KR / 16; ++ks)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {       // rows lane / 4 (and + 8), inner values k (and + 8)
+                const int t = (lane >> 2) + 8 * (e & 1), kk = k0 + ks * 16 + 8 * (e >> 1) + k;
+                const float* src = p.x + (size_t)t * p.ld + q.x_off + kk;
+                x[ks][e] = make_float2(0.f, 0.f);
+                if (t < p.T) {
+                    if (vec) { if (kk < q.rank) x[ks][e] = *reinterpret_cast<const float2*>(src); }
+                    else {
+                        if (kk < q.rank) x[ks][e].x = src[0];
+                        if (kk + 1 < q.rank) x[ks][e].y = src[1];
+                    }
+                }
+            }
+#pragma unroll
+        for (int ks = 0; ks < KR / 16; ++ks) {
+            if (k0 + ks * 16 >= q.rank) break;
+            uint32_t ah[4], al[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) split2(x[ks][e].x, x[ks][e].y, ah[e], al[e]);
+            mma_bf16(acc[0], al, b[ks][0], b[ks][1]);
+            mma_bf16(acc[0], ah, b[ks][0], b[ks][1]);
+        }
+    }
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const int row = (lane >> 2) + 8 * half;
+        if (row < p.T) store_pair(q, row, o0 + k, acc[0][2 * half], acc[0][2 * half + 1]);
+    }
+}
+
+// Many tokens: a block of 8 warps makes 64 tokens x 128 outputs, each warp 16 tokens x two stretches of 32 outputs; 128 inner values at
+// a time; the weights are requested before the wait for the kernels before.  Rows of shared memory are padded to 272 bytes, so that
+// the 8 rows of an ldmatrix fall into different banks.
+constexpr int MT = 64, MO = 128, MROW = (KR + 8) * 2;
+constexpr int SMEM_MMA = (2 * MT + MO) * MROW;
+
+__global__ void __launch_bounds__(256)
 lowrank_mma_kernel(LowRankParams p) {
     BW_PDL_TRIGGER();
     const Part q = p.part[blockIdx.z];
     const int t0 = blockIdx.x * MT, o0 = blockIdx.y * MO;
     if (o0 >= q.n_out) return;
-    __shared__ __align__(16) uint8_t xh[MT * MROW], xl[MT * MROW], ws[MO * MROW];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    extern __shared__ __align__(16) uint8_t smem[];
+    uint8_t *xh = smem, *xl = smem + MT * MROW, *ws = smem + 2 * MT * MROW;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wm = warp & 3, wn = warp >> 2;
     const bf16* w = (const bf16*)q.w;
-    float acc[MO / 8][4];
+    float acc[2][4][4];
 #pragma unroll
-    for (int j = 0; j < MO / 8; ++j) { acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f; }
-    const int srow = threadIdx.x >> 1, scol = (threadIdx.x & 1) * 32;       // this thread stages 32 inner values of a row of each
-    const int t = t0 + srow, o = o0 + srow;
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) { acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f; }
     const bool vec = (p.vec >> blockIdx.z) & 1;
-    BW_PDL_WAIT();
-    for (int k0 = 0; k0 < q.rank; k0 += MK) {
-        const float* src = p.x + (size_t)(t < p.T ? t : 0) * p.ld + q.x_off + k0 + scol;
-        const bf16* wsrc = w + (size_t)(o < q.n_out ? o : 0) * q.rank + k0 + scol;
+    for (int k0 = 0; k0 < q.rank; k0 += KR) {
+        // eight inner values of a weight row, then of a token row, per step of a thread
 #pragma unroll
-        for (int c = 0; c < 32; c += 8) {
-            float v[8];
-            uint4 wv = make_uint4(0, 0, 0, 0);
+        for (int i = 0; i < MO * (KR / 8) / 256; ++i) {
+            const int idx = threadIdx.x + i * 256, r = idx / (KR / 8), c = idx % (KR / 8) * 8, o = o0 + r;
+            uint8_t* dst = ws + r * MROW + c * 2;
+            const bf16* src = w + (size_t)(o < q.n_out ? o : 0) * q.rank + k0 + c;
             if (vec) {           // (the inner size is a multiple of 8: a stretch of eight is inside or outside)
-                const bool in = k0 + scol + c < q.rank;
-                const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-                const float4 a = in && t < p.T ? *reinterpret_cast<const float4*>(src + c) : zero;
-                const float4 b = in && t < p.T ? *reinterpret_cast<const float4*>(src + c + 4) : zero;
-                v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-                if (in && o < q.n_out) wv = __ldg(reinterpret_cast<const uint4*>(wsrc + c));
+                const bool in = o < q.n_out && k0 + c < q.rank;
+                const int n = in ? 16 : 0;
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" :: "r"(smem_addr(dst)), "l"(in ? src : w), "r"(n) : "memory");
             } else {
-                bf16 we[8];
+                bf16 e[8];
 #pragma unroll
-                for (int i = 0; i < 8; ++i) {
-                    const bool ok = k0 + scol + c + i < q.rank;
-                    v[i] = (ok && t < p.T) ? src[c + i] : 0.f;
-                    we[i] = (ok && o < q.n_out) ? wsrc[c + i] : __float2bfloat16_rn(0.f);
-                }
-                wv = *reinterpret_cast<const uint4*>(we);
+                for (int j = 0; j < 8; ++j) e[j] = (o < q.n_out && k0 + c + j < q.rank) ? src[j] : __float2bfloat16_rn(0.f);
+                *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(e);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        if (k0 == 0) BW_PDL_WAIT();
+#pragma unroll
+        for (int i = 0; i < MT * (KR / 8) / 256; ++i) {
+            const int idx = threadIdx.x + i * 256, r = idx / (KR / 8), c = idx % (KR / 8) * 8, t = t0 + r;
+            const float* src = p.x + (size_t)(t < p.T ? t : 0) * p.ld + q.x_off + k0 + c;
+            float v[8];
+            if (vec) {
+                const bool in = t < p.T && k0 + c < q.rank;
+                const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+                const float4 a = in ? *reinterpret_cast<const float4*>(src) : zero, b = in ? *reinterpret_cast<const float4*>(src + 4) : zero;
+                v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+            } else {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) v[j] = (t < p.T && k0 + c + j < q.rank) ? src[j] : 0.f;
             }
             uint4 hi, lo;
             split2(v[0], v[1], hi.x, lo.x); split2(v[2], v[3], hi.y, lo.y); split2(v[4], v[5], hi.z, lo.z); split2(v[6], v[7], hi.w, lo.w);
-            *reinterpret_cast<uint4*>(xh + srow * MROW + (scol + c) * 2) = hi;
-            *reinterpret_cast<uint4*>(xl + srow * MROW + (scol + c) * 2) = lo;
-            *reinterpret_cast<uint4*>(ws + srow * MROW + (scol + c) * 2) = wv;
+            *reinterpret_cast<uint4*>(xh + r * MROW + c * 2) = hi;
+            *reinterpret_cast<uint4*>(xl + r * MROW + c * 2) = lo;
         }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
 #pragma unroll
-        for (int ks = 0; ks < MK / 16; ++ks) {
+        for (int ks = 0; ks < KR / 16; ++ks) {
             if (k0 + ks * 16 >= q.rank) break;
             uint32_t ah[4], al[4];
-            const int at = (warp * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * MROW + 16 * (lane >> 4) + ks * 32;
+            const int at = (wm * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * MROW + 16 * (lane >> 4) + ks * 32;
             ldsm_x4(smem_addr(xh) + at, ah);
             ldsm_x4(smem_addr(xl) + at, al);
 #pragma unroll
-            for (int nb = 0; nb < MO / 16; ++nb) {
-                uint32_t b[4];
-                ldsm_x4(smem_addr(ws) + (nb * 16 + (lane & 7) + 8 * (lane >> 4)) * MROW + 16 * ((lane >> 3) & 1) + ks * 32, b);
-                mma_bf16(acc[2 * nb], al, b[0], b[1]);
-                mma_bf16(acc[2 * nb + 1], al, b[2], b[3]);
-                mma_bf16(acc[2 * nb], ah, b[0], b[1]);
-                mma_bf16(acc[2 * nb + 1], ah, b[2], b[3]);
-            }
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int nb = 0; nb < 2; ++nb) {
+                    uint32_t b[4];
+                    ldsm_x4(smem_addr(ws) + (i * 64 + wn * 32 + nb * 16 + (lane & 7) + 8 * (lane >> 4)) * MROW + 16 * ((lane >> 3) & 1) + ks * 32, b);
+                    mma_bf16(acc[i][2 * nb], al, b[0], b[1]);
+                    mma_bf16(acc[i][2 * nb + 1], al, b[2], b[3]);
+                    mma_bf16(acc[i][2 * nb], ah, b[0], b[1]);
+                    mma_bf16(acc[i][2 * nb + 1], ah, b[2], b[3]);
+                }
         }
-        __syncthreads();
+        if (k0 + KR < q.rank) __syncthreads();
     }
-    const bool pairs = (q.n_out & 1) == 0 && ((uintptr_t)q.out & 7) == 0;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
-        const int row = t0 + warp * 16 + (lane >> 2) + 8 * half;
+        const int row = t0 + wm * 16 + (lane >> 2) + 8 * half;
         if (row >= p.T) continue;
-        float* dst = q.out + (size_t)row * q.n_out;
 #pragma unroll
-        for (int j = 0; j < MO / 8; ++j) {
-            const int c = o0 + j * 8 + 2 * (lane & 3);
-            if (pairs && c + 1 < q.n_out)
-                *reinterpret_cast<float2*>(dst + c) = make_float2(finish(q, c, acc[j][2 * half]), finish(q, c + 1, acc[j][2 * half + 1]));
-            else {
-                if (c < q.n_out) dst[c] = finish(q, c, acc[j][2 * half]);
-                if (c + 1 < q.n_out) dst[c + 1] = finish(q, c + 1, acc[j][2 * half + 1]);
-            }
-        }
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                store_pair(q, row, o0 + i * 64 + wn * 32 + j * 8 + 2 * (lane & 3), acc[i][j][2 * half], acc[i][j][2 * half + 1]);
     }
 }
 
@@ -213,7 +293,14 @@ BW_EXPORT int bw_lowrank_gates(const float* x, long long ld, int w_type, int T, 
     if (w_type == BW_F32)
         bw::launch((lowrank_f32_kernel), dim3((T + FT - 1) / FT, (widest + FO - 1) / FO, n), dim3(256), 0, s, p);
     else if (w_type == BW_BF16)
-        bw::launch((lowrank_mma_kernel), dim3((T + MT - 1) / MT, (widest + MO - 1) / MO, n), dim3(128), 0, s, p);
+    {
+        static bool raised[bw::MAX_DEVICES] = {};
+        if (T <= FEW) bw::launch((lowrank_few_kernel), dim3((widest + 31) / 32, 1, n), dim3(128), 0, s, p);
+        else {
+            if (bw::allow_dynamic_smem(lowrank_mma_kernel, SMEM_MMA, raised) != cudaSuccess) return BW_ERR_DRIVER;
+            bw::launch((lowrank_mma_kernel), dim3((T + MT - 1) / MT, (widest + MO - 1) / MO, n), dim3(256), SMEM_MMA, s, p);
+        }
+    }
     else return BW_ERR_BAD_ARG;
     BW_LAUNCH_CHECK();
     return 0;
