@@ -199,7 +199,7 @@ template <int DKP>
 __global__ void __launch_bounds__(128)
 chunk_rows_channel_kernel(ChunkParams p) {
     BW_PDL_TRIGGER();
-    constexpr int lds = DKP + 4, CH = DKP / 8;             // channels of a lane
+    constexpr int lds = DKP + 4;
     const int h = blockIdx.y, hk = h / p.rep;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     int t0, n, index;
@@ -236,12 +236,13 @@ chunk_rows_channel_kernel(ChunkParams p) {
     }
     __syncthreads();
     {
-        // Warp w has the tokens s = 8 w .. 8 w + 7, lane = 8 sl + cg two of them (8 w + 2 sl and + 1) on the channels
-        // (8 j + cg) 4 + e; z = D_ts o k_s goes along t, zero before s.
-        const int cg = lane & 7, s0 = 8 * warp + 2 * (lane >> 3);
-        bw::f32x2 z[2][CH / 2];
+        // Warp w has the tokens s = 8 w .. 8 w + 7, lane = NG sl + cg the NS of them from 8 w + NS sl on, on the channels
+        // (NG j + cg) 4 + e; z = D_ts o k_s goes along t, zero before s.
+        constexpr int NG = DKP >= 64 ? 16 : 8, NS = NG / 4, CH = DKP / NG;
+        const int cg = lane % NG, s0 = 8 * warp + NS * (lane / NG);
+        bw::f32x2 z[NS][CH / 2];
 #pragma unroll
-        for (int u = 0; u < 2; ++u)
+        for (int u = 0; u < NS; ++u)
 #pragma unroll
             for (int j = 0; j < CH / 2; ++j) z[u][j] = 0;              // (pairs of zeros)
         for (int idx = threadIdx.x; idx < C * (C + 4); idx += 128) kk[idx] = kq[idx] = 0.f;
@@ -249,31 +250,38 @@ chunk_rows_channel_kernel(ChunkParams p) {
         const ulonglong2 *k4 = reinterpret_cast<const ulonglong2*>(ks) + cg, *q4 = reinterpret_cast<const ulonglong2*>(qs) + cg,
                          *g4 = reinterpret_cast<const ulonglong2*>(gs) + cg;
         for (int t = 8 * warp; t < n; ++t) {
-            bw::f32x2 a[2] = {0, 0}, b[2] = {0, 0};
+            bw::f32x2 a[2 * NS];                                       // sums with k_t, then with q_t
+#pragma unroll
+            for (int u = 0; u < 2 * NS; ++u) a[u] = 0;
             const bool near = t < 8 * warp + 8;                        // (uniform over the warp)
 #pragma unroll
             for (int j = 0; j < CH / 4; ++j) {
-                const int at = t * (lds / 4) + 8 * j;
+                const int at = t * (lds / 4) + NG * j;
                 const ulonglong2 k = k4[at], q = q4[at], g = g4[at];
 #pragma unroll
-                for (int u = 0; u < 2; ++u) {
+                for (int u = 0; u < NS; ++u) {
                     z[u][2 * j] = bw::mul2(z[u][2 * j], g.x);
                     z[u][2 * j + 1] = bw::mul2(z[u][2 * j + 1], g.y);
                     if (near && t == s0 + u) { z[u][2 * j] = k.x; z[u][2 * j + 1] = k.y; }
                     a[u] = bw::fma2(z[u][2 * j], k.x, a[u]);
                     a[u] = bw::fma2(z[u][2 * j + 1], k.y, a[u]);
-                    b[u] = bw::fma2(z[u][2 * j], q.x, b[u]);
-                    b[u] = bw::fma2(z[u][2 * j + 1], q.y, b[u]);
+                    a[NS + u] = bw::fma2(z[u][2 * j], q.x, a[NS + u]);
+                    a[NS + u] = bw::fma2(z[u][2 * j + 1], q.y, a[NS + u]);
                 }
             }
-            // four sums over the eight lanes of a token pair: the lane ends with the one its bits 2 and 1 name
-            const float a0 = bw::sum2(a[0]), a1 = bw::sum2(a[1]), b0 = bw::sum2(b[0]), b1 = bw::sum2(b[1]);
-            const bool hi4 = lane & 4, hi2 = lane & 2;
-            const float x0 = (hi4 ? b0 : a0) + __shfl_xor_sync(0xffffffffu, hi4 ? a0 : b0, 4);
-            const float x1 = (hi4 ? b1 : a1) + __shfl_xor_sync(0xffffffffu, hi4 ? a1 : b1, 4);
-            float x = (hi2 ? x1 : x0) + __shfl_xor_sync(0xffffffffu, hi2 ? x0 : x1, 2);
-            x += __shfl_xor_sync(0xffffffffu, x, 1);
-            if (!(lane & 1)) (hi4 ? kq : kk)[t * (C + 4) + s0 + (hi2 ? 1 : 0)] = x;
+            // 2 NS sums over the NG lanes of a group of tokens: at every step a lane keeps half of its sums and gives the other half
+            // away; it ends with the one that its bits from NG / 2 down to 2 name
+            float v[2 * NS];
+#pragma unroll
+            for (int u = 0; u < 2 * NS; ++u) v[u] = bw::sum2(a[u]);
+#pragma unroll
+            for (int m = NG / 2, w = NS; m >= 2; m >>= 1, w >>= 1) {
+                const bool hi = lane & m;
+#pragma unroll
+                for (int u = 0; u < w; ++u) v[u] = (hi ? v[w + u] : v[u]) + __shfl_xor_sync(0xffffffffu, hi ? v[u] : v[w + u], m);
+            }
+            v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
+            if (!(lane & 1)) ((lane & (NG / 2)) ? kq : kk)[t * (C + 4) + s0 + ((lane & (NG / 2 - 1)) >> 1)] = v[0];
         }
     }
     __syncthreads();
@@ -324,28 +332,40 @@ chunk_rows_channel_kernel(ChunkParams p) {
         }
     }
     __syncthreads();
-    // W = T beta (G o K) and U0 = T beta V: a thread per column, which it keeps in registers
+    // W = T beta (G o K) and U0 = T beta V: two columns a thread, which it keeps in registers
     const int cols = p.dk + p.dv;
-    for (int c = threadIdx.x; c < cols; c += 128) {
-        const bool is_k = c < p.dk;
-        float x[C];
-        const float* v = p.qkv + (size_t)t0 * p.ld + p.v_off + h * p.dv + (c - p.dk);
+    for (int c0 = threadIdx.x; c0 < cols; c0 += 256) {
+        float x[2][C];
+        float* dst[2];
+        size_t step[2];
 #pragma unroll
-        for (int t = 0; t < C; ++t) x[t] = is_k ? ks[t * lds + c] : (t < n ? v[(size_t)t * p.ld] : 0.f);
-        float* dst = is_k ? p.chan + ((size_t)t0 * p.heads + h) * 3 * p.dk + c : p.u0 + ((size_t)t0 * p.heads + h) * p.dv + (c - p.dk);
-        const size_t step = (size_t)p.heads * (is_k ? 3 * p.dk : p.dv);
+        for (int u = 0; u < 2; ++u) {
+            const int c = c0 + 128 * u;
+            const bool is_k = c < p.dk, there = c < cols;
+            const float* v = p.qkv + (size_t)t0 * p.ld + p.v_off + h * p.dv + (c - p.dk);
+            dst[u] = is_k ? p.chan + ((size_t)t0 * p.heads + h) * 3 * p.dk + c : (there ? p.u0 + ((size_t)t0 * p.heads + h) * p.dv + (c - p.dk) : nullptr);
+            step[u] = (size_t)p.heads * (is_k ? 3 * p.dk : p.dv);
+#pragma unroll
+            for (int t = 0; t < C; ++t) x[u][t] = is_k ? ks[t * lds + c] : (there && t < n ? v[(size_t)t * p.ld] : 0.f);
+        }
 #pragma unroll
         for (int t = 0; t < C; ++t) {
-            float a0 = 0.f, a1 = 0.f;
+            float a[2][2] = {{0.f, 0.f}, {0.f, 0.f}};
 #pragma unroll
             for (int j = 0; j <= t; j += 4) {
                 const float4 m = *reinterpret_cast<const float4*>(kk + t * (C + 4) + j);     // (zeros above the diagonal)
-                a0 = fmaf(m.x, x[j], a0);
-                a1 = fmaf(m.y, x[j + 1], a1);
-                a0 = fmaf(m.z, x[j + 2], a0);
-                a1 = fmaf(m.w, x[j + 3], a1);
+#pragma unroll
+                for (int u = 0; u < 2; ++u) {
+                    a[u][0] = fmaf(m.x, x[u][j], a[u][0]);
+                    a[u][1] = fmaf(m.y, x[u][j + 1], a[u][1]);
+                    a[u][0] = fmaf(m.z, x[u][j + 2], a[u][0]);
+                    a[u][1] = fmaf(m.w, x[u][j + 3], a[u][1]);
+                }
             }
-            if (t < n) dst[t * step] = a0 + a1;
+            if (t < n) {
+                dst[0][t * step[0]] = a[0][0] + a[0][1];
+                if (dst[1]) dst[1][t * step[1]] = a[1][0] + a[1][1];
+            }
         }
     }
 }

@@ -28,11 +28,10 @@ struct LowRankParams {
     Part part[MAX_PARTS];
 };
 
+__device__ __forceinline__ float sigmoid(float z) { return __fdividef(1.f, 1.f + expf(-z)); }   // (a quotient flushed to zero is the sigmoid's)
+__device__ __forceinline__ float decay(float A, float z) { return expf(A * (fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))))); }
 __device__ __forceinline__ float finish(const Part& q, int c, float z) {
-    if (q.kind == PART_SIGMOID) return __fdividef(1.f, 1.f + expf(-z));      // (z < -87: the quotient's flush to zero is the sigmoid's)
-    z += q.bias[c];
-    const float d = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
-    return expf(q.A[c / q.per] * d);
+    return q.kind == PART_SIGMOID ? sigmoid(z) : decay(q.A[c / q.per], z + q.bias[c]);
 }
 
 // float32 weights: 32 tokens x 64 outputs a block, 32 inner values at a time
@@ -176,7 +175,7 @@ lowrank_few_kernel(LowRankParams p) {
 constexpr int MT = 64, MO = 128, MROW = (KR + 8) * 2;
 constexpr int SMEM_MMA = (2 * MT + MO) * MROW;
 
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 3)
 lowrank_mma_kernel(LowRankParams p) {
     BW_PDL_TRIGGER();
     const Part q = p.part[blockIdx.z];
@@ -254,16 +253,42 @@ lowrank_mma_kernel(LowRankParams p) {
         }
         if (k0 + KR < q.rank) __syncthreads();
     }
+    // a column's head and bias serve both of the lane's rows; the columns rise
+    const bool dec = q.kind == PART_DECAY;
+    const bool pairs = (q.n_out & 1) == 0 && ((uintptr_t)q.out & 7) == 0;
+    int head = dec ? (o0 + wn * 32) / q.per : 0, end = dec ? (head + 1) * q.per : 0;
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-        const int row = t0 + wm * 16 + (lane >> 2) + 8 * half;
-        if (row >= p.T) continue;
+    for (int i = 0; i < 2; ++i)
 #pragma unroll
-        for (int i = 0; i < 2; ++i)
+        for (int j = 0; j < 4; ++j) {
+            const int c = o0 + i * 64 + wn * 32 + j * 8 + 2 * (lane & 3);
+            float A[2] = {0.f, 0.f}, bias[2] = {0.f, 0.f};
+            if (dec) {
 #pragma unroll
-            for (int j = 0; j < 4; ++j)
-                store_pair(q, row, o0 + i * 64 + wn * 32 + j * 8 + 2 * (lane & 3), acc[i][j][2 * half], acc[i][j][2 * half + 1]);
-    }
+                for (int e = 0; e < 2; ++e)
+                    if (c + e < q.n_out) {
+                        while (c + e >= end) { ++head; end += q.per; }
+                        A[e] = q.A[head]; bias[e] = q.bias[c + e];
+                    }
+            }
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int row = t0 + wm * 16 + (lane >> 2) + 8 * half;
+                if (row >= p.T || c >= q.n_out) continue;
+                float r[2];
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const float z = acc[i][j][2 * half + e];
+                    r[e] = dec ? decay(A[e], z + bias[e]) : sigmoid(z);
+                }
+                float* dst = q.out + (size_t)row * q.n_out + c;
+                if (pairs) *reinterpret_cast<float2*>(dst) = make_float2(r[0], r[1]);
+                else {
+                    dst[0] = r[0];
+                    if (c + 1 < q.n_out) dst[1] = r[1];
+                }
+            }
+        }
 }
 
 }  // namespace
