@@ -196,10 +196,10 @@ chunk_rows_kernel(ChunkParams p) {
 
 // The same for a decay per key channel.  One block per (chunk, head).  DKP: dk up to a multiple of 32.
 template <int DKP>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, DKP <= 128 ? 4 : 1)
 chunk_rows_channel_kernel(ChunkParams p) {
     BW_PDL_TRIGGER();
-    constexpr int lds = DKP + 4;
+    constexpr int lds = DKP;
     const int h = blockIdx.y, hk = h / p.rep;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     int t0, n, index;
@@ -209,8 +209,9 @@ chunk_rows_channel_kernel(ChunkParams p) {
     float* ks = sm;                        // [C][lds] each
     float* qs = ks + C * lds;
     float* gs = qs + C * lds;
-    float* kk = gs + C * lds;              // [C][C + 4]: sum_c k_s D_ts k_t, turned into L in place
-    float* kq = kk + C * (C + 4);          // [C][C + 4]
+    float* kk = gs + C * lds;              // [C][C + 4]: sum_c k_s D_ts k_t, turned into L and then into T beta in place
+    float* m_rows = p.rows + ((size_t)t0 * p.heads + h) * ROW_CHANNEL;      // M: what the walk reads of it (8 x 8 blocks up to the diagonal's)
+    const size_t m_step = (size_t)p.heads * ROW_CHANNEL;
     BW_PDL_WAIT();
     if (p.vec & 1) {
 #pragma unroll 4
@@ -245,7 +246,7 @@ chunk_rows_channel_kernel(ChunkParams p) {
         for (int u = 0; u < NS; ++u)
 #pragma unroll
             for (int j = 0; j < CH / 2; ++j) z[u][j] = 0;              // (pairs of zeros)
-        for (int idx = threadIdx.x; idx < C * (C + 4); idx += 128) kk[idx] = kq[idx] = 0.f;
+        for (int idx = threadIdx.x; idx < C * (C + 4); idx += 128) kk[idx] = 0.f;
         __syncthreads();
         const ulonglong2 *k4 = reinterpret_cast<const ulonglong2*>(ks) + cg, *q4 = reinterpret_cast<const ulonglong2*>(qs) + cg,
                          *g4 = reinterpret_cast<const ulonglong2*>(gs) + cg;
@@ -281,17 +282,15 @@ chunk_rows_channel_kernel(ChunkParams p) {
                 for (int u = 0; u < w; ++u) v[u] = (hi ? v[w + u] : v[u]) + __shfl_xor_sync(0xffffffffu, hi ? v[u] : v[w + u], m);
             }
             v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
-            if (!(lane & 1)) ((lane & (NG / 2)) ? kq : kk)[t * (C + 4) + s0 + ((lane & (NG / 2 - 1)) >> 1)] = v[0];
+            if (!(lane & 1)) *((lane & (NG / 2)) ? m_rows + t * m_step + s0 + ((lane & (NG / 2 - 1)) >> 1)
+                                                 : kk + t * (C + 4) + s0 + ((lane & (NG / 2 - 1)) >> 1)) = v[0];
         }
     }
     __syncthreads();
     if (warp == 0) {
-        float* base = p.rows + ((size_t)t0 * p.heads + h) * ROW_CHANNEL;
-        const size_t step = (size_t)p.heads * ROW_CHANNEL;
         const float beta = lane < n ? p.second[(size_t)(t0 + lane) * p.heads + h] : 0.f;
         for (int t = 0; t < n; ++t) {
             const float bt = __shfl_sync(0xffffffffu, beta, t);
-            base[t * step + lane] = t >= lane ? kq[t * (C + 4) + lane] : 0.f;
             kk[t * (C + 4) + lane] = t > lane ? bt * kk[t * (C + 4) + lane] : 0.f;
         }
         __syncwarp();
@@ -350,6 +349,7 @@ chunk_rows_channel_kernel(ChunkParams p) {
         }
 #pragma unroll
         for (int t = 0; t < C; ++t) {
+            asm volatile("" ::: "memory");        // (rows of T beta are not fetched ahead: there are no registers for that)
             float a[2][2] = {{0.f, 0.f}, {0.f, 0.f}};
 #pragma unroll
             for (int j = 0; j <= t; j += 4) {
@@ -700,7 +700,7 @@ int launch_rows(const ChunkParams& p, cudaStream_t s) {
 
 template <int DKP>
 int launch_rows_channel(const ChunkParams& p, cudaStream_t s) {
-    constexpr int smem = (3 * C * (DKP + 4) + 2 * C * (C + 4)) * (int)sizeof(float);
+    constexpr int smem = (3 * C * DKP + C * (C + 4)) * (int)sizeof(float);
     static bool raised[bw::MAX_DEVICES] = {};
     if (bw::allow_dynamic_smem(chunk_rows_channel_kernel<DKP>, smem, raised) != cudaSuccess) return BW_ERR_DRIVER;
     bw::launch((chunk_rows_channel_kernel<DKP>), dim3(p.T / C + p.R, p.heads), dim3(128), smem, s, p);

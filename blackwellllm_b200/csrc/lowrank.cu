@@ -253,42 +253,43 @@ lowrank_mma_kernel(LowRankParams p) {
         }
         if (k0 + KR < q.rank) __syncthreads();
     }
-    // a column's head and bias serve both of the lane's rows; the columns rise
-    const bool dec = q.kind == PART_DECAY;
-    const bool pairs = (q.n_out & 1) == 0 && ((uintptr_t)q.out & 7) == 0;
-    int head = dec ? (o0 + wn * 32) / q.per : 0, end = dec ? (head + 1) * q.per : 0;
+    // the sums change places through shared memory: a thread finishes four neighbouring columns of every eighth row (few
+    // instructions for the many results, whole sectors for the stores)
+    constexpr int ZS = MO + 4;
+    static_assert(MT * ZS * 4 <= SMEM_MMA, "the sums take the operands' place");
+    float* zs = reinterpret_cast<float*>(smem);
+    __syncthreads();
 #pragma unroll
     for (int i = 0; i < 2; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            const int c = o0 + i * 64 + wn * 32 + j * 8 + 2 * (lane & 3);
-            float A[2] = {0.f, 0.f}, bias[2] = {0.f, 0.f};
-            if (dec) {
+        for (int j = 0; j < 4; ++j)
 #pragma unroll
-                for (int e = 0; e < 2; ++e)
-                    if (c + e < q.n_out) {
-                        while (c + e >= end) { ++head; end += q.per; }
-                        A[e] = q.A[head]; bias[e] = q.bias[c + e];
-                    }
-            }
+            for (int half = 0; half < 2; ++half)
+                *reinterpret_cast<float2*>(zs + (wm * 16 + (lane >> 2) + 8 * half) * ZS + i * 64 + wn * 32 + j * 8 + 2 * (lane & 3)) =
+                    make_float2(acc[i][j][2 * half], acc[i][j][2 * half + 1]);
+    __syncthreads();
+    const int c = o0 + lane * 4, n = min(4, q.n_out - c);
+    if (n <= 0) return;
+    const bool dec = q.kind == PART_DECAY, quads = (q.n_out & 3) == 0 && ((uintptr_t)q.out & 15) == 0;
+    float A[4] = {0.f, 0.f, 0.f, 0.f}, bias[4] = {0.f, 0.f, 0.f, 0.f};
+    if (dec)
+        for (int e = 0; e < n; ++e) { A[e] = q.A[(c + e) / q.per]; bias[e] = q.bias[c + e]; }
+#pragma unroll 1
+    for (int r = warp; r < MT && t0 + r < p.T; r += 8) {
+        const float4 z = *reinterpret_cast<const float4*>(zs + r * ZS + lane * 4);
+        float v[4] = {z.x, z.y, z.z, z.w};
+        if (dec) {
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                const int row = t0 + wm * 16 + (lane >> 2) + 8 * half;
-                if (row >= p.T || c >= q.n_out) continue;
-                float r[2];
+            for (int e = 0; e < 4; ++e) v[e] = decay(A[e], v[e] + bias[e]);
+        } else {
 #pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const float z = acc[i][j][2 * half + e];
-                    r[e] = dec ? decay(A[e], z + bias[e]) : sigmoid(z);
-                }
-                float* dst = q.out + (size_t)row * q.n_out + c;
-                if (pairs) *reinterpret_cast<float2*>(dst) = make_float2(r[0], r[1]);
-                else {
-                    dst[0] = r[0];
-                    if (c + 1 < q.n_out) dst[1] = r[1];
-                }
-            }
+            for (int e = 0; e < 4; ++e) v[e] = sigmoid(v[e]);
         }
+        float* dst = q.out + (size_t)(t0 + r) * q.n_out + c;
+        if (quads) *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+        else
+            for (int e = 0; e < n; ++e) dst[e] = v[e];
+    }
 }
 
 }  // namespace

@@ -416,6 +416,42 @@ def test_one_loud_key_at_the_edge_of_a_block_of_positions(ops, dtype, dim, vdim,
     assert float((results[edge] - results[edge - 1]).abs().max()) > 0.3 and float((results[edge - 1] - results[3]).abs().max()) < 1e-9
 
 
+@pytest.mark.parametrize("hd,nh,nkv,page", [(48, 4, 2, 16), (64, 4, 1, 8), (64, 32, 4, 16), (128, 8, 4, 16), (192, 4, 2, 32), (256, 4, 1, 64), (16, 16, 1, 8),
+                                            (80, 6, 3, 16), (64, 16, 1, 5), (128, 16, 1, 16), (64, 40, 2, 16), (272, 4, 2, 16)])
+@pytest.mark.parametrize("q_lens,kv_lens", [([1, 1], [700, 33]), ([1], [2500]), ([50, 1, 3], [400, 90, 3]), ([130], [131]), ([1] * 9, [70] * 9)])
+def test_pairs_of_heads_become_one_in_the_attention_kernels(ops, hd, nh, nkv, page, q_lens, kv_lens):
+    """bfloat16, every kernel's epilogue (prompt tiles on either tensor path, one key slice, few and many slices): a1 - lambda a2 in
+    float32 before anything is rounded, over the channels that are values, times the gate of the head.  (Maps that nearly cancel:
+    outputs rounded one by one would be off by far more than the bound.)"""
+    from test_kernels_gpu import FakeBatch, paged_case
+    dv = hd - hd // 8
+    chunk, eps, factor = 200, 1e-6, 0.7
+
+    def spike(r, q, k, v):
+        v[..., dv:] = 0
+        q[:, 1::2] = q[:, 0::2] + 0.1 * q[:, 1::2]
+    q, kp, vp, table, refs = paged_case(q_lens, kv_lens, nh, nkv, hd, page, torch.bfloat16, seed=hd, spike=spike)
+    T, H = sum(q_lens), nh // 2
+    lam = torch.tensor([0.9])
+    gate = rnd(T, H + 3, seed=1)
+    batch = FakeBatch(q_lens, kv_lens)
+    scale = 0.5 * hd ** -0.5
+    out = ops.paged_attention(q, kp, vp, batch, table, nh, None, scale, chunk, gate=(gate.to(DEV)[:, 2:2 + H], dv, "head"),
+                              diff=(d(lam), eps, factor, dv)).view(T, H, hd).double().cpu()
+    want = []
+    for q_, k_, v_, start in refs:
+        L = q_.shape[0]
+        seen = plain.block_mask(L, chunk)[start:]
+        maps = [plain.softmax_rows(q_[start:, h].double() @ k_[:, h // (nh // nkv)].double().T * scale, seen) @ v_[:, h // (nh // nkv), :dv].double()
+                for h in range(nh)]
+        want.append(torch.stack([plain.rms_unit(maps[2 * h] - float(lam) * maps[2 * h + 1], eps) * factor for h in range(H)], 1))
+    want = torch.cat(want) * torch.sigmoid(gate[:, 2:2 + H].double()).unsqueeze(-1)
+    assert float(out[..., dv:].abs().sum()) == 0.0
+    # (the CUDA-core kernel, for sizes the others do not take, rounds its outputs first; attention weights are bfloat16 in P V)
+    err = float((out[..., :dv] - want).abs().max()) / float(want.abs().max())
+    assert err < (0.2 if nh // nkv > 16 or hd > 256 else 0.06), err
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("hd", [48, 64])
 @pytest.mark.parametrize("q_len", [1, 2, 50])
